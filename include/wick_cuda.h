@@ -38,6 +38,7 @@ extern "C" {
 #define WICK_CUDA_ERR_CONTEXT_FULL (-5)
 #define WICK_CUDA_ERR_TIMEOUT (-6)
 #define WICK_CUDA_ERR_BAD_GGUF (-7)
+#define WICK_CUDA_ERR_BAD_MODEL (-8) /* a model folder (config.json, model.safetensors) that cannot be used */
 
 /* GGML tensor type ids of the two supported weight formats (wick/src/gguf.rs:38, :42). */
 #define WICK_DTYPE_Q4_0 2
@@ -78,6 +79,20 @@ int32_t wick_cuda_model_create(const uint8_t* gguf_host, size_t gguf_len, uint32
 /* Same, reading the file itself (GgufFile::open, gguf.rs:336-360). */
 int32_t wick_cuda_model_create_from_file(const char* path, uint32_t context_size, int32_t device,
                                          wick_cuda_model** out);
+/* The same for any model this library knows, chosen by what is at `path`: a GGUF file, or a folder with config.json (its
+ * "architecture" names the model class) and model.safetensors.  `compute` picks the arithmetic of a folder model:
+ * BF16 (the default) multiplies bfloat16 weights with bfloat16 activations and sums in f32, with everything that is
+ * sensitive (norms, scores, recurrences, residual) in f32; F32 keeps every activation in f32 and multiplies in true f32.
+ * GGUF models have one arithmetic and accept DEFAULT only.  context_size = positions a sequence can hold. */
+#define WICK_CUDA_COMPUTE_DEFAULT 0
+#define WICK_CUDA_COMPUTE_BF16 1
+#define WICK_CUDA_COMPUTE_F32 2
+int32_t wick_cuda_model_create_from_path(const char* path, uint32_t context_size, int32_t device, int32_t compute,
+                                         wick_cuda_model** out);
+/* Architecture name of the model file ("lfm2", "Nositar") and type name of a layer ("Attention", "GatedConv", or the
+ * mixer's name in config.json); "" for a NULL handle or a layer that does not exist. */
+const char* wick_cuda_model_architecture(const wick_cuda_model* m);
+const char* wick_cuda_model_layer_type(const wick_cuda_model* m, uint32_t layer);
 /* Drop. NULL is allowed. */
 void wick_cuda_model_destroy(wick_cuda_model* m);
 
@@ -300,8 +315,8 @@ int32_t wick_cuda_attention_decode_splitk(const float* q_dev, const float* k_cac
  * a CUDA event after each group of kernels of one kind and adds the differences to a running total per category
  * (milliseconds since the last enable).  wick_cuda_profile_category_name(i), i < WICK_CUDA_PROFILE_CATEGORIES, names them:
  * embedding, rmsnorm+quantise, gemm, short-conv, qk-norm+rope+kv-append, attention, activation+quantise,
- * output-norm+logits.  (The persistent decode kernel has its own per-phase timeline: wick_cuda_decode_profile.) */
-#define WICK_CUDA_PROFILE_CATEGORIES 8
+ * output-norm+logits, recurrence.  (The persistent decode kernel has its own per-phase timeline: wick_cuda_decode_profile.) */
+#define WICK_CUDA_PROFILE_CATEGORIES 9
 int32_t wick_cuda_profile_enable(wick_cuda_model* m, int32_t on);
 int32_t wick_cuda_profile_read(wick_cuda_model* m, double* ms_out, uint32_t capacity);
 const char* wick_cuda_profile_category_name(uint32_t i);
@@ -341,6 +356,10 @@ int32_t wick_cuda_seq_destroy(wick_cuda_model* m, uint32_t seq_id);
 int32_t wick_cuda_seq_length(const wick_cuda_model* m, uint32_t seq_id, uint32_t* out);
 int32_t wick_cuda_seq_prefill(wick_cuda_model* m, uint32_t seq_id, const uint32_t* tokens_host, uint32_t n,
                               uint32_t start_pos, float* logits_host);
+/* wick_cuda_seq_prefill with logits at chosen places: want_host lists n_want places among the n tokens (any order, possibly
+ * none); logits_host gets [n_want][vocab_size] in that order. */
+int32_t wick_cuda_seq_prefill_logits(wick_cuda_model* m, uint32_t seq_id, const uint32_t* tokens_host, uint32_t n,
+                                     uint32_t start_pos, const uint32_t* want_host, uint32_t n_want, float* logits_host);
 int32_t wick_cuda_decode_batch(wick_cuda_model* m, const uint32_t* tokens_host, const uint32_t* seq_ids_host,
                                uint32_t bs, uint32_t* next_tokens_host);
 int32_t wick_cuda_decode_batch_steps(wick_cuda_model* m, const uint32_t* first_tokens_host,

@@ -13,10 +13,10 @@ _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "libwick_cuda.so")
 
 OK = 0
-ERR_BAD_ARG, ERR_CUDA, ERR_OOM, ERR_UNSUPPORTED_DTYPE, ERR_CONTEXT_FULL, ERR_TIMEOUT, ERR_BAD_GGUF = -1, -2, -3, -4, -5, -6, -7
+ERR_BAD_ARG, ERR_CUDA, ERR_OOM, ERR_UNSUPPORTED_DTYPE, ERR_CONTEXT_FULL, ERR_TIMEOUT, ERR_BAD_GGUF, ERR_BAD_MODEL = -1, -2, -3, -4, -5, -6, -7, -8
 ERR_NAMES = {
     ERR_BAD_ARG: "BAD_ARG", ERR_CUDA: "CUDA", ERR_OOM: "OOM", ERR_UNSUPPORTED_DTYPE: "UNSUPPORTED_DTYPE",
-    ERR_CONTEXT_FULL: "CONTEXT_FULL", ERR_TIMEOUT: "TIMEOUT", ERR_BAD_GGUF: "BAD_GGUF",
+    ERR_CONTEXT_FULL: "CONTEXT_FULL", ERR_TIMEOUT: "TIMEOUT", ERR_BAD_GGUF: "BAD_GGUF", ERR_BAD_MODEL: "BAD_MODEL",
 }
 
 
@@ -42,6 +42,7 @@ SIGNATURES = {
     "wick_cuda_device_count": [C.POINTER(_i32)],
     "wick_cuda_model_create": [_vp, C.c_size_t, _u32, _i32, C.POINTER(_vp)],
     "wick_cuda_model_create_from_file": [C.c_char_p, _u32, _i32, C.POINTER(_vp)],
+    "wick_cuda_model_create_from_path": [C.c_char_p, _u32, _i32, _i32, C.POINTER(_vp)],
     "wick_cuda_model_config": [_vp, C.POINTER(Config)],
     "wick_cuda_model_kv_heads_per_layer": [_vp, _vp, _u32],
     "wick_cuda_gpu_memory_bytes": [_vp, C.POINTER(_u64)],
@@ -79,6 +80,7 @@ SIGNATURES = {
     "wick_cuda_seq_destroy": [_vp, _u32],
     "wick_cuda_seq_length": [_vp, _u32, C.POINTER(_u32)],
     "wick_cuda_seq_prefill": [_vp, _u32, _vp, _u32, _u32, _vp],
+    "wick_cuda_seq_prefill_logits": [_vp, _u32, _vp, _u32, _u32, _vp, _u32, _vp],
     "wick_cuda_decode_batch": [_vp, _vp, _vp, _u32, _vp],
     "wick_cuda_decode_batch_steps": [_vp, _vp, _vp, _u32, _u32, _vp],
     "wick_cuda_decode_batch_logits": [_vp, _vp, _vp, _u32, _vp],
@@ -108,7 +110,8 @@ SIGNATURES = {
 }
 VOID_FUNCS = {"wick_cuda_model_destroy": [_vp], "wick_cuda_weight_destroy": [_vp], "wick_cuda_tp_comm_destroy": [_vp]}
 ALL_SYMBOLS = sorted(list(SIGNATURES) + list(VOID_FUNCS) + ["wick_cuda_last_error", "wick_cuda_argmax_noalloc_last_error",
-                                                            "wick_cuda_tp_last_error", "wick_cuda_profile_category_name"])
+                                                            "wick_cuda_tp_last_error", "wick_cuda_profile_category_name",
+                                                            "wick_cuda_model_architecture", "wick_cuda_model_layer_type"])
 
 _lib = None
 
@@ -138,6 +141,10 @@ def load() -> C.CDLL:
     lib.wick_cuda_tp_last_error.restype = C.c_char_p
     lib.wick_cuda_profile_category_name.argtypes = [_u32]
     lib.wick_cuda_profile_category_name.restype = C.c_char_p
+    lib.wick_cuda_model_architecture.argtypes = [_vp]
+    lib.wick_cuda_model_architecture.restype = C.c_char_p
+    lib.wick_cuda_model_layer_type.argtypes = [_vp, _u32]
+    lib.wick_cuda_model_layer_type.restype = C.c_char_p
     _lib = lib
     return lib
 

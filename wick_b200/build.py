@@ -6,6 +6,7 @@ explicitly where the reference uses a fused NEON instruction.
 """
 from __future__ import annotations
 
+import fcntl
 import os
 import shutil
 import subprocess
@@ -15,7 +16,8 @@ from typing import List
 _HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(_HERE, "csrc")
 LIB_PATH = os.path.join(_HERE, "libwick_cuda.so")
-SOURCES = ["kernels_basic.cu", "kernels_gemv.cu", "kernels_attn.cu", "kernels_q6k.cu", "kernels_batch.cu", "kernels_sample.cu", "tp_comm.cu", "decode_mega.cu", "gemm_tc.cu", "argmax_noalloc.cu", "wick_cuda.cu"]
+SOURCES = ["kernels_basic.cu", "kernels_gemv.cu", "kernels_attn.cu", "kernels_q6k.cu", "kernels_batch.cu", "kernels_sample.cu", "tp_comm.cu", "decode_mega.cu", "gemm_tc.cu", "argmax_noalloc.cu",
+           "kernels_hyper.cu", "kernels_dense.cu", "kernels_mixattn.cu", "kernels_delta.cu", "hybrid.cu", "wick_cuda.cu"]
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
@@ -31,22 +33,30 @@ def _nvcc() -> str:
     raise RuntimeError("nvcc not found")
 
 
-def _stale() -> bool:
-    if not os.path.exists(LIB_PATH):
-        return True
-    t = os.path.getmtime(LIB_PATH)
-    for f in os.listdir(CSRC):
-        if os.path.getmtime(os.path.join(CSRC, f)) > t:
-            return True
-    inc = os.path.join(_HERE, "..", "include", "wick_cuda.h")
-    return os.path.getmtime(inc) > t or os.path.getmtime(__file__) > t
+def _inputs() -> tuple[dict, float]:
+    """Modification time of every source, and the newest of what all of them may include (headers, this file)."""
+    srcs = {f: os.path.getmtime(os.path.join(CSRC, f)) for f in SOURCES}
+    shared = [os.path.join(CSRC, f) for f in os.listdir(CSRC) if not f.endswith(".cu")]
+    shared += [os.path.join(_HERE, "..", "include", "wick_cuda.h"), __file__]
+    return srcs, max(os.path.getmtime(f) for f in shared)
 
 
 def build(force: bool = False, verbose: bool = False, extra: List[str] | None = None) -> str:
-    if not force and not _stale():
+    """Compiles what is out of date and links; safe to call from several processes at once."""
+    srcs, shared = _inputs()
+    newest = max(shared, *srcs.values())
+    if not force and os.path.exists(LIB_PATH) and os.path.getmtime(LIB_PATH) >= newest:
         return LIB_PATH
     objdir = os.path.join(_HERE, "build")
     os.makedirs(objdir, exist_ok=True)
+    with open(os.path.join(objdir, ".lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        if not force and os.path.exists(LIB_PATH) and os.path.getmtime(LIB_PATH) >= newest:
+            return LIB_PATH  # another process has just done it
+        return _compile(objdir, srcs, shared, force or bool(extra), verbose, extra or [])
+
+
+def _compile(objdir: str, srcs: dict, shared: float, force: bool, verbose: bool, extra: List[str]) -> str:
     nvcc = _nvcc()
     env = dict(os.environ)
     # the environment may export CC/CXX pointing at a non-system compiler; nvcc wants the system g++
@@ -55,19 +65,29 @@ def build(force: bool = False, verbose: bool = False, extra: List[str] | None = 
     procs = []
     for src in SOURCES:
         obj = os.path.join(objdir, src.replace(".cu", ".o"))
-        cmd = [nvcc, "-ccbin", ccbin, *NVCC_FLAGS, *(extra or []), "-c", os.path.join(CSRC, src), "-o", obj]
+        objs.append(obj)
+        if not force and os.path.exists(obj) and os.path.getmtime(obj) >= max(shared, srcs[src]):
+            continue
+        part = f"{obj}.{os.getpid()}.part.o"
+        cmd = [nvcc, "-ccbin", ccbin, *NVCC_FLAGS, *extra, "-c", os.path.join(CSRC, src), "-o", part]
         if verbose:
             cmd.insert(1, "-Xptxas=-v")
-        procs.append((cmd, subprocess.Popen(cmd, env=env, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)))
-        objs.append(obj)
-    for cmd, p in procs:
+        procs.append((cmd, part, obj, subprocess.Popen(cmd, env=env, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)))
+    failed = None
+    for cmd, part, obj, p in procs:
         out, _ = p.communicate()
         if verbose or p.returncode:
             sys.stderr.write(out)
         if p.returncode:
-            raise RuntimeError("nvcc failed: " + " ".join(cmd))
-    link = [nvcc, "-ccbin", ccbin, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-o", LIB_PATH, *objs]
+            failed = failed or cmd
+        else:
+            os.replace(part, obj)
+    if failed:
+        raise RuntimeError("nvcc failed: " + " ".join(failed))
+    part = f"{LIB_PATH}.{os.getpid()}.part"
+    link = [nvcc, "-ccbin", ccbin, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-o", part, *objs]
     subprocess.check_call(link, env=env)
+    os.replace(part, LIB_PATH)
     return LIB_PATH
 
 

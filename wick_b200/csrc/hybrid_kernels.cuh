@@ -1,0 +1,187 @@
+// Launch wrappers of the kernels behind models that are described by a config.json layer list (hybrid.cu): dense bfloat16
+// matrices, hyper-connection streams, windowed attention with blended sigmoid scores, and the channel-decay delta rule.
+// Sizes and constants are arguments, so that another design can use the same kernels.
+//
+// Activations are token-major.  "act" buffers hold the model's activation type: bfloat16, or f32 for a model created with
+// WICK_CUDA_COMPUTE_F32; `bf16` says which.  Row pitches of act buffers are multiples of 8 elements and their padding
+// stays zero.
+#pragma once
+#include <cuda.h>
+#include <cuda_bf16.h>
+
+#include <algorithm>
+
+#include "kernels.cuh"
+
+namespace wick {
+
+__host__ __device__ constexpr int round_up(int v, int to) { return (v + to - 1) / to * to; }
+
+// ── dense matrices ─────────────────────────────────────────────────────────
+// [m][ld] bfloat16, ld = k rounded up to 8, padding zero, base 16-byte aligned.  The weights of the file are bfloat16, so
+// this is exact in both activation types.
+struct DenseWeight {
+    const __nv_bfloat16* w = nullptr;
+    int m = 0, k = 0, ld = 0;
+};
+enum Activation { ACT_RELU = 0, ACT_SILU = 1 };
+struct DenseJob {
+    DenseWeight w;
+    const void* x = nullptr;  // act [n][ldx]
+    int ldx = 0;
+    void* y = nullptr;        // act or f32 [n][ldy]
+    int ldy = 0;
+};
+// y = x W^T for n rows.  Up to two independent jobs share a launch; or (gated) the two jobs are gate and up matrices of the
+// same shape and input and job[0].y = activation(gate x) * (up x).
+struct DenseCall {
+    DenseJob job[2];
+    int count = 1, n = 0;
+    bool out_f32 = false;   // y is f32 whatever the activation type
+    bool gated = false;
+    Activation act = ACT_RELU;
+    float softcap = 0.0f;   // > 0: y = softcap * tanh(y / softcap)
+    uint32_t* err = nullptr;  // device word for expired waits of the tensor-core kernel
+};
+// Chooses between the row-streaming kernel (few rows), the tcgen05 kernel (bfloat16) and the f32 kernel.
+cudaError_t launch_dense(cudaStream_t st, bool bf16, const DenseCall& call);
+// The individual kernels (launch_dense picks one).
+void launch_dense_rows(cudaStream_t st, bool bf16, const DenseCall& call);    // n <= DENSE_ROWS_MAX
+void launch_dense_simt(cudaStream_t st, bool bf16, const DenseCall& call);    // any n
+cudaError_t launch_dense_tc(cudaStream_t st, const DenseCall& call);          // bfloat16, tcgen05
+constexpr int DENSE_ROWS_MAX = 8;
+
+// ── where the rows of a launch live ────────────────────────────────────────
+// Either n consecutive tokens of one sequence (positions == NULL: row j is at start_pos + j, state s0 / s1), or one token of
+// each of n sequences (positions[j], and p0[j] / p1[j] unless there is a single row with state s0 / s1).
+struct RowState {
+    void* const* p0 = nullptr;
+    void* const* p1 = nullptr;
+    void *s0 = nullptr, *s1 = nullptr;
+    const uint32_t* positions = nullptr;
+    int start_pos = 0;
+    __device__ void* st0(int j) const { return p0 ? p0[j] : s0; }
+    __device__ void* st1(int j) const { return p1 ? p1[j] : s1; }
+    __device__ int pos(int j) const { return positions ? (int)positions[j] : start_pos + j; }
+    bool separate() const { return positions != nullptr; }
+};
+
+// ── hyper-connections + RMS norm with a scalar gain ────────────────────────
+// x [n][S][W] f32 streams.  One launch applies the previous sublayer's write (if any), reads the next sublayer's input and
+// normalises it:
+//   x_t <- sum_s mix[s][t] x_s + out[t] y        (y != NULL)
+//   h   =  g * u / sqrt(mean(u^2) + eps),  u = sum_s in[s] x_s   (in == NULL: plain sum)
+struct HyperArgs {
+    // first launch of a step: the streams all equal scale * embed[token] (tokens) or the given frame (frames); x is written
+    const uint32_t* tokens = nullptr;
+    const DecodeCtl* ctl = nullptr;       // the single token of a decode step, when tokens == NULL
+    const __nv_bfloat16* embed = nullptr;
+    int ld_embed = 0;
+    float embed_scale = 1.0f;
+    const float* frames = nullptr;        // [n][W]
+    float* x = nullptr;
+    bool store_x = true;
+    const float* y = nullptr;             // [n][ldy] f32 output of the previous sublayer
+    int ldy = 0;
+    const float *mix = nullptr, *out = nullptr;  // of the previous sublayer: [S][S], [S]
+    const float* in = nullptr;            // of the next sublayer: [S]
+    const float* gain = nullptr;          // [1]
+    float eps = 0.0f;
+    const int* rows = nullptr;            // if set, output row i comes from row rows[i] of x and y (x is then not written)
+    void* h = nullptr;                    // act [n][ldh]
+    int ldh = 0;
+    float* normed = nullptr;              // optional f32 copy of the last row's h [W]
+    int n = 0, S = 1, W = 0;
+};
+constexpr int HYPER_MAX_STREAMS = 16;
+void launch_hyper_norm(cudaStream_t st, bool bf16, const HyperArgs& a);
+
+// ── windowed attention with blended sigmoid scores ─────────────────────────
+struct MixAttnShape {
+    int heads = 0, kv_heads = 0, dim = 0, vdim = 0;
+    int size = 0;        // sliding window (0: none): key j is seen by i when i - j < size
+    int keep_first = 0;  // ... or j < keep_first
+    float scale = 1.0f, eps = 0.0f;
+    const float* talk = nullptr;  // [H][H] or NULL
+    const float* bias = nullptr;  // [H] added to the blended score, or NULL
+    int seen(int max_seq) const { return size > 0 && size + keep_first < max_seq ? size + keep_first : max_seq; }
+};
+// Splits qkv [n][ld] (heads*dim q, kv_heads*dim k, kv_heads*vdim v): q and k divided by their root mean square per head, q
+// back in place, k and v rows appended to the caches (act [pos][kv_heads*dim], [pos][kv_heads*vdim]).
+void launch_qk_rms_append(cudaStream_t st, bool bf16, void* qkv, int ld, int n, const MixAttnShape& s, const RowState& rs);
+// out act [n][ldo] (heads*vdim).  partial: mix_attn_partial_floats() floats.
+size_t mix_attn_partial_floats(const MixAttnShape& s, int max_rows);
+bool mix_attn_supported(const MixAttnShape& s);
+cudaError_t launch_mix_attn(cudaStream_t st, bool bf16, const void* q, int ldq, int n, const MixAttnShape& s, const RowState& rs, void* out,
+                            int ldo, float* partial, int max_seq);
+
+// ── channel-decay delta rule ───────────────────────────────────────────────
+struct DeltaShape {
+    int heads = 0, kv_heads = 0, dim = 0, vdim = 0, taps = 1;
+    float eps = 0.0f;
+    __host__ __device__ int dimp() const { return round_up(dim, 32); }            // key channels per head in f32 work rows and in the state
+    __host__ __device__ int channels() const { return 2 * kv_heads * dim + heads * vdim; }
+    size_t state_floats() const { return (size_t)heads * vdim * dimp(); }   // [H][vdim][dimp]
+    size_t conv_floats() const { return (size_t)(taps - 1) * channels(); }  // [taps - 1][channels]
+};
+constexpr int DELTA_MAX_DIM = 256, DELTA_MAX_TAPS = 16;
+// f32 work rows of n tokens that the recurrence reads
+struct DeltaWork {
+    float *q = nullptr, *k = nullptr;  // [n][G][dimp] unit vectors, q times dim^-1/2
+    float* v = nullptr;                // [n][H*vdim]
+    float* g = nullptr;                // [n][H][dimp] decay factors
+    float* beta = nullptr;             // [n][H]
+    float* kq = nullptr;               // [n][G] k . q
+    float* o = nullptr;                // [n][H*vdim] read-outs
+};
+struct DeltaPrepArgs {
+    const void* p = nullptr;  // act [n][ldp]: the q | k | v channels at 0.., the beta logits at off_b
+    int ldp = 0, off_b = 0;
+    const float* a = nullptr;  // [n][lda] decay projection H*dim
+    int lda = 0;
+    const float *conv_w = nullptr, *A_log = nullptr, *dt_bias = nullptr;  // [channels][taps], [H], [H*dim]
+    int n = 0;
+};
+// Short convolution + silu, unit q and k, decays and step sizes; advances the convolution state (s1 / p1).
+void launch_delta_prep(cudaStream_t st, bool bf16, const DeltaPrepArgs& a, const DeltaShape& s, const RowState& rs, const DeltaWork& w);
+// The recurrence: n tokens of one sequence, or one token of each row; state in s0 / p0.
+void launch_delta_scan(cudaStream_t st, int n, const DeltaShape& s, const RowState& rs, const DeltaWork& w);
+// out act [n][ldo] = rms(o) * norm * sigmoid(gate), gate f32 [n][ldg]
+void launch_delta_out(cudaStream_t st, bool bf16, int n, const DeltaShape& s, const float* o, const float* norm, const float* gate, int ldg,
+                      void* out, int ldo);
+
+// ── shared device helpers ──────────────────────────────────────────────────
+__device__ __forceinline__ float act_f(float v) { return v; }
+__device__ __forceinline__ float act_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <class T>
+__device__ __forceinline__ T f_act(float v);
+template <>
+__device__ __forceinline__ float f_act<float>(float v) { return v; }
+template <>
+__device__ __forceinline__ __nv_bfloat16 f_act<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+
+// eight consecutive values from a 16-byte aligned address
+__device__ __forceinline__ void bf16x8_f(const uint4 u, float* f) {
+    const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        f[2 * i] = __uint_as_float(w[i] << 16);
+        f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+    }
+}
+__device__ __forceinline__ void load8(const __nv_bfloat16* p, float* f) { bf16x8_f(*reinterpret_cast<const uint4*>(p), f); }
+__device__ __forceinline__ void load8(const float* p, float* f) {
+    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+    f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float activate(float z, Activation a) { return a == ACT_RELU ? fmaxf(z, 0.0f) : silu_f(z); }
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+}
+
+}  // namespace wick

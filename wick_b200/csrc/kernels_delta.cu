@@ -1,0 +1,278 @@
+// The gated delta rule with one decay per head and key channel (f32 throughout, as the state is):
+//     S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+// k_delta_prep   short causal convolutions + silu, unit q and k, decays and step sizes: one warp per (token, group of
+//                channels that is normalised together).
+// k_delta_scan   the recurrence.  The columns of S (value channels) do not depend on each other: eight lanes hold one column,
+//                4 * R4 key channels each, in registers, from the first token of the launch to the last.  The read-out is
+//                folded into the same pass over the column, o = (diag(g) S)^T q + (k . q) u, so that a token costs one
+//                round of cross-lane sums; k . q comes from k_delta_prep.  A block of tokens' q, k, g rows is staged in shared
+//                memory with cp.async, one block ahead.
+// k_delta_out    RMS norm over the value channels of a head, gain, sigmoid gate.
+#include "hybrid_kernels.cuh"
+
+namespace wick {
+
+namespace {
+
+// ── preparation ────────────────────────────────────────────────────────────
+constexpr int PREP_WARPS = 8;
+constexpr int PREP_REG = DELTA_MAX_DIM / 32;
+
+// Convolution of channel ch at row j followed by silu; `advance`: also moves the row's own state on (rows are separate
+// sequences then, and this lane owns the channel).
+template <class T>
+__device__ __forceinline__ float conv_silu(const DeltaPrepArgs& a, const DeltaShape& s, float* state, int j, int ch, bool separate) {
+    const int t = s.taps, C = s.channels();
+    const float* w = a.conv_w + (size_t)ch * t;
+    const T* p = (const T*)a.p;
+    const float cur = act_f(p[(size_t)j * a.ldp + ch]);
+    float sum = 0.0f;
+    for (int i = 0; i < t - 1; i++) {
+        const int src = j - (t - 1 - i);  // row of the launch; negative: kept from before
+        float v;
+        if (separate) v = state[(size_t)i * C + ch];
+        else v = src >= 0 ? act_f(p[(size_t)src * a.ldp + ch]) : state[(size_t)(t - 1 + src) * C + ch];
+        sum = fmaf(w[i], v, sum);
+        if (separate && i > 0) state[(size_t)(i - 1) * C + ch] = v;
+    }
+    if (separate && t > 1) state[(size_t)(t - 2) * C + ch] = cur;
+    return silu_f(fmaf(w[t - 1], cur, sum));
+}
+
+template <class T>
+__global__ void __launch_bounds__(PREP_WARPS * 32) k_delta_prep(const __grid_constant__ DeltaPrepArgs a, const __grid_constant__ DeltaShape s,
+                                                               const __grid_constant__ RowState rs, bool separate, const __grid_constant__ DeltaWork w) {
+    const int lane = threadIdx.x & 31;
+    const int seg_n = s.kv_heads + 2 * s.heads;
+    const size_t unit = (size_t)blockIdx.x * PREP_WARPS + (threadIdx.x >> 5);
+    if (unit >= (size_t)a.n * seg_n) return;
+    const int j = (int)(unit / seg_n), seg = (int)(unit % seg_n);
+    float* state = (float*)rs.st1(separate ? j : 0);
+    const int G = s.kv_heads, H = s.heads, D = s.dim, E = s.vdim, DP = s.dimp();
+    if (seg < G) {  // q and k of key head `seg`
+        float q[PREP_REG], k[PREP_REG], qq = 0.0f, kk = 0.0f, kq = 0.0f;
+#pragma unroll
+        for (int r = 0; r < PREP_REG; r++) {
+            const int i = r * 32 + lane;
+            q[r] = k[r] = 0.0f;
+            if (i < D) {
+                q[r] = conv_silu<T>(a, s, state, j, seg * D + i, separate);
+                k[r] = conv_silu<T>(a, s, state, j, (G + seg) * D + i, separate);
+            }
+            qq = fmaf(q[r], q[r], qq);
+            kk = fmaf(k[r], k[r], kk);
+        }
+        const float qs = 1.0f / sqrtf((float)D) / sqrtf(warp_sum(qq) + 1e-6f), ks = 1.0f / sqrtf(warp_sum(kk) + 1e-6f);
+        float* qo = w.q + ((size_t)j * G + seg) * DP;
+        float* ko = w.k + ((size_t)j * G + seg) * DP;
+#pragma unroll
+        for (int r = 0; r < PREP_REG; r++) {
+            const int i = r * 32 + lane;
+            if (i < DP) {  // the padding channels are zero
+                qo[i] = q[r] *= qs;
+                ko[i] = k[r] *= ks;
+                kq = fmaf(q[r], k[r], kq);
+            }
+        }
+        kq = warp_sum(kq);
+        if (lane == 0) w.kq[(size_t)j * G + seg] = kq;
+    } else if (seg < G + H) {  // v of head h
+        const int h = seg - G;
+        for (int i = lane; i < E; i += 32) w.v[(size_t)j * H * E + h * E + i] = conv_silu<T>(a, s, state, j, 2 * G * D + h * E + i, separate);
+    } else {  // decays and step size of head h
+        const int h = seg - G - H;
+        const float rate = expf(a.A_log[h]);
+        float* go = w.g + ((size_t)j * H + h) * DP;
+        for (int i = lane; i < DP; i += 32) {
+            float g = 1.0f;
+            if (i < D) {
+                const float z = a.a[(size_t)j * a.lda + h * D + i] + a.dt_bias[h * D + i];
+                const float sp = fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z)));
+                g = expf(-rate * sp);
+            }
+            go[i] = g;
+        }
+        if (lane == 0) w.beta[(size_t)j * H + h] = sigmoid_f(act_f(((const T*)a.p)[(size_t)j * a.ldp + a.off_b + h]));
+    }
+}
+
+// The last taps - 1 inputs after n consecutive tokens of one sequence.  A channel's rows are moved in ascending order, so
+// that a kept row is read before it is overwritten.
+template <class T>
+__global__ void __launch_bounds__(256) k_delta_conv_state(const T* __restrict__ p, int ldp, int n, int channels, int taps, float* __restrict__ state) {
+    const int ch = blockIdx.x * 256 + threadIdx.x;
+    if (ch >= channels) return;
+    for (int r = 0; r < taps - 1; r++) {
+        const int src = n - (taps - 1) + r;
+        state[(size_t)r * channels + ch] = src >= 0 ? act_f(p[(size_t)src * ldp + ch]) : state[(size_t)(taps - 1 + src) * channels + ch];
+    }
+}
+
+// ── recurrence ─────────────────────────────────────────────────────────────
+constexpr int SCAN_THREADS = 128, SCAN_COLS = SCAN_THREADS / 8;  // value channels per CTA
+constexpr int SCAN_TB = 16;                                      // tokens staged at a time
+
+__device__ __forceinline__ void cp16(float* dst, const float* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp4(float* dst, const float* src) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+
+__host__ __device__ constexpr int scan_tok_floats(int dp) { return 3 * dp + SCAN_COLS + 4; }  // q k g rows, v, beta, kq (+ pad)
+
+// R4 * 4 key channels per lane: dimp = 32 * R4.  Lane l of a column's eight holds channels 32 r + 4 l .. + 3.
+template <int R4>
+__global__ void __launch_bounds__(SCAN_THREADS) k_delta_scan(int n, const __grid_constant__ DeltaShape s, const __grid_constant__ RowState rs,
+                                                            bool separate, const __grid_constant__ DeltaWork w) {
+    extern __shared__ __align__(16) float sm[];
+    constexpr int DP = 32 * R4, TOK = scan_tok_floats(DP);
+    const int tid = threadIdx.x, l8 = tid & 7, col = tid >> 3;
+    const int h = blockIdx.y, G = s.kv_heads, H = s.heads, E = s.vdim;
+    const int kh = h / (H / G), c0 = blockIdx.x * SCAN_COLS, c = c0 + col;
+    const int row0 = separate ? blockIdx.z : 0, nt = separate ? 1 : n;
+    float* state = (float*)rs.st0(row0) + ((size_t)h * E + min(c, E - 1)) * DP;
+    float S[R4][4];
+#pragma unroll
+    for (int r = 0; r < R4; r++) {
+        const float4 v = *reinterpret_cast<const float4*>(state + 32 * r + 4 * l8);
+        S[r][0] = v.x; S[r][1] = v.y; S[r][2] = v.z; S[r][3] = v.w;
+    }
+    auto stage = [&](int t0, int buf) {  // tokens t0 .. t0 + SCAN_TB - 1 (as many as there are) into buffer `buf`
+        const int cnt = min(SCAN_TB, nt - t0);
+        float* dst = sm + buf * SCAN_TB * TOK;
+        constexpr int V4 = DP / 4;
+        for (int i = tid; i < cnt * 3 * V4; i += SCAN_THREADS) {
+            const int t = i / (3 * V4), q = i % (3 * V4), which = q / V4, x = q % V4;
+            const size_t row = (size_t)(row0 + t0 + t);
+            const float* src = which == 0 ? w.q + (row * G + kh) * DP : which == 1 ? w.k + (row * G + kh) * DP : w.g + (row * H + h) * DP;
+            cp16(dst + t * TOK + which * DP + 4 * x, src + 4 * x);
+        }
+        for (int i = tid; i < cnt * (SCAN_COLS + 2); i += SCAN_THREADS) {
+            const int t = i / (SCAN_COLS + 2), x = i % (SCAN_COLS + 2);
+            const size_t row = (size_t)(row0 + t0 + t);
+            if (x < SCAN_COLS) {
+                if (c0 + x < E) cp4(dst + t * TOK + 3 * DP + x, w.v + row * H * E + h * E + c0 + x);
+            } else if (x == SCAN_COLS) {
+                cp4(dst + t * TOK + 3 * DP + x, w.beta + row * H + h);
+            } else {
+                cp4(dst + t * TOK + 3 * DP + x, w.kq + row * G + kh);
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    stage(0, 0);
+    int buf = 0;
+    for (int t0 = 0; t0 < nt; t0 += SCAN_TB, buf ^= 1) {
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();  // the block's rows are there, and everyone has left the other buffer
+        if (t0 + SCAN_TB < nt) stage(t0 + SCAN_TB, buf ^ 1);
+        const int cnt = min(SCAN_TB, nt - t0);
+        const float* tk = sm + buf * SCAN_TB * TOK;
+#pragma unroll 2
+        for (int t = 0; t < cnt; t++, tk += TOK) {
+            float r1[2] = {0.f, 0.f}, r2[2] = {0.f, 0.f};
+            float4 k4[R4];
+#pragma unroll
+            for (int r = 0; r < R4; r++) {
+                const float4 q = *reinterpret_cast<const float4*>(tk + 32 * r + 4 * l8);
+                k4[r] = *reinterpret_cast<const float4*>(tk + DP + 32 * r + 4 * l8);
+                const float4 g = *reinterpret_cast<const float4*>(tk + 2 * DP + 32 * r + 4 * l8);
+                S[r][0] *= g.x; S[r][1] *= g.y; S[r][2] *= g.z; S[r][3] *= g.w;
+                r1[0] = fmaf(S[r][0], k4[r].x, r1[0]); r1[1] = fmaf(S[r][1], k4[r].y, r1[1]);
+                r2[0] = fmaf(S[r][0], q.x, r2[0]);     r2[1] = fmaf(S[r][1], q.y, r2[1]);
+                r1[0] = fmaf(S[r][2], k4[r].z, r1[0]); r1[1] = fmaf(S[r][3], k4[r].w, r1[1]);
+                r2[0] = fmaf(S[r][2], q.z, r2[0]);     r2[1] = fmaf(S[r][3], q.w, r2[1]);
+            }
+            float a = r1[0] + r1[1], b = r2[0] + r2[1];
+#pragma unroll
+            for (int o = 4; o > 0; o >>= 1) {
+                a += __shfl_xor_sync(0xffffffffu, a, o);
+                b += __shfl_xor_sync(0xffffffffu, b, o);
+            }
+            const float u = tk[3 * DP + SCAN_COLS] * (tk[3 * DP + col] - a);
+            const float out = fmaf(tk[3 * DP + SCAN_COLS + 1], u, b);
+#pragma unroll
+            for (int r = 0; r < R4; r++) {
+                S[r][0] = fmaf(k4[r].x, u, S[r][0]);
+                S[r][1] = fmaf(k4[r].y, u, S[r][1]);
+                S[r][2] = fmaf(k4[r].z, u, S[r][2]);
+                S[r][3] = fmaf(k4[r].w, u, S[r][3]);
+            }
+            if (l8 == 0 && c < E) w.o[(size_t)(row0 + t0 + t) * H * E + h * E + c] = out;
+        }
+    }
+    if (c < E)
+#pragma unroll
+        for (int r = 0; r < R4; r++)
+            *reinterpret_cast<float4*>(state + 32 * r + 4 * l8) = make_float4(S[r][0], S[r][1], S[r][2], S[r][3]);
+}
+
+template <int R4>
+void scan_go(cudaStream_t st, int n, const DeltaShape& s, const RowState& rs, const DeltaWork& w) {
+    const bool sep = rs.separate();
+    const dim3 grid((s.vdim + SCAN_COLS - 1) / SCAN_COLS, s.heads, sep ? n : 1);
+    const size_t smem = (size_t)2 * SCAN_TB * scan_tok_floats(32 * R4) * 4;
+    if (smem > 48 * 1024) cudaFuncSetAttribute(k_delta_scan<R4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    k_delta_scan<R4><<<grid, SCAN_THREADS, smem, st>>>(n, s, rs, sep, w);
+}
+
+// ── output ─────────────────────────────────────────────────────────────────
+template <class T>
+__global__ void __launch_bounds__(256) k_delta_out(int n, int H, int E, float eps, const float* __restrict__ o, const float* __restrict__ norm,
+                                                   const float* __restrict__ gate, int ldg, T* __restrict__ out, int ldo) {
+    const int lane = threadIdx.x & 31;
+    const size_t unit = (size_t)blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (unit >= (size_t)n * H) return;
+    const int j = (int)(unit / H), h = (int)(unit % H);
+    const float* src = o + (size_t)j * H * E + h * E;
+    float ss = 0.0f;
+    for (int i = lane; i < E; i += 32) ss = fmaf(src[i], src[i], ss);
+    const float r = 1.0f / sqrtf(warp_sum(ss) / (float)E + eps);
+    for (int i = lane; i < E; i += 32)
+        out[(size_t)j * ldo + h * E + i] = f_act<T>(src[i] * r * norm[i] * sigmoid_f(gate[(size_t)j * ldg + h * E + i]));
+}
+
+}  // namespace
+
+void launch_delta_prep(cudaStream_t st, bool bf16, const DeltaPrepArgs& a, const DeltaShape& s, const RowState& rs, const DeltaWork& w) {
+    if (a.n <= 0) return;
+    const bool sep = rs.separate();
+    const size_t units = (size_t)a.n * (s.kv_heads + 2 * s.heads);
+    const unsigned grid = (unsigned)((units + PREP_WARPS - 1) / PREP_WARPS);
+    g_kernel_launches++;
+    if (bf16) k_delta_prep<__nv_bfloat16><<<grid, PREP_WARPS * 32, 0, st>>>(a, s, rs, sep, w);
+    else k_delta_prep<float><<<grid, PREP_WARPS * 32, 0, st>>>(a, s, rs, sep, w);
+    if (!sep && s.taps > 1) {
+        const int C = s.channels();
+        g_kernel_launches++;
+        if (bf16) k_delta_conv_state<__nv_bfloat16><<<(C + 255) / 256, 256, 0, st>>>((const __nv_bfloat16*)a.p, a.ldp, a.n, C, s.taps, (float*)rs.s1);
+        else k_delta_conv_state<float><<<(C + 255) / 256, 256, 0, st>>>((const float*)a.p, a.ldp, a.n, C, s.taps, (float*)rs.s1);
+    }
+}
+
+void launch_delta_scan(cudaStream_t st, int n, const DeltaShape& s, const RowState& rs, const DeltaWork& w) {
+    if (n <= 0) return;
+    g_kernel_launches++;
+    switch (s.dimp() / 32) {
+        case 1: return scan_go<1>(st, n, s, rs, w);
+        case 2: return scan_go<2>(st, n, s, rs, w);
+        case 3: return scan_go<3>(st, n, s, rs, w);
+        case 4: return scan_go<4>(st, n, s, rs, w);
+        case 5: return scan_go<5>(st, n, s, rs, w);
+        case 6: return scan_go<6>(st, n, s, rs, w);
+        case 7: return scan_go<7>(st, n, s, rs, w);
+        default: return scan_go<8>(st, n, s, rs, w);
+    }
+}
+
+void launch_delta_out(cudaStream_t st, bool bf16, int n, const DeltaShape& s, const float* o, const float* norm, const float* gate, int ldg,
+                      void* out, int ldo) {
+    if (n <= 0) return;
+    const unsigned grid = (unsigned)(((size_t)n * s.heads + 7) / 8);
+    g_kernel_launches++;
+    if (bf16) k_delta_out<__nv_bfloat16><<<grid, 256, 0, st>>>(n, s.heads, s.vdim, s.eps, o, norm, gate, ldg, (__nv_bfloat16*)out, ldo);
+    else k_delta_out<float><<<grid, 256, 0, st>>>(n, s.heads, s.vdim, s.eps, o, norm, gate, ldg, (float*)out, ldo);
+}
+
+}  // namespace wick

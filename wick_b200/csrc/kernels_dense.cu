@@ -1,0 +1,184 @@
+// Dense bfloat16 matrices times f32 or bfloat16 activation rows.
+//   k_dense_rows  up to DENSE_ROWS_MAX rows (decode): a warp streams R weight rows with 16-byte loads, every loaded weight
+//                 feeds all the activation rows.  HBM-bound: the weight bytes once.
+//   k_dense_simt  any number of rows, f32 multiply-adds on the CUDA cores: the f32 models' prompts, and shapes the tensor-core
+//                 kernel (gemm_bf16.cu) is not worth starting for.
+// Both accumulate in f32 and share the epilogues: plain store, activation(gate) * up, soft cap.
+#include "hybrid_kernels.cuh"
+
+namespace wick {
+
+namespace {
+
+template <class T, class O>
+__device__ __forceinline__ void dense_store(const DenseCall& c, const DenseJob& j, int row, int col, float v, float up) {
+    if (c.gated) v = activate(v, c.act) * up;
+    if (c.softcap > 0.0f) v = c.softcap * tanhf(v / c.softcap);
+    ((O*)j.y)[(size_t)row * j.ldy + col] = f_act<O>(v);
+}
+
+constexpr int ROWS_WARPS = 4;
+
+// NB activation rows, R weight rows (of each matrix when gated) per warp.
+template <class T, class O, int NB, int R, bool GATED>
+__global__ void __launch_bounds__(ROWS_WARPS * 32) k_dense_rows(const __grid_constant__ DenseCall c) {
+    constexpr int M = GATED ? 2 : 1;
+    const int lane = threadIdx.x & 31;
+    int unit = blockIdx.x * ROWS_WARPS + (threadIdx.x >> 5);
+    int ji = 0;
+    if (!GATED && c.count == 2) {
+        const int units0 = (c.job[0].w.m + R - 1) / R;
+        if (unit >= units0) {
+            ji = 1;
+            unit -= units0;
+        }
+    }
+    const DenseJob& j = c.job[ji];
+    const int m = j.w.m, ld = j.w.ld, row0 = unit * R;
+    if (row0 >= m) return;
+    const __nv_bfloat16* wp[M][R];
+#pragma unroll
+    for (int q = 0; q < M; q++)
+#pragma unroll
+        for (int r = 0; r < R; r++)  // a row past the end repeats the last one and is not stored
+            wp[q][r] = c.job[ji + q].w.w + (size_t)min(row0 + r, m - 1) * ld;
+    float acc[M][R][NB];
+#pragma unroll
+    for (int q = 0; q < M; q++)
+#pragma unroll
+        for (int r = 0; r < R; r++)
+#pragma unroll
+            for (int b = 0; b < NB; b++) acc[q][r][b] = 0.0f;
+    const T* x = (const T*)j.x;
+#pragma unroll 4
+    for (int k = lane * 8; k < ld; k += 256) {
+        uint4 wv[M][R];
+#pragma unroll
+        for (int q = 0; q < M; q++)
+#pragma unroll
+            for (int r = 0; r < R; r++) wv[q][r] = __ldg(reinterpret_cast<const uint4*>(wp[q][r] + k));
+#pragma unroll
+        for (int b = 0; b < NB; b++) {
+            float xv[8];
+            load8(x + (size_t)min(b, c.n - 1) * j.ldx + k, xv);
+#pragma unroll
+            for (int q = 0; q < M; q++)
+#pragma unroll
+                for (int r = 0; r < R; r++) {
+                    float w[8];
+                    bf16x8_f(wv[q][r], w);
+#pragma unroll
+                    for (int i = 0; i < 8; i++) acc[q][r][b] = fmaf(w[i], xv[i], acc[q][r][b]);
+                }
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < R; r++)
+#pragma unroll
+        for (int b = 0; b < NB; b++) {
+            const float v = warp_sum(acc[0][r][b]);
+            const float u = GATED ? warp_sum(acc[M - 1][r][b]) : 0.0f;
+            if (lane == 0 && row0 + r < m && b < c.n) dense_store<T, O>(c, j, b, row0 + r, v, u);
+        }
+}
+
+template <class T, class O, int NB, int R>
+void dense_rows_go(cudaStream_t st, const DenseCall& c) {
+    int units = (c.job[0].w.m + R - 1) / R;
+    if (!c.gated && c.count == 2) units += (c.job[1].w.m + R - 1) / R;
+    const unsigned grid = (unsigned)((units + ROWS_WARPS - 1) / ROWS_WARPS);
+    if (c.gated) k_dense_rows<T, O, NB, (R > 1 ? R / 2 : 1), true><<<(unsigned)(((c.job[0].w.m + (R > 1 ? R / 2 : 1) - 1) / (R > 1 ? R / 2 : 1) + ROWS_WARPS - 1) / ROWS_WARPS), ROWS_WARPS * 32, 0, st>>>(c);
+    else k_dense_rows<T, O, NB, R, false><<<grid, ROWS_WARPS * 32, 0, st>>>(c);
+}
+
+template <class T, class O>
+void dense_rows_n(cudaStream_t st, const DenseCall& c) {
+    if (c.n == 1) dense_rows_go<T, O, 1, 2>(st, c);
+    else if (c.n == 2) dense_rows_go<T, O, 2, 2>(st, c);
+    else if (c.n <= 4) dense_rows_go<T, O, 4, 2>(st, c);
+    else dense_rows_go<T, O, 8, 2>(st, c);
+}
+
+// ── f32 tile kernel ────────────────────────────────────────────────────────
+constexpr int ST = 64, SK = 16;  // 64 x 64 outputs per CTA, 16 columns of k per step; 256 threads, 4 x 4 outputs each
+
+template <class T, class O, bool GATED>
+__global__ void __launch_bounds__(256) k_dense_simt(const __grid_constant__ DenseCall c) {
+    constexpr int M = GATED ? 2 : 1;
+    __shared__ float xs[SK][ST + 4], ws[M][SK][ST + 4];
+    const DenseJob& j = c.job[GATED ? 0 : blockIdx.z];
+    const int m0 = blockIdx.x * ST, n0 = blockIdx.y * ST;
+    if (m0 >= j.w.m) return;
+    const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+    float acc[M][4][4] = {};
+    const int lr = tid >> 2, lk = (tid & 3) * 4;  // the element this thread stages: row lr, four k from lk
+    const bool x_ok = n0 + lr < c.n, w_ok = m0 + lr < j.w.m;
+    const T* xp = (const T*)j.x + (size_t)(x_ok ? n0 + lr : 0) * j.ldx;
+    for (int k0 = 0; k0 < j.w.k; k0 += SK) {
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            const int k = k0 + lk + i;
+            xs[lk + i][lr] = x_ok && k < j.w.k ? act_f(xp[k]) : 0.0f;
+#pragma unroll
+            for (int q = 0; q < M; q++)
+                ws[q][lk + i][lr] = w_ok && k < j.w.k ? __bfloat162float(c.job[GATED ? q : blockIdx.z].w.w[(size_t)(m0 + lr) * j.w.ld + k]) : 0.0f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < SK; k++) {
+            const float4 xv = *reinterpret_cast<const float4*>(&xs[k][ty * 4]);
+            const float xa[4] = {xv.x, xv.y, xv.z, xv.w};
+#pragma unroll
+            for (int q = 0; q < M; q++) {
+                const float4 wv = *reinterpret_cast<const float4*>(&ws[q][k][tx * 4]);
+                const float wa[4] = {wv.x, wv.y, wv.z, wv.w};
+#pragma unroll
+                for (int a = 0; a < 4; a++)
+#pragma unroll
+                    for (int b = 0; b < 4; b++) acc[q][a][b] = fmaf(xa[a], wa[b], acc[q][a][b]);
+            }
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int a = 0; a < 4; a++)
+#pragma unroll
+        for (int b = 0; b < 4; b++) {
+            const int row = n0 + ty * 4 + a, col = m0 + tx * 4 + b;
+            if (row < c.n && col < j.w.m) dense_store<T, O>(c, j, row, col, acc[0][a][b], acc[M - 1][a][b]);
+        }
+}
+
+template <class T, class O>
+void dense_simt_go(cudaStream_t st, const DenseCall& c) {
+    const int m = c.gated || c.count == 1 ? c.job[0].w.m : max(c.job[0].w.m, c.job[1].w.m);
+    const dim3 grid((m + ST - 1) / ST, (c.n + ST - 1) / ST, c.gated ? 1 : c.count);
+    if (c.gated) k_dense_simt<T, O, true><<<grid, 256, 0, st>>>(c);
+    else k_dense_simt<T, O, false><<<grid, 256, 0, st>>>(c);
+}
+
+}  // namespace
+
+void launch_dense_rows(cudaStream_t st, bool bf16, const DenseCall& c) {
+    if (c.n <= 0) return;
+    g_kernel_launches++;
+    if (!bf16) dense_rows_n<float, float>(st, c);
+    else if (c.out_f32) dense_rows_n<__nv_bfloat16, float>(st, c);
+    else dense_rows_n<__nv_bfloat16, __nv_bfloat16>(st, c);
+}
+
+void launch_dense_simt(cudaStream_t st, bool bf16, const DenseCall& c) {
+    if (c.n <= 0) return;
+    g_kernel_launches++;
+    if (!bf16) dense_simt_go<float, float>(st, c);
+    else if (c.out_f32) dense_simt_go<__nv_bfloat16, float>(st, c);
+    else dense_simt_go<__nv_bfloat16, __nv_bfloat16>(st, c);
+}
+
+cudaError_t launch_dense(cudaStream_t st, bool bf16, const DenseCall& c) {
+    if (c.n <= DENSE_ROWS_MAX) launch_dense_rows(st, bf16, c);
+    else launch_dense_simt(st, bf16, c);
+    return cudaGetLastError();
+}
+
+}  // namespace wick

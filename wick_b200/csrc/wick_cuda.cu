@@ -14,48 +14,21 @@
 #include <string>
 #include <vector>
 
-#include "../../include/wick_cuda.h"
 #include "gguf.hpp"
-#include "decode_mega.cuh"
-#include "gemm_tc.cuh"
-#include "kernels.cuh"
+#include "hybrid.cuh"
+#include "model_internal.cuh"
+
+#include <sys/stat.h>
 
 using namespace wick;
 
 // ── errors ─────────────────────────────────────────────────────────────────
 static thread_local std::string g_last_error;
 
-static int32_t fail(int32_t code, const std::string& msg) {
+int32_t wick::fail(int32_t code, const std::string& msg) {
     g_last_error = msg;
     return code;
 }
-#define CU_TRY(expr)                                                                              \
-    do {                                                                                          \
-        cudaError_t e__ = (expr);                                                                 \
-        if (e__ != cudaSuccess)                                                                   \
-            return fail(e__ == cudaErrorMemoryAllocation ? WICK_CUDA_ERR_OOM : WICK_CUDA_ERR_CUDA, \
-                        std::string(#expr) + ": " + cudaGetErrorString(e__));                     \
-    } while (0)
-#define W_TRY(expr)                  \
-    do {                             \
-        int32_t r__ = (expr);        \
-        if (r__ != WICK_CUDA_OK) return r__; \
-    } while (0)
-
-namespace {
-
-struct Layer {
-    bool is_attn = false;
-    int n_kv = 0;
-    float *attn_norm = nullptr, *ffn_norm = nullptr, *q_norm = nullptr, *k_norm = nullptr, *conv_w = nullptr;
-    DevWeight in_proj, out_proj, q, k, v, o, gate, up, down;
-    // int8 copies for the tensor-core prefill GEMM (gemm_tc.cu); q == nullptr when unavailable
-    TcWeight tc_in_proj, tc_out_proj, tc_q, tc_k, tc_v, tc_o, tc_gate, tc_up, tc_down;
-    float *k_cache = nullptr, *v_cache = nullptr;  // [max_seq][kv_dim]
-    float* conv_state = nullptr;                   // [d_conv][hidden]
-};
-
-}  // namespace
 
 struct wick_cuda_weight {
     DevWeight w;
@@ -64,123 +37,25 @@ struct wick_cuda_weight {
     uint32_t* tc_err = nullptr;
 };
 
-struct wick_cuda_model {
-    int device = 0;
-    cudaStream_t stream = nullptr;
-    wick_cuda_config cfg{};
-    int head_dim = 0;
-    std::vector<Layer> layers;
-    DevWeight embd;
-    TcWeight tc_embd;       // tensor-core copy of the vocabulary matrix, made for the multi-sequence step only
-    bool embd_q6k = false;  // token_embd is Q6_K: embd6 is used for the embedding rows and the logits, embd is empty
-    DevQ6K embd6;
-    float* output_norm = nullptr;
-    float *rope_cos = nullptr, *rope_sin = nullptr;
-    int max_chunk = 0;  // tokens of scratch
-    // tensor-core prefill GEMMs: available when every matrix meets tc_gemm_supported(); prefill_mode
-    // picks the bit-exact one (default), the fused-chain one, or the bit-exact CUDA-core kernel
-    bool tc_ok = false;     // the model's shapes allow the tensor-core GEMM
-    bool tc_built = false;  // its int8 weight copies and buffers exist (made by the first call that needs them)
-    int prefill_mode = WICK_CUDA_PREFILL_EXACT;
-    CUtensorMap map_x_hs[2], map_x_is[2];  // activations [max_chunk][hs | is], box of 64 / 128 rows
-    int8_t* q8m = nullptr;                  // lane-group-masked activations [4 * max_chunk][hs | is] (exact tensor-core GEMM)
-    CUtensorMap map_xm_hs, map_xm_is, map_xm_hs32, map_xm_is32;  // boxes of 64 rows (16 tokens) and of 32 rows (8 tokens)
-    float* normed_last = nullptr;  // output-normed hidden row of the last prefilled token
-    float* rope_delta = nullptr;   // [head_dim]: cos then sin of the n_keep shift rotation
-    uint32_t* tc_err = nullptr;
-    // scratch, token-major
-    float *hidden = nullptr, *block_out = nullptr, *ffn_out = nullptr, *proj = nullptr, *qbuf = nullptr, *kbuf = nullptr,
-          *vbuf = nullptr, *attn_out = nullptr, *gate = nullptr, *up = nullptr, *logits = nullptr;
-    float* q8s = nullptr;
-    int8_t* q8q = nullptr;
-    uint32_t* tokens_dev = nullptr;
-    DecodeCtl* ctl = nullptr;
-    uint32_t* argmax_tok = nullptr;
-    uint32_t* ring = nullptr;
-    int ring_len = 0;
-    // pinned host staging
-    uint32_t* h_u32 = nullptr;   // [ring_len] tokens in / out
-    float* h_logits = nullptr;   // [vocab]
-    cudaGraphExec_t g_logits = nullptr, g_greedy = nullptr;
-    uint64_t nodes_logits = 0, nodes_greedy = 0;  // kernels per graph replay
-    uint64_t launches = 0;                        // kernels launched so far
-    cudaEvent_t ev0 = nullptr, ev1 = nullptr;     // bracket the GPU work of the last call
-    // persistent decode kernel (decode_mega.cu); falls back to the captured graphs when the
-    // model does not meet its layout requirements or WICK_CUDA_DECODE=graph is set
-    bool mega_ok = false;
-    int mega_ctas = 0;
-    MegaParams mega{};
-    MegaPhase* d_phases = nullptr;
-    MegaPhase* d_phases_long = nullptr;  // the same list with an MPH_SCORES phase before every MPH_ATTN (long contexts)
-    int n_phases_long = 0;
-    float* scores_g = nullptr;
-    bool last_launch_long = false, long_ok = false;
-    MegaLayer* d_mlayers = nullptr;
-    unsigned long long* d_sync = nullptr;  // [0] barrier counter, [1..2] argmax accumulators
-    unsigned long long* hidden_flagged = nullptr;  // [hs] flagged copy of the hidden row (persistent decode kernel)
-    unsigned long long* d_prof = nullptr;  // [n_phases][4] timestamps of the last step
-    unsigned long long bar_base = 0;
-    DecodeCtl* h_ctl = nullptr;            // pinned copy of the control block
-    uint32_t seq_len = 0;
-    uint64_t bytes = 0;
-    std::vector<void*> allocs;
-    // extra sequence slots for wick_cuda_decode_batch (the model's own sequence is not one of them)
-    struct SeqSlot {
-        bool live = false;
-        uint32_t seq_len = 0;
-        std::vector<float*> k_cache, v_cache, conv_state;  // per layer (NULL where the layer has none)
-    };
-    std::vector<SeqSlot> seqs;
-    // per-category device timers of the prefill pipeline (WICK_CUDA_PROFILE=events or wick_cuda_profile_enable)
-    bool prof_on = false;
-    std::vector<cudaEvent_t> prof_events;   // pool, reused chunk after chunk
-    std::vector<int> prof_marks;            // category that ENDS at event i + 1 of the current chunk
-    size_t prof_used = 0;
-    double prof_ms[WICK_CUDA_PROFILE_CATEGORIES] = {};
-    // opt-in split-K decode attention (graph decode path and the multi-sequence step; the persistent kernel stays exact)
-    bool attn_splitk = false;
-    float* splitk_scratch = nullptr;
-    size_t splitk_floats = 0;
-    float* sample_val = nullptr;        // [vocab] work arrays of the on-device sampler, made on first use
-    int* sample_idx = nullptr;
-    uint32_t* sample_status = nullptr;
-    int batch_cap = 0;                  // rows the batch buffers below hold
-    float* logits_rows = nullptr;       // [batch_cap][vocab]
-    uint32_t *rows_tok = nullptr, *rows_next = nullptr, *rows_pos = nullptr, *rows_out = nullptr;  // device; rows_out [steps][rows]
-    size_t rows_out_cap = 0;
-    float** rows_ptrs = nullptr;        // device [n_layers][2][batch_cap] per-row state pointers
-    uint8_t* h_rows = nullptr;          // pinned staging for tokens, positions, pointers and results
-    size_t h_rows_bytes = 0;
+wick_cuda_model::wick_cuda_model() = default;
 
-    ~wick_cuda_model() {
-        cudaSetDevice(device);
-        if (stream) cudaStreamSynchronize(stream);
-        if (g_logits) cudaGraphExecDestroy(g_logits);
-        if (g_greedy) cudaGraphExecDestroy(g_greedy);
-        if (ev0) cudaEventDestroy(ev0);
-        if (ev1) cudaEventDestroy(ev1);
-        for (cudaEvent_t e : prof_events) cudaEventDestroy(e);
-        for (void* p : allocs) cudaFree(p);
-        if (h_u32) cudaFreeHost(h_u32);
-        if (h_logits) cudaFreeHost(h_logits);
-        if (h_ctl) cudaFreeHost(h_ctl);
-        if (h_rows) cudaFreeHost(h_rows);
-        if (stream) cudaStreamDestroy(stream);
-    }
-};
+wick_cuda_model::~wick_cuda_model() {
+    cudaSetDevice(device);
+    if (stream) cudaStreamSynchronize(stream);
+    if (g_logits) cudaGraphExecDestroy(g_logits);
+    if (g_greedy) cudaGraphExecDestroy(g_greedy);
+    if (ev0) cudaEventDestroy(ev0);
+    if (ev1) cudaEventDestroy(ev1);
+    for (cudaEvent_t e : prof_events) cudaEventDestroy(e);
+    for (void* p : allocs) cudaFree(p);
+    if (h_u32) cudaFreeHost(h_u32);
+    if (h_logits) cudaFreeHost(h_logits);
+    if (h_ctl) cudaFreeHost(h_ctl);
+    if (h_rows) cudaFreeHost(h_rows);
+    if (stream) cudaStreamDestroy(stream);
+}
 
 namespace {
-
-template <class T>
-int32_t dev_alloc(wick_cuda_model* m, T** out, size_t count) {
-    void* p = nullptr;
-    size_t bytes = std::max<size_t>(count * sizeof(T), 256);
-    CU_TRY(cudaMalloc(&p, bytes));
-    m->allocs.push_back(p);
-    m->bytes += bytes;
-    *out = (T*)p;
-    return WICK_CUDA_OK;
-}
 
 int32_t upload_f32(wick_cuda_model* m, const GgufImage& g, const std::string& name, size_t expect, float** out) {
     const GgufTensor* t = g.tensor(name);
@@ -316,8 +191,8 @@ int32_t build_mega(wick_cuda_model* m) {
     for (uint32_t i = 0; i < c.n_layers; i++) {
         Layer& L = m->layers[i];
         MegaLayer& M = ml[i];
-        M.conv_w = L.conv_w; M.conv_state = L.conv_state; M.q_norm = L.q_norm; M.k_norm = L.k_norm;
-        M.k_cache = L.k_cache; M.v_cache = L.v_cache; M.n_kv = L.n_kv;
+        M.conv_w = L.conv_w; M.conv_state = L.conv_state(); M.q_norm = L.q_norm; M.k_norm = L.k_norm;
+        M.k_cache = L.k_cache(); M.v_cache = L.v_cache(); M.n_kv = L.n_kv;
         MegaPhase a{};
         a.kind = MPH_NORM; a.k = hs; a.layer = (int)i; a.embed = i == 0; a.conv_commit = -1; a.norm_w = L.attn_norm;
         if (!L.is_attn) {
@@ -556,7 +431,21 @@ int32_t ensure_splitk_scratch(wick_cuda_model* m, int rows) {
     return WICK_CUDA_OK;
 }
 
-void enqueue_decode(wick_cuda_model* m, bool greedy) {
+}  // namespace
+
+// The end of a decode step on the device, for any architecture: argmax feeds the control block, or the position advances.
+void wick::enqueue_step_end(wick_cuda_model* m, bool greedy) {
+    if (greedy) {
+        launch_argmax(m->stream, m->logits, m->cfg.vocab_size, &m->ctl->argmax, m->argmax_tok);
+        launch_decode_advance(m->stream, m->ctl, m->argmax_tok, m->ring, m->ring_len);
+    } else {
+        launch_decode_advance(m->stream, m->ctl, &m->ctl->token, nullptr, 0);  // keeps the token, pos += 1
+    }
+}
+
+namespace {
+
+int32_t lfm2_enqueue_decode(wick_cuda_model* m, bool greedy) {
     cudaStream_t st = m->stream;
     const int hs = m->cfg.hidden_size, is = m->cfg.intermediate_size, hd = m->head_dim;
     embed_rows(m, nullptr, m->ctl, 1);
@@ -568,7 +457,7 @@ void enqueue_decode(wick_cuda_model* m, bool greedy) {
             GemvJob j{};
             j.count = 1; j.w[0] = L.in_proj; j.y[0] = m->proj;
             launch_gemv(st, j, m->q8s, m->q8q);
-            launch_shortconv(st, m->proj, L.conv_w, L.conv_state, 1, hs, m->cfg.conv_kernel_size, nullptr, m->q8s, m->q8q);
+            launch_shortconv(st, m->proj, L.conv_w, L.conv_state(), 1, hs, m->cfg.conv_kernel_size, nullptr, m->q8s, m->q8q);
             GemvJob o{};
             o.count = 1; o.w[0] = L.out_proj; o.y[0] = m->block_out;
             launch_gemv(st, o, m->q8s, m->q8q);
@@ -580,12 +469,12 @@ void enqueue_decode(wick_cuda_model* m, bool greedy) {
             j.w[2] = L.v; j.y[2] = m->vbuf;
             launch_gemv(st, j, m->q8s, m->q8q);
             launch_qknorm_rope_kv(st, m->qbuf, m->kbuf, m->vbuf, L.q_norm, L.k_norm, m->cfg.rms_norm_eps, m->rope_cos,
-                                  m->rope_sin, L.k_cache, L.v_cache, 1, -1, m->ctl, m->cfg.n_heads, L.n_kv, hd);
+                                  m->rope_sin, L.k_cache(), L.v_cache(), 1, -1, m->ctl, m->cfg.n_heads, L.n_kv, hd);
             if (m->attn_splitk)
-                launch_attention_splitk(st, m->qbuf, nullptr, nullptr, L.k_cache, L.v_cache, &m->ctl->pos, m->attn_out, m->splitk_scratch, 1,
+                launch_attention_splitk(st, m->qbuf, nullptr, nullptr, L.k_cache(), L.v_cache(), &m->ctl->pos, m->attn_out, m->splitk_scratch, 1,
                                         m->cfg.n_heads, L.n_kv, hd, m->cfg.max_seq_len);
             else
-                launch_attention_naive(st, m->qbuf, L.k_cache, L.v_cache, m->attn_out, 1, -1, m->ctl, m->cfg.n_heads, L.n_kv, hd,
+                launch_attention_naive(st, m->qbuf, L.k_cache(), L.v_cache(), m->attn_out, 1, -1, m->ctl, m->cfg.n_heads, L.n_kv, hd,
                                        m->cfg.max_seq_len);
             launch_quant_rows(st, m->attn_out, 1, hs, m->q8s, m->q8q);
             GemvJob o{};
@@ -606,21 +495,21 @@ void enqueue_decode(wick_cuda_model* m, bool greedy) {
     }
     launch_add_rmsnorm_quant(st, m->hidden, pending, m->output_norm, m->cfg.rms_norm_eps, 1, hs, m->q8s, m->q8q, nullptr);
     logits_matvec(m);
-    if (greedy) {
-        launch_argmax(st, m->logits, m->cfg.vocab_size, &m->ctl->argmax, m->argmax_tok);
-        launch_decode_advance(st, m->ctl, m->argmax_tok, m->ring, m->ring_len);
-    } else {
-        launch_decode_advance(st, m->ctl, &m->ctl->token, nullptr, 0);  // keeps the token, pos += 1
-    }
+    enqueue_step_end(m, greedy);
+    return WICK_CUDA_OK;
 }
 
 int32_t capture_graph(wick_cuda_model* m, bool greedy, cudaGraphExec_t* out, uint64_t* nodes) {
     cudaGraph_t graph = nullptr;
     CU_TRY(cudaStreamBeginCapture(m->stream, cudaStreamCaptureModeThreadLocal));
     const unsigned long long before = g_kernel_launches;
-    enqueue_decode(m, greedy);
+    const int32_t r = m->family->enqueue_decode(m, greedy);
     *nodes = g_kernel_launches - before;
     cudaError_t e = cudaStreamEndCapture(m->stream, &graph);
+    if (r != WICK_CUDA_OK) {
+        if (graph) cudaGraphDestroy(graph);
+        return r;
+    }
     if (e != cudaSuccess) return fail(WICK_CUDA_ERR_CUDA, std::string("graph capture: ") + cudaGetErrorString(e));
     e = cudaGraphInstantiate(out, graph, 0);
     cudaGraphDestroy(graph);
@@ -628,13 +517,14 @@ int32_t capture_graph(wick_cuda_model* m, bool greedy, cudaGraphExec_t* out, uin
     return WICK_CUDA_OK;
 }
 
+}  // namespace
+
 // Per-category device timers (the counterpart of wick's WICK_PROFILE=timing|gpu switches, metal_lfm2.rs:529-533,
 // :596-600): an event after every group of kernels of one kind; the differences are added up per category once the
 // chunk has finished.  Off by default: an event per kernel group costs a little launch time.
-enum ProfCat { PC_EMBED = 0, PC_NORM_QUANT, PC_GEMM, PC_SHORTCONV, PC_QK_ROPE_KV, PC_ATTENTION, PC_ACT_QUANT, PC_LOGITS };
 static const char* const PROF_NAMES[WICK_CUDA_PROFILE_CATEGORIES] = {"embedding", "rmsnorm+quantise", "gemm", "short-conv", "qk-norm+rope+kv-append",
-                                                                      "attention", "activation+quantise", "output-norm+logits"};
-void prof_begin(wick_cuda_model* m) {
+                                                                      "attention", "activation+quantise", "output-norm+logits", "recurrence"};
+void wick::prof_begin(wick_cuda_model* m) {
     if (!m->prof_on) return;
     m->prof_used = 0;
     m->prof_marks.clear();
@@ -647,7 +537,7 @@ void prof_begin(wick_cuda_model* m) {
         m->prof_used = 1;
     }
 }
-void prof_mark(wick_cuda_model* m, int cat) {  // the kernels enqueued since the previous mark belong to `cat`
+void wick::prof_mark(wick_cuda_model* m, int cat) {  // the kernels enqueued since the previous mark belong to `cat`
     if (!m->prof_on || m->prof_used == 0) return;
     if (m->prof_used == m->prof_events.size()) {
         cudaEvent_t e;
@@ -657,6 +547,8 @@ void prof_mark(wick_cuda_model* m, int cat) {  // the kernels enqueued since the
     cudaEventRecord(m->prof_events[m->prof_used++], m->stream);
     m->prof_marks.push_back(cat);
 }
+namespace {
+
 void prof_collect(wick_cuda_model* m) {  // after the stream has been synchronised
     if (!m->prof_on) return;
     for (size_t i = 0; i + 1 < m->prof_used; i++) {
@@ -704,10 +596,9 @@ void run_gemms(wick_cuda_model* m, int n, std::initializer_list<GemmTarget> list
 // One internal prefill chunk of n <= max_chunk tokens already in m->tokens_dev
 // (prefill_layers_and_logits, lfm2.rs:1139-2213, aarch64 non-BLAS branch).
 // `embed`: fill hidden from the token ids (false: the caller has copied input embeddings into m->hidden).
-// `last`: this chunk ends the call: the last row goes through the output norm and then, with `want_logits`,
-// through the vocabulary head (always leaving the normed row in m->normed_last).
-void enqueue_prefill_chunk(wick_cuda_model* m, int n, int start_pos, bool flash, bool last, bool embed = true,
-                           bool want_logits = true) {
+// `out`: the rows that go through the output norm (leaving the normed row in m->normed_last) and, if wanted, the
+// vocabulary head.
+int32_t lfm2_enqueue_prefill_chunk(wick_cuda_model* m, int n, int start_pos, bool flash, bool embed, const LogitRows& out) {
     cudaStream_t st = m->stream;
     const int hs = m->cfg.hidden_size, is = m->cfg.intermediate_size, hd = m->head_dim;
     const float eps = m->cfg.rms_norm_eps;
@@ -723,20 +614,20 @@ void enqueue_prefill_chunk(wick_cuda_model* m, int n, int start_pos, bool flash,
         if (!L.is_attn) {
             gemms({{&L.in_proj, &L.tc_in_proj, m->proj}});
             prof_mark(m, PC_GEMM);
-            launch_shortconv(st, m->proj, L.conv_w, L.conv_state, n, hs, m->cfg.conv_kernel_size, nullptr, m->q8s, m->q8q);
+            launch_shortconv(st, m->proj, L.conv_w, L.conv_state(), n, hs, m->cfg.conv_kernel_size, nullptr, m->q8s, m->q8q);
             prof_mark(m, PC_SHORTCONV);
             gemms({{&L.out_proj, &L.tc_out_proj, m->block_out}});
             prof_mark(m, PC_GEMM);
         } else {
             gemms({{&L.q, &L.tc_q, m->qbuf}, {&L.k, &L.tc_k, m->kbuf}, {&L.v, &L.tc_v, m->vbuf}});
             prof_mark(m, PC_GEMM);
-            launch_qknorm_rope_kv(st, m->qbuf, m->kbuf, m->vbuf, L.q_norm, L.k_norm, eps, m->rope_cos, m->rope_sin, L.k_cache,
-                                  L.v_cache, n, start_pos, nullptr, m->cfg.n_heads, L.n_kv, hd);
+            launch_qknorm_rope_kv(st, m->qbuf, m->kbuf, m->vbuf, L.q_norm, L.k_norm, eps, m->rope_cos, m->rope_sin, L.k_cache(),
+                                  L.v_cache(), n, start_pos, nullptr, m->cfg.n_heads, L.n_kv, hd);
             prof_mark(m, PC_QK_ROPE_KV);
             if (flash)  // (shapes the tiled kernel does not take were refused when the model was created)
-                launch_attention_flash(st, m->qbuf, L.k_cache, L.v_cache, m->attn_out, n, start_pos, m->cfg.n_heads, L.n_kv, hd, m->tc_err);
+                launch_attention_flash(st, m->qbuf, L.k_cache(), L.v_cache(), m->attn_out, n, start_pos, m->cfg.n_heads, L.n_kv, hd, m->tc_err);
             else
-                launch_attention_naive(st, m->qbuf, L.k_cache, L.v_cache, m->attn_out, n, start_pos, nullptr, m->cfg.n_heads,
+                launch_attention_naive(st, m->qbuf, L.k_cache(), L.v_cache(), m->attn_out, n, start_pos, nullptr, m->cfg.n_heads,
                                        L.n_kv, hd, m->cfg.max_seq_len);
             prof_mark(m, PC_ATTENTION);
             launch_quant_rows(st, m->attn_out, n, hs, m->q8s, m->q8q);
@@ -754,13 +645,18 @@ void enqueue_prefill_chunk(wick_cuda_model* m, int n, int start_pos, bool flash,
         prof_mark(m, PC_GEMM);
         pending = m->ffn_out;
     }
-    if (last) {
-        // last token only (lfm2.rs:2190-2212)
-        size_t lastrow = (size_t)(n - 1) * hs;
-        launch_add_rmsnorm_quant(st, m->hidden + lastrow, pending + lastrow, m->output_norm, eps, 1, hs, m->q8s, m->q8q, m->normed_last);
-        if (want_logits) logits_matvec(m);
-        prof_mark(m, PC_LOGITS);
+    for (int i = 0; i < out.count; i++) {
+        // wick computes the last token's logits only (lfm2.rs:2190-2212)
+        const size_t row = (size_t)out.rows[i] * hs;
+        launch_add_rmsnorm_quant(st, m->hidden + row, pending + row, m->output_norm, eps, 1, hs, m->q8s, m->q8q, m->normed_last);
+        if (!out.want_logits) continue;
+        logits_matvec(m);
+        float* dst = out.dst + (size_t)i * m->cfg.vocab_size;
+        if (dst != m->logits)
+            CU_TRY(cudaMemcpyAsync(dst, m->logits, (size_t)m->cfg.vocab_size * 4, cudaMemcpyDeviceToDevice, st));
     }
+    if (out.count) prof_mark(m, PC_LOGITS);
+    return WICK_CUDA_OK;
 }
 
 // Tensor-core prefill GEMM: decided at load (tc_ok = the shapes allow it), built on first use (ensure_tc): the int8
@@ -819,10 +715,11 @@ int32_t ensure_tc(wick_cuda_model* m) {
     return WICK_CUDA_OK;
 }
 
+// The fixed-size part of the state starts at zero; cached rows are written before they are read.
 int32_t reset_sequence(wick_cuda_model* m) {
-    const int hs = m->cfg.hidden_size, dc = (int)m->cfg.conv_kernel_size - 1;
     for (Layer& L : m->layers)
-        if (!L.is_attn && dc > 0) CU_TRY(cudaMemsetAsync(L.conv_state, 0, (size_t)dc * hs * sizeof(float), m->stream));
+        for (int b = 0; b < 2; b++)
+            if (L.sd[b].fixed) CU_TRY(cudaMemsetAsync(L.state[b], 0, L.sd[b].fixed, m->stream));
     DecodeCtl z{};
     // pinned staging keeps the copy asynchronous and ordered on the stream
     memcpy(m->h_u32, &z, sizeof(z));
@@ -832,12 +729,67 @@ int32_t reset_sequence(wick_cuda_model* m) {
     return WICK_CUDA_OK;
 }
 
-int32_t build_model(wick_cuda_model* m, const GgufImage& g, uint32_t context_size) {
+int32_t alloc_sequence_state(wick_cuda_model* m) {
+    for (Layer& L : m->layers)
+        for (int b = 0; b < 2; b++) {
+            const size_t bytes = L.sd[b].bytes(m->cfg.max_seq_len);
+            if (bytes) W_TRY(dev_alloc(m, (uint8_t**)&L.state[b], bytes));
+        }
+    return WICK_CUDA_OK;
+}
+
+}  // namespace
+
+// Tokens of activation scratch (longer prefill calls are cut into pieces of this size internally; results do not
+// depend on it).  The default is wick's own prefill chunk of 512 tokens (--ubatch-size); WICK_CUDA_MAX_CHUNK
+// overrides it (e.g. 4096: one GEMM pass per 4096-token call, at 0.45 GB more scratch for a 1.6B-class model).
+void wick::choose_max_chunk(wick_cuda_model* m) {
+    int want = 512;
+    if (const char* e = getenv("WICK_CUDA_MAX_CHUNK")) want = std::max(16, std::min(atoi(e), 8192));
+    m->max_chunk = (int)std::min<uint32_t>(m->cfg.max_seq_len, (uint32_t)want);
+}
+
+namespace {
+
+// What every architecture's handle has besides weights and scratch: control block, token ring, logits, pinned staging,
+// timers.  Needs cfg, max_chunk and the layers' state.
+int32_t init_common(wick_cuda_model* m) {
+    const wick_cuda_config& c = m->cfg;
+    W_TRY(dev_alloc(m, &m->logits, (size_t)c.vocab_size));
+    W_TRY(dev_alloc(m, &m->tokens_dev, (size_t)m->max_chunk));
+    W_TRY(dev_alloc(m, &m->normed_last, (size_t)c.hidden_size));
+    W_TRY(dev_alloc(m, &m->ctl, 1));
+    W_TRY(dev_alloc(m, &m->argmax_tok, 1));
+    m->ring_len = (int)c.max_seq_len;
+    W_TRY(dev_alloc(m, &m->ring, (size_t)m->ring_len));
+    CU_TRY(cudaMallocHost((void**)&m->h_u32, std::max<size_t>((size_t)std::max<int>(m->ring_len, m->max_chunk) * 4, 256)));
+    CU_TRY(cudaMallocHost((void**)&m->h_logits, (size_t)c.vocab_size * 4));
+    CU_TRY(cudaMallocHost((void**)&m->h_ctl, sizeof(DecodeCtl)));
+    memset(m->h_ctl, 0, sizeof(DecodeCtl));
+    CU_TRY(cudaMemset(m->ctl, 0, sizeof(DecodeCtl)));
+    W_TRY(reset_sequence(m));
+    CU_TRY(cudaEventCreate(&m->ev0));
+    CU_TRY(cudaEventCreate(&m->ev1));
+    {
+        const char* pe = getenv("WICK_CUDA_PROFILE");
+        m->prof_on = pe && strcmp(pe, "events") == 0;
+    }
+    return WICK_CUDA_OK;
+}
+
+int32_t capture_decode_graphs(wick_cuda_model* m) {
+    W_TRY(capture_graph(m, false, &m->g_logits, &m->nodes_logits));
+    W_TRY(capture_graph(m, true, &m->g_greedy, &m->nodes_greedy));
+    CU_TRY(cudaStreamSynchronize(m->stream));
+    return WICK_CUDA_OK;
+}
+
+int32_t lfm2_prepare(wick_cuda_model* m, int n) { return n >= 16 ? ensure_tc(m) : WICK_CUDA_OK; }
+int32_t lfm2_enqueue_decode_rows(wick_cuda_model* m, int n);
+const ModelFamily LFM2_FAMILY = {lfm2_enqueue_decode, lfm2_prepare, lfm2_enqueue_prefill_chunk, lfm2_enqueue_decode_rows, true};
+
+int32_t lfm2_build(wick_cuda_model* m, const GgufImage& g, uint32_t context_size) {
     // config: Lfm2Model::from_gguf_with_id, lfm2.rs:97-185
-    std::string arch;
-    if (!g.get_str("general.architecture", &arch) || arch != "lfm2")
-        return fail(WICK_CUDA_ERR_BAD_GGUF, "unsupported architecture: " + (arch.empty() ? std::string("unknown") : arch));
-    if (context_size == 0) return fail(WICK_CUDA_ERR_BAD_ARG, "context_size must be > 0");
     wick_cuda_config& c = m->cfg;
     if (!g.get_u32("lfm2.block_count", &c.n_layers)) return fail(WICK_CUDA_ERR_BAD_GGUF, "missing lfm2.block_count");
     if (!g.get_u32("lfm2.embedding_length", &c.hidden_size)) return fail(WICK_CUDA_ERR_BAD_GGUF, "missing lfm2.embedding_length");
@@ -925,15 +877,15 @@ int32_t build_model(wick_cuda_model* m, const GgufImage& g, uint32_t context_siz
             W_TRY(upload_weight(m, g, p + "attn_output.weight", hs, hs, staging, &L.o));
             W_TRY(upload_f32(m, g, p + "attn_q_norm.weight", hd, &L.q_norm));
             W_TRY(upload_f32(m, g, p + "attn_k_norm.weight", hd, &L.k_norm));
-            W_TRY(dev_alloc(m, &L.k_cache, (size_t)c.max_seq_len * kv_dim));
-            W_TRY(dev_alloc(m, &L.v_cache, (size_t)c.max_seq_len * kv_dim));
+            L.sd[0].per_pos = L.sd[1].per_pos = (size_t)kv_dim * 4;
         } else {
             W_TRY(upload_weight(m, g, p + "shortconv.in_proj.weight", 3 * hs, hs, staging, &L.in_proj));
             W_TRY(upload_weight(m, g, p + "shortconv.out_proj.weight", hs, hs, staging, &L.out_proj));
             W_TRY(upload_f32(m, g, p + "shortconv.conv.weight", (size_t)hs * c.conv_kernel_size, &L.conv_w));
-            W_TRY(dev_alloc(m, &L.conv_state, (size_t)std::max(dc, 1) * hs));
+            L.sd[0].fixed = (size_t)dc * hs * 4;
         }
     }
+    W_TRY(alloc_sequence_state(m));
     // RoPE table
     {
         std::vector<float> cs, sn;
@@ -944,14 +896,7 @@ int32_t build_model(wick_cuda_model* m, const GgufImage& g, uint32_t context_siz
         CU_TRY(cudaMemcpy(m->rope_sin, sn.data(), sn.size() * 4, cudaMemcpyHostToDevice));
     }
     // scratch
-    // Tokens of activation scratch (longer prefill calls are cut into pieces of this size internally; results do not
-    // depend on it).  The default is wick's own prefill chunk of 512 tokens (--ubatch-size); WICK_CUDA_MAX_CHUNK
-    // overrides it (e.g. 4096: one GEMM pass per 4096-token call, at 0.45 GB more scratch for a 1.6B-class model).
-    {
-        int want = 512;
-        if (const char* e = getenv("WICK_CUDA_MAX_CHUNK")) want = std::max(16, std::min(atoi(e), 8192));
-        m->max_chunk = (int)std::min<uint32_t>(c.max_seq_len, (uint32_t)want);
-    }
+    choose_max_chunk(m);
     const size_t N = m->max_chunk;
     const int kvmax = c.n_kv_heads * hd;
     W_TRY(dev_alloc(m, &m->hidden, N * hs));
@@ -964,30 +909,12 @@ int32_t build_model(wick_cuda_model* m, const GgufImage& g, uint32_t context_siz
     W_TRY(dev_alloc(m, &m->attn_out, N * hs));
     W_TRY(dev_alloc(m, &m->gate, N * is));
     W_TRY(dev_alloc(m, &m->up, N * is));
-    W_TRY(dev_alloc(m, &m->logits, (size_t)c.vocab_size));
     W_TRY(dev_alloc(m, &m->q8s, N * (std::max(hs, is) / QK)));
     W_TRY(dev_alloc(m, &m->q8q, N * std::max(hs, is)));
-    W_TRY(dev_alloc(m, &m->tokens_dev, N));
-    W_TRY(dev_alloc(m, &m->normed_last, (size_t)hs));
     W_TRY(dev_alloc(m, &m->rope_delta, (size_t)hd));
-    W_TRY(dev_alloc(m, &m->ctl, 1));
-    W_TRY(dev_alloc(m, &m->argmax_tok, 1));
-    m->ring_len = (int)c.max_seq_len;
-    W_TRY(dev_alloc(m, &m->ring, (size_t)m->ring_len));
-    CU_TRY(cudaMallocHost((void**)&m->h_u32, std::max<size_t>((size_t)std::max<int>(m->ring_len, m->max_chunk) * 4, 256)));
-    CU_TRY(cudaMallocHost((void**)&m->h_logits, (size_t)c.vocab_size * 4));
-    CU_TRY(cudaMallocHost((void**)&m->h_ctl, sizeof(DecodeCtl)));
-    memset(m->h_ctl, 0, sizeof(DecodeCtl));
-    CU_TRY(cudaMemset(m->ctl, 0, sizeof(DecodeCtl)));
-    W_TRY(reset_sequence(m));
+    W_TRY(init_common(m));
     if (naive_attn_smem(m) > 48 * 1024) {
         configure_naive_attention_smem(naive_attn_smem(m));
-    }
-    CU_TRY(cudaEventCreate(&m->ev0));
-    CU_TRY(cudaEventCreate(&m->ev1));
-    {
-        const char* pe = getenv("WICK_CUDA_PROFILE");
-        m->prof_on = pe && strcmp(pe, "events") == 0;
     }
     W_TRY(build_tc(m));
     W_TRY(build_mega(m));
@@ -998,10 +925,52 @@ int32_t build_model(wick_cuda_model* m, const GgufImage& g, uint32_t context_siz
             m->attn_splitk = true;
         }
     }
-    W_TRY(capture_graph(m, false, &m->g_logits, &m->nodes_logits));
-    W_TRY(capture_graph(m, true, &m->g_greedy, &m->nodes_greedy));
-    CU_TRY(cudaStreamSynchronize(m->stream));
-    return WICK_CUDA_OK;
+    return capture_decode_graphs(m);
+}
+
+// ── registry of architectures ──────────────────────────────────────────────
+// One line per architecture: its name in the model file, the code behind its steps, and the loader for the container
+// it comes in (a GGUF image, or a folder with config.json and model.safetensors).
+struct ArchEntry {
+    const char* name;
+    const ModelFamily* family;
+    int32_t (*build_gguf)(wick_cuda_model* m, const GgufImage& g, uint32_t context_size);
+    int32_t (*build_folder)(wick_cuda_model* m, const JsonValue& config, const SafeTensors& tensors, uint32_t context_size, int32_t compute);
+};
+const ArchEntry ARCHITECTURES[] = {
+    {"lfm2", &LFM2_FAMILY, lfm2_build, nullptr},
+    {"Nositar", &HYBRID_FAMILY, nullptr, nositar_build},
+};
+const ArchEntry* find_architecture(const std::string& name) {
+    for (const ArchEntry& a : ARCHITECTURES)
+        if (name == a.name) return &a;
+    return nullptr;
+}
+
+int32_t build_gguf_model(wick_cuda_model* m, const GgufImage& g, uint32_t context_size) {
+    g.get_str("general.architecture", &m->arch);
+    const ArchEntry* a = find_architecture(m->arch);
+    if (!a || !a->build_gguf)
+        return fail(WICK_CUDA_ERR_BAD_GGUF, "unsupported architecture: " + (m->arch.empty() ? std::string("unknown") : m->arch));
+    if (context_size == 0) return fail(WICK_CUDA_ERR_BAD_ARG, "context_size must be > 0");
+    m->family = a->family;
+    return a->build_gguf(m, g, context_size);
+}
+
+// A model folder: config.json names the architecture, model.safetensors holds the tensors.
+int32_t build_folder_model(wick_cuda_model* m, const JsonValue& config, const SafeTensors& tensors, uint32_t context_size, int32_t compute) {
+    const JsonValue* name = config.find("architecture");
+    if (name && name->is_string()) m->arch = name->str;
+    const ArchEntry* a = find_architecture(m->arch);
+    if (!a || !a->build_folder)
+        return fail(WICK_CUDA_ERR_BAD_MODEL, "unsupported architecture: " + (m->arch.empty() ? std::string("unknown") : m->arch));
+    if (context_size == 0) return fail(WICK_CUDA_ERR_BAD_ARG, "context_size must be > 0");
+    m->family = a->family;
+    CU_TRY(cudaStreamCreateWithFlags(&m->stream, cudaStreamNonBlocking));
+    W_TRY(a->build_folder(m, config, tensors, context_size, compute));
+    W_TRY(alloc_sequence_state(m));
+    W_TRY(init_common(m));
+    return capture_decode_graphs(m);
 }
 
 int32_t check_model(const wick_cuda_model* m) {
@@ -1026,12 +995,7 @@ int32_t with_slot(wick_cuda_model* m, uint32_t id, F&& fn) {
     auto swap_state = [&]() {
         for (size_t li = 0; li < m->layers.size(); li++) {
             Layer& L = m->layers[li];
-            if (L.is_attn) {
-                std::swap(L.k_cache, sl.k_cache[li]);
-                std::swap(L.v_cache, sl.v_cache[li]);
-            } else {
-                std::swap(L.conv_state, sl.conv_state[li]);
-            }
+            for (int b = 0; b < 2; b++) std::swap(L.state[b], sl.state[li * 2 + b]);
         }
         std::swap(m->seq_len, sl.seq_len);
     };
@@ -1091,7 +1055,7 @@ int32_t ensure_batch_buffers(wick_cuda_model* m, uint32_t rows, uint32_t steps) 
 // One decode step for n rows: tokens in m->rows_tok, positions in m->rows_pos, per-row state pointers in m->rows_ptrs
 // (run_layers, lfm2.rs:1020-1124, for every row; the mat-vecs as batched GEMMs, bit-identical to the mat-vec per row,
 // simd.rs:1440-1623).  Leaves the logits of every row in m->logits_rows.
-int32_t enqueue_decode_rows(wick_cuda_model* m, int n) {
+int32_t lfm2_enqueue_decode_rows(wick_cuda_model* m, int n) {
     cudaStream_t st = m->stream;
     const int hs = m->cfg.hidden_size, is = m->cfg.intermediate_size, hd = m->head_dim, cap = m->batch_cap;
     const float eps = m->cfg.rms_norm_eps;
@@ -1100,8 +1064,8 @@ int32_t enqueue_decode_rows(wick_cuda_model* m, int n) {
     const float* pending = nullptr;
     for (size_t li = 0; li < m->layers.size(); li++) {
         Layer& L = m->layers[li];
-        float** p0 = m->rows_ptrs + (li * 2) * cap;
-        float** p1 = m->rows_ptrs + (li * 2 + 1) * cap;
+        float** p0 = (float**)(m->rows_ptrs + (li * 2) * cap);
+        float** p1 = (float**)(m->rows_ptrs + (li * 2 + 1) * cap);
         launch_add_rmsnorm_quant(st, m->hidden, pending, L.attn_norm, eps, n, hs, m->q8s, m->q8q, nullptr);
         if (!L.is_attn) {
             gemms({{&L.in_proj, &L.tc_in_proj, m->proj}});
@@ -1157,7 +1121,7 @@ int32_t decode_rows(wick_cuda_model* m, const uint32_t* tokens_host, const uint3
                                                         std::to_string(m->cfg.max_seq_len));
     }
     CU_TRY(cudaSetDevice(m->device));
-    if (bs >= 16) W_TRY(ensure_tc(m));
+    W_TRY(m->family->prepare(m, (int)bs));
     if (m->attn_splitk) W_TRY(ensure_splitk_scratch(m, (int)bs));
     W_TRY(ensure_batch_buffers(m, bs, n_steps));
     const size_t nl = m->layers.size();
@@ -1165,24 +1129,24 @@ int32_t decode_rows(wick_cuda_model* m, const uint32_t* tokens_host, const uint3
     // staging: tokens, positions, then the per-layer pointer table
     uint32_t* h_tok = (uint32_t*)m->h_rows;
     uint32_t* h_pos = h_tok + cap;
-    float** h_ptr = (float**)(m->h_rows + (size_t)cap * 8);
+    void** h_ptr = (void**)(m->h_rows + (size_t)cap * 8);
     uint32_t* h_out = (uint32_t*)(m->h_rows + (size_t)cap * (8 + nl * 16));
     for (uint32_t j = 0; j < bs; j++) {
         const wick_cuda_model::SeqSlot& sl = m->seqs[seq_ids_host[j]];
         h_tok[j] = tokens_host[j];
         h_pos[j] = sl.seq_len;
         for (size_t li = 0; li < nl; li++) {
-            h_ptr[(li * 2) * cap + j] = m->layers[li].is_attn ? sl.k_cache[li] : sl.conv_state[li];
-            h_ptr[(li * 2 + 1) * cap + j] = m->layers[li].is_attn ? sl.v_cache[li] : nullptr;
+            h_ptr[(li * 2) * cap + j] = sl.state[li * 2];
+            h_ptr[(li * 2 + 1) * cap + j] = sl.state[li * 2 + 1];
         }
     }
     CU_TRY(cudaEventRecord(m->ev0, m->stream));
     CU_TRY(cudaMemcpyAsync(m->rows_tok, h_tok, (size_t)bs * 4, cudaMemcpyHostToDevice, m->stream));
     CU_TRY(cudaMemcpyAsync(m->rows_pos, h_pos, (size_t)bs * 4, cudaMemcpyHostToDevice, m->stream));
-    CU_TRY(cudaMemcpyAsync(m->rows_ptrs, h_ptr, nl * 2 * cap * sizeof(float*), cudaMemcpyHostToDevice, m->stream));
+    CU_TRY(cudaMemcpyAsync(m->rows_ptrs, h_ptr, nl * 2 * cap * sizeof(void*), cudaMemcpyHostToDevice, m->stream));
     const unsigned long long before = g_kernel_launches;
     for (uint32_t s_i = 0; s_i < n_steps; s_i++) {
-        W_TRY(enqueue_decode_rows(m, (int)bs));
+        W_TRY(m->family->enqueue_decode_rows(m, (int)bs));
         if (!logits_host) {
             launch_argmax_rows(m->stream, m->logits_rows, (int)bs, (int)m->cfg.vocab_size, m->rows_next);
             launch_rows_advance(m->stream, m->rows_tok, m->rows_next, m->rows_pos, m->rows_out, (int)bs, (int)s_i);
@@ -1257,14 +1221,39 @@ int32_t wick_cuda_model_create(const uint8_t* gguf_host, size_t gguf_len, uint32
     CU_TRY(cudaSetDevice(device));
     std::unique_ptr<wick_cuda_model> m(new wick_cuda_model());
     m->device = device;
-    int32_t r = build_model(m.get(), *img, context_size);
+    int32_t r = build_gguf_model(m.get(), *img, context_size);
     if (r != WICK_CUDA_OK) return r;
     *out = m.release();
     return WICK_CUDA_OK;
 }
 
 int32_t wick_cuda_model_create_from_file(const char* path, uint32_t context_size, int32_t device, wick_cuda_model** out) {
+    return wick_cuda_model_create_from_path(path, context_size, device, WICK_CUDA_COMPUTE_DEFAULT, out);
+}
+
+int32_t wick_cuda_model_create_from_path(const char* path, uint32_t context_size, int32_t device, int32_t compute, wick_cuda_model** out) {
     if (!path || !out) return fail(WICK_CUDA_ERR_BAD_ARG, "NULL argument");
+    *out = nullptr;
+    if (compute < WICK_CUDA_COMPUTE_DEFAULT || compute > WICK_CUDA_COMPUTE_F32) return fail(WICK_CUDA_ERR_BAD_ARG, "unknown compute type " + std::to_string(compute));
+    struct stat sb;
+    if (stat(path, &sb) == 0 && S_ISDIR(sb.st_mode)) {
+        std::unique_ptr<wick_cuda_model> m(new wick_cuda_model());
+        try {
+            const JsonValue config = JsonValue::parse_file(std::string(path) + "/config.json");
+            const SafeTensors tensors(std::string(path) + "/model.safetensors");
+            int ndev = 0;
+            CU_TRY(cudaGetDeviceCount(&ndev));
+            if (device < 0 || device >= ndev) return fail(WICK_CUDA_ERR_BAD_ARG, "no such CUDA device: " + std::to_string(device));
+            CU_TRY(cudaSetDevice(device));
+            m->device = device;
+            W_TRY(build_folder_model(m.get(), config, tensors, context_size, compute));
+        } catch (const std::exception& e) {
+            return fail(WICK_CUDA_ERR_BAD_MODEL, e.what());
+        }
+        *out = m.release();
+        return WICK_CUDA_OK;
+    }
+    if (compute != WICK_CUDA_COMPUTE_DEFAULT) return fail(WICK_CUDA_ERR_BAD_ARG, "GGUF models have one compute type: quantised integer products with f32 sums");
     std::ifstream f(path, std::ios::binary | std::ios::ate);
     if (!f) return fail(WICK_CUDA_ERR_BAD_GGUF, std::string("cannot open ") + path);
     std::streamsize len = f.tellg();
@@ -1281,6 +1270,14 @@ int32_t wick_cuda_model_config(const wick_cuda_model* m, wick_cuda_config* out) 
     if (!out) return fail(WICK_CUDA_ERR_BAD_ARG, "out is NULL");
     *out = m->cfg;
     return WICK_CUDA_OK;
+}
+
+const char* wick_cuda_model_architecture(const wick_cuda_model* m) { return m ? m->arch.c_str() : ""; }
+
+const char* wick_cuda_model_layer_type(const wick_cuda_model* m, uint32_t layer) {
+    if (!m || layer >= m->layers.size()) return "";
+    if (m->hybrid) return hybrid_layer_type(m, (int)layer);
+    return m->layers[layer].is_attn ? "Attention" : "GatedConv";
 }
 
 int32_t wick_cuda_model_kv_heads_per_layer(const wick_cuda_model* m, uint32_t* out, uint32_t n) {
@@ -1412,8 +1409,9 @@ int32_t wick_cuda_generate_greedy(wick_cuda_model* m, uint32_t first_token, uint
 
 // forward_prefill and its embedding-input relatives: exactly one of tokens_host / emb_host is given; the
 // result is the logits of the last position (logits_host) and / or its output-normed hidden row (hidden_host).
+// With `want` (n_want places among the n tokens, in any order) logits_host gets one row per place instead.
 static int32_t prefill_core(wick_cuda_model* m, const uint32_t* tokens_host, const float* emb_host, uint32_t n, uint32_t start_pos,
-                            float* logits_host, float* hidden_host) {
+                            float* logits_host, float* hidden_host, const uint32_t* want = nullptr, uint32_t n_want = 0) {
     const int hs = m->cfg.hidden_size;
     if (n == 0) return fail(WICK_CUDA_ERR_BAD_ARG, "forward_prefill requires at least one token");
     if (tokens_host)
@@ -1426,10 +1424,17 @@ static int32_t prefill_core(wick_cuda_model* m, const uint32_t* tokens_host, con
     if ((uint64_t)start_pos + n > m->cfg.max_seq_len)
         return fail(WICK_CUDA_ERR_CONTEXT_FULL, "start_pos + n = " + std::to_string((uint64_t)start_pos + n) +
                                                     " exceeds max_seq_len " + std::to_string(m->cfg.max_seq_len));
+    for (uint32_t i = 0; i < n_want; i++)
+        if (want[i] >= n) return fail(WICK_CUDA_ERR_BAD_ARG, "logits asked for at place " + std::to_string(want[i]) + " of " + std::to_string(n) + " tokens");
     CU_TRY(cudaSetDevice(m->device));
-    if (n >= 16) W_TRY(ensure_tc(m));
+    W_TRY(m->family->prepare(m, (int)n));
+    if (want && m->want_cap < m->max_chunk) {
+        W_TRY(dev_alloc(m, &m->logits_want, (size_t)m->max_chunk * m->cfg.vocab_size));
+        m->want_cap = m->max_chunk;
+    }
+    std::vector<int> rows;       // places of the chunk that get logits
     if (start_pos == 0) W_TRY(reset_sequence(m));  // new sequence, metal_lfm2.rs:2361-2397
-    const bool flash = n >= 256;  // FLASH_ATTN_THRESHOLD, lfm2.rs:1646-1647
+    const bool flash = n >= 256 && !m->hybrid;  // FLASH_ATTN_THRESHOLD, lfm2.rs:1646-1647
     CU_TRY(cudaEventRecord(m->ev0, m->stream));
     for (uint32_t c0 = 0; c0 < n; c0 += m->max_chunk) {
         uint32_t cn = std::min<uint32_t>(m->max_chunk, n - c0);
@@ -1440,16 +1445,39 @@ static int32_t prefill_core(wick_cuda_model* m, const uint32_t* tokens_host, con
             CU_TRY(cudaMemcpyAsync(m->hidden, emb_host + (size_t)c0 * hs, (size_t)cn * hs * 4, cudaMemcpyHostToDevice, m->stream));
         }
         const unsigned long long before = g_kernel_launches;
-        enqueue_prefill_chunk(m, (int)cn, (int)(start_pos + c0), flash, c0 + cn == n, tokens_host != nullptr, logits_host != nullptr);
+        LogitRows lr;
+        rows.clear();
+        if (want) {
+            for (uint32_t p = 0; p < cn; p++)   // each place once, however often it is asked for
+                for (uint32_t i = 0; i < n_want; i++)
+                    if (want[i] == c0 + p) {
+                        rows.push_back((int)p);
+                        break;
+                    }
+            lr.dst = m->logits_want;
+        } else if (c0 + cn == n) {
+            rows.push_back((int)cn - 1);
+            lr.dst = m->logits;
+            lr.want_logits = logits_host != nullptr;
+        }
+        lr.rows = rows.data();
+        lr.count = (int)rows.size();
+        W_TRY(m->family->enqueue_prefill_chunk(m, (int)cn, (int)(start_pos + c0), flash, tokens_host != nullptr, lr));
         m->launches += g_kernel_launches - before;
         CU_TRY(cudaGetLastError());
         CU_TRY(cudaStreamSynchronize(m->stream));  // h_u32 is reused by the next chunk
         prof_collect(m);
+        if (want)
+            for (size_t r = 0; r < rows.size(); r++)
+                for (uint32_t i = 0; i < n_want; i++)
+                    if (want[i] == c0 + (uint32_t)rows[r])
+                        CU_TRY(cudaMemcpy(logits_host + (size_t)i * m->cfg.vocab_size, m->logits_want + r * m->cfg.vocab_size,
+                                          (size_t)m->cfg.vocab_size * 4, cudaMemcpyDeviceToHost));
     }
     uint32_t newpos[2] = {0, start_pos + n};
     memcpy(m->h_u32, newpos, 8);
     CU_TRY(cudaMemcpyAsync(&m->ctl->pos, m->h_u32 + 1, 4, cudaMemcpyHostToDevice, m->stream));
-    if (logits_host) CU_TRY(cudaMemcpyAsync(m->h_logits, m->logits, (size_t)m->cfg.vocab_size * 4, cudaMemcpyDeviceToHost, m->stream));
+    if (logits_host && !want) CU_TRY(cudaMemcpyAsync(m->h_logits, m->logits, (size_t)m->cfg.vocab_size * 4, cudaMemcpyDeviceToHost, m->stream));
     m->h_u32[2] = 0;
     if (m->tc_err) CU_TRY(cudaMemcpyAsync(m->h_u32 + 2, m->tc_err, 4, cudaMemcpyDeviceToHost, m->stream));
     CU_TRY(cudaEventRecord(m->ev1, m->stream));
@@ -1459,7 +1487,7 @@ static int32_t prefill_core(wick_cuda_model* m, const uint32_t* tokens_host, con
         cudaMemsetAsync(m->tc_err, 0, 4, m->stream);
         return fail(WICK_CUDA_ERR_TIMEOUT, "prefill kernel (tensor-core GEMM or tiled attention): a bounded wait expired (code " + std::to_string(code) + ")");
     }
-    if (logits_host) memcpy(logits_host, m->h_logits, (size_t)m->cfg.vocab_size * 4);
+    if (logits_host && !want) memcpy(logits_host, m->h_logits, (size_t)m->cfg.vocab_size * 4);
     if (hidden_host) CU_TRY(cudaMemcpy(hidden_host, m->normed_last, (size_t)hs * 4, cudaMemcpyDeviceToHost));
     m->seq_len = start_pos + n;
     return WICK_CUDA_OK;
@@ -1506,6 +1534,7 @@ int32_t wick_cuda_forward_embedding(wick_cuda_model* m, uint32_t token, uint32_t
 // Model::shift_kv (mod.rs:158-170; lfm2.rs:2507-2516 -> kv_cache.rs:601-715).
 int32_t wick_cuda_shift_kv(wick_cuda_model* m, uint32_t n_keep, uint32_t shift) {
     W_TRY(check_model(m));
+    if (!m->family->kv_shift) return fail(WICK_CUDA_ERR_BAD_ARG, "shift_kv: architecture " + m->arch + " carries recurrent state that cannot be shifted");
     if (shift == 0) return fail(WICK_CUDA_ERR_BAD_ARG, "shift must be > 0");
     if ((uint64_t)n_keep + shift > m->seq_len)
         return fail(WICK_CUDA_ERR_BAD_ARG, "shift range out of bounds: n_keep=" + std::to_string(n_keep) + " + shift=" +
@@ -1536,10 +1565,10 @@ int32_t wick_cuda_shift_kv(wick_cuda_model* m, uint32_t n_keep, uint32_t shift) 
             for (int r0 = 0; r0 < retained; r0 += rows_per_pass) {
                 const int rows = std::min(rows_per_pass, retained - r0);
                 const int row0 = (int)n_keep + r0;
-                launch_kv_shift_gather(m->stream, L.k_cache, m->gate, row0, rows, (int)shift, kv_dim, hd, m->rope_delta, m->rope_delta + half);
-                launch_kv_shift_gather(m->stream, L.v_cache, m->up, row0, rows, (int)shift, kv_dim, hd, nullptr, nullptr);
-                CU_TRY(cudaMemcpyAsync(L.k_cache + (size_t)row0 * kv_dim, m->gate, (size_t)rows * kv_dim * 4, cudaMemcpyDeviceToDevice, m->stream));
-                CU_TRY(cudaMemcpyAsync(L.v_cache + (size_t)row0 * kv_dim, m->up, (size_t)rows * kv_dim * 4, cudaMemcpyDeviceToDevice, m->stream));
+                launch_kv_shift_gather(m->stream, L.k_cache(), m->gate, row0, rows, (int)shift, kv_dim, hd, m->rope_delta, m->rope_delta + half);
+                launch_kv_shift_gather(m->stream, L.v_cache(), m->up, row0, rows, (int)shift, kv_dim, hd, nullptr, nullptr);
+                CU_TRY(cudaMemcpyAsync(L.k_cache() + (size_t)row0 * kv_dim, m->gate, (size_t)rows * kv_dim * 4, cudaMemcpyDeviceToDevice, m->stream));
+                CU_TRY(cudaMemcpyAsync(L.v_cache() + (size_t)row0 * kv_dim, m->up, (size_t)rows * kv_dim * 4, cudaMemcpyDeviceToDevice, m->stream));
             }
         }
         m->launches += g_kernel_launches - before;
@@ -1556,6 +1585,7 @@ int32_t wick_cuda_set_prefill_mode(wick_cuda_model* m, int32_t mode) {
     W_TRY(check_model(m));
     if (mode != WICK_CUDA_PREFILL_EXACT && mode != WICK_CUDA_PREFILL_TENSOR && mode != WICK_CUDA_PREFILL_EXACT_CUDA_CORES)
         return fail(WICK_CUDA_ERR_BAD_ARG, "unknown prefill mode " + std::to_string(mode));
+    if (m->hybrid && mode != WICK_CUDA_PREFILL_EXACT) return fail(WICK_CUDA_ERR_BAD_ARG, "prefill modes are a choice of quantised models");
     if (mode == WICK_CUDA_PREFILL_TENSOR && !m->tc_ok)
         return fail(WICK_CUDA_ERR_BAD_ARG, "tensor-core prefill needs hidden and feed-forward sizes that are multiples of 128");
     m->prefill_mode = mode;
@@ -1589,17 +1619,15 @@ int32_t wick_cuda_seq_len(const wick_cuda_model* m, uint32_t* out) {
     return WICK_CUDA_OK;
 }
 
-// snapshot image: u32 magic, u32 seq_len, then per layer either K rows + V rows (seq_len x
-// kv_dim f32 each) or the conv buffer (d_conv x hidden f32)
+// snapshot image: u32 magic, u32 seq_len, then per layer its state buffers: K rows + V rows (seq_len of them) or the
+// fixed-size buffers (for lfm2 the conv buffer, d_conv x hidden f32)
 static const uint32_t SNAP_MAGIC = 0x534B4357u;  // "WCKS"
 
 int32_t wick_cuda_snapshot_size(const wick_cuda_model* m, uint64_t* bytes) {
     W_TRY(check_model(m));
     if (!bytes) return fail(WICK_CUDA_ERR_BAD_ARG, "bytes is NULL");
     uint64_t b = 8;
-    const int dc = (int)m->cfg.conv_kernel_size - 1;
-    for (const Layer& L : m->layers)
-        b += L.is_attn ? (uint64_t)2 * m->seq_len * L.n_kv * m->head_dim * 4 : (uint64_t)dc * m->cfg.hidden_size * 4;
+    for (const Layer& L : m->layers) b += L.sd[0].bytes(m->seq_len) + L.sd[1].bytes(m->seq_len);
     *bytes = b;
     return WICK_CUDA_OK;
 }
@@ -1613,21 +1641,12 @@ int32_t wick_cuda_snapshot(wick_cuda_model* m, uint8_t* out_host, uint64_t capac
     uint32_t head[2] = {SNAP_MAGIC, m->seq_len};
     memcpy(out_host, head, 8);
     uint8_t* p = out_host + 8;
-    const int dc = (int)m->cfg.conv_kernel_size - 1;
-    for (const Layer& L : m->layers) {
-        if (L.is_attn) {
-            size_t b = (size_t)m->seq_len * L.n_kv * m->head_dim * 4;
-            if (b) {
-                CU_TRY(cudaMemcpy(p, L.k_cache, b, cudaMemcpyDeviceToHost));
-                CU_TRY(cudaMemcpy(p + b, L.v_cache, b, cudaMemcpyDeviceToHost));
-            }
-            p += 2 * b;
-        } else {
-            size_t b = (size_t)dc * m->cfg.hidden_size * 4;
-            if (b) CU_TRY(cudaMemcpy(p, L.conv_state, b, cudaMemcpyDeviceToHost));
-            p += b;
+    for (const Layer& L : m->layers)
+        for (int b = 0; b < 2; b++) {
+            const size_t bytes = L.sd[b].bytes(m->seq_len);
+            if (bytes) CU_TRY(cudaMemcpy(p, L.state[b], bytes, cudaMemcpyDeviceToHost));
+            p += bytes;
         }
-    }
     return WICK_CUDA_OK;
 }
 
@@ -1649,21 +1668,12 @@ int32_t wick_cuda_restore(wick_cuda_model* m, const uint8_t* snap_host, uint64_t
     CU_TRY(cudaSetDevice(m->device));
     CU_TRY(cudaStreamSynchronize(m->stream));
     const uint8_t* p = snap_host + 8;
-    const int dc = (int)m->cfg.conv_kernel_size - 1;
-    for (const Layer& L : m->layers) {
-        if (L.is_attn) {
-            size_t b = (size_t)m->seq_len * L.n_kv * m->head_dim * 4;
-            if (b) {
-                CU_TRY(cudaMemcpy(L.k_cache, p, b, cudaMemcpyHostToDevice));
-                CU_TRY(cudaMemcpy(L.v_cache, p + b, b, cudaMemcpyHostToDevice));
-            }
-            p += 2 * b;
-        } else {
-            size_t b = (size_t)dc * m->cfg.hidden_size * 4;
-            if (b) CU_TRY(cudaMemcpy(L.conv_state, p, b, cudaMemcpyHostToDevice));
-            p += b;
+    for (const Layer& L : m->layers)
+        for (int b = 0; b < 2; b++) {
+            const size_t bytes = L.sd[b].bytes(m->seq_len);
+            if (bytes) CU_TRY(cudaMemcpy(L.state[b], p, bytes, cudaMemcpyHostToDevice));
+            p += bytes;
         }
-    }
     CU_TRY(cudaMemcpy(&m->ctl->pos, &m->seq_len, 4, cudaMemcpyHostToDevice));
     return WICK_CUDA_OK;
 }
@@ -1689,6 +1699,7 @@ int32_t wick_cuda_set_decode_attention(wick_cuda_model* m, int32_t mode) {
     if (mode != WICK_CUDA_DECODE_ATTENTION_EXACT && mode != WICK_CUDA_DECODE_ATTENTION_SPLITK)
         return fail(WICK_CUDA_ERR_BAD_ARG, "unknown decode attention mode " + std::to_string(mode));
     const bool want = mode == WICK_CUDA_DECODE_ATTENTION_SPLITK;
+    if (m->hybrid) return fail(WICK_CUDA_ERR_BAD_ARG, "set_decode_attention: not a choice for architecture " + m->arch);
     if (want == m->attn_splitk) return WICK_CUDA_OK;
     CU_TRY(cudaSetDevice(m->device));
     CU_TRY(cudaStreamSynchronize(m->stream));
@@ -1755,22 +1766,24 @@ int32_t wick_cuda_decode_path(const wick_cuda_model* m, int32_t* persistent) {
 int32_t wick_cuda_read_kv(wick_cuda_model* m, uint32_t layer, float* k_host, float* v_host) {
     W_TRY(check_model(m));
     if (layer >= m->layers.size() || !m->layers[layer].is_attn) return fail(WICK_CUDA_ERR_BAD_ARG, "not an attention layer");
+    if (m->hybrid) return fail(WICK_CUDA_ERR_BAD_ARG, "read_kv: not available for architecture " + m->arch);
     CU_TRY(cudaSetDevice(m->device));
     CU_TRY(cudaStreamSynchronize(m->stream));
     const Layer& L = m->layers[layer];
     size_t b = (size_t)m->seq_len * L.n_kv * m->head_dim * 4;
-    if (b && k_host) CU_TRY(cudaMemcpy(k_host, L.k_cache, b, cudaMemcpyDeviceToHost));
-    if (b && v_host) CU_TRY(cudaMemcpy(v_host, L.v_cache, b, cudaMemcpyDeviceToHost));
+    if (b && k_host) CU_TRY(cudaMemcpy(k_host, L.k_cache(), b, cudaMemcpyDeviceToHost));
+    if (b && v_host) CU_TRY(cudaMemcpy(v_host, L.v_cache(), b, cudaMemcpyDeviceToHost));
     return WICK_CUDA_OK;
 }
 
 int32_t wick_cuda_read_conv_state(wick_cuda_model* m, uint32_t layer, float* out_host) {
     W_TRY(check_model(m));
     if (layer >= m->layers.size() || m->layers[layer].is_attn || !out_host) return fail(WICK_CUDA_ERR_BAD_ARG, "not a conv layer");
+    if (m->hybrid) return fail(WICK_CUDA_ERR_BAD_ARG, "read_conv_state: not available for architecture " + m->arch);
     CU_TRY(cudaSetDevice(m->device));
     CU_TRY(cudaStreamSynchronize(m->stream));
     size_t b = (size_t)((int)m->cfg.conv_kernel_size - 1) * m->cfg.hidden_size * 4;
-    if (b) CU_TRY(cudaMemcpy(out_host, m->layers[layer].conv_state, b, cudaMemcpyDeviceToHost));
+    if (b) CU_TRY(cudaMemcpy(out_host, m->layers[layer].conv_state(), b, cudaMemcpyDeviceToHost));
     return WICK_CUDA_OK;
 }
 
@@ -1782,29 +1795,22 @@ int32_t wick_cuda_seq_create(wick_cuda_model* m, uint32_t* seq_id) {
     CU_TRY(cudaSetDevice(m->device));
     size_t id = 0;
     while (id < m->seqs.size() && m->seqs[id].live) id++;
-    const int hs = m->cfg.hidden_size, dc = (int)m->cfg.conv_kernel_size - 1;
     if (id == m->seqs.size()) {
         if (m->seqs.size() >= 65536) return fail(WICK_CUDA_ERR_BAD_ARG, "too many sequence slots");
         wick_cuda_model::SeqSlot sl;
         const size_t nl = m->layers.size();
-        sl.k_cache.assign(nl, nullptr);
-        sl.v_cache.assign(nl, nullptr);
-        sl.conv_state.assign(nl, nullptr);
-        for (size_t li = 0; li < nl; li++) {
-            const Layer& L = m->layers[li];
-            if (L.is_attn) {
-                const size_t rows = (size_t)m->cfg.max_seq_len * L.n_kv * m->head_dim;
-                W_TRY(dev_alloc(m, &sl.k_cache[li], rows));
-                W_TRY(dev_alloc(m, &sl.v_cache[li], rows));
-            } else {
-                W_TRY(dev_alloc(m, &sl.conv_state[li], (size_t)std::max(dc, 1) * hs));
-            }
+        sl.state.assign(nl * 2, nullptr);
+        for (size_t i = 0; i < nl * 2; i++) {
+            const size_t bytes = m->layers[i / 2].sd[i % 2].bytes(m->cfg.max_seq_len);
+            if (bytes) W_TRY(dev_alloc(m, (uint8_t**)&sl.state[i], bytes));
         }
         m->seqs.push_back(std::move(sl));
     }
     wick_cuda_model::SeqSlot& sl = m->seqs[id];  // a recycled slot keeps its buffers
-    for (size_t li = 0; li < m->layers.size(); li++)
-        if (!m->layers[li].is_attn && dc > 0) CU_TRY(cudaMemsetAsync(sl.conv_state[li], 0, (size_t)dc * hs * sizeof(float), m->stream));
+    for (size_t i = 0; i < m->layers.size() * 2; i++) {
+        const StateDesc& d = m->layers[i / 2].sd[i % 2];
+        if (d.fixed) CU_TRY(cudaMemsetAsync(sl.state[i], 0, d.fixed, m->stream));
+    }
     CU_TRY(cudaStreamSynchronize(m->stream));
     sl.live = true;
     sl.seq_len = 0;
@@ -1835,6 +1841,18 @@ int32_t wick_cuda_seq_prefill(wick_cuda_model* m, uint32_t seq_id, const uint32_
     if (!tokens_host || !logits_host) return fail(WICK_CUDA_ERR_BAD_ARG, "NULL argument");
     CU_TRY(cudaSetDevice(m->device));
     return with_slot(m, seq_id, [&]() { return prefill_core(m, tokens_host, nullptr, n, start_pos, logits_host, nullptr); });
+}
+
+int32_t wick_cuda_seq_prefill_logits(wick_cuda_model* m, uint32_t seq_id, const uint32_t* tokens_host, uint32_t n, uint32_t start_pos,
+                                     const uint32_t* want_host, uint32_t n_want, float* logits_host) {
+    static const uint32_t none = 0;
+    W_TRY(check_model(m));
+    W_TRY(check_seq(m, seq_id));
+    if (!tokens_host || (n_want && (!want_host || !logits_host))) return fail(WICK_CUDA_ERR_BAD_ARG, "NULL argument");
+    CU_TRY(cudaSetDevice(m->device));
+    return with_slot(m, seq_id, [&]() {
+        return prefill_core(m, tokens_host, nullptr, n, start_pos, logits_host, nullptr, n_want ? want_host : &none, n_want);
+    });
 }
 
 int32_t wick_cuda_decode_batch(wick_cuda_model* m, const uint32_t* tokens_host, const uint32_t* seq_ids_host, uint32_t bs,

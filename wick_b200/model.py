@@ -1,6 +1,6 @@
 """Host-side mirror of wick's `Model` trait for the CUDA backend.
 
-`CudaLfm2Model` has the methods of `trait Model` (wick/src/model/mod.rs:72-323) with the
+`CudaModel` (and its subclasses per architecture) has the methods of `trait Model` (wick/src/model/mod.rs:72-323) with the
 same names, argument meaning and failure behaviour as wick's GPU backends: the sequence
 state lives in the model (metal_lfm2.rs:170-277), every call also updates the caller's
 `InferenceState.seq_len` (metal_lfm2.rs:2146-2147), misuse raises (wick asserts), and only
@@ -12,6 +12,8 @@ from __future__ import annotations
 
 import ctypes as C
 import dataclasses
+import json
+import os
 import threading
 from typing import List, Optional, Sequence, Tuple
 
@@ -51,27 +53,38 @@ def device_count() -> int:
     return n.value
 
 
-class CudaLfm2Model:
-    """`load_model_cuda(gguf, path, context_size)`: the `--device cuda` arm of
-    engine::load_text_model (wick/src/engine.rs:1073-1102)."""
+COMPUTE_TYPES = {"default": 0, "bfloat16": 1, "float32": 2}
 
-    def __init__(self, path: str, context_size: int = 4096, device: int = 0):
+
+class CudaModel:
+    """A loaded model of any architecture behind the C ABI: the methods of `trait Model` plus sequence slots and batching.
+    `architecture` of a subclass is the name its model files carry; `load_model_cuda` picks the subclass."""
+    architecture: Optional[str] = None
+
+    def __init__(self, path: str, context_size: int = 4096, device: int = 0, dtype: str = "default"):
         self._lib = _lib.load()
         self._h = C.c_void_p()
         self._lock = threading.Lock()  # infer_lock, metal_lfm2.rs:254-267
-        check(self._lib.wick_cuda_model_create_from_file(path.encode(), context_size, device, C.byref(self._h)))
+        check(self._lib.wick_cuda_model_create_from_path(os.fspath(path).encode(), context_size, device, COMPUTE_TYPES[dtype], C.byref(self._h)))
+        self._read_config(device)
+
+    def _read_config(self, device: int) -> None:
         cfg = _lib.Config()
         check(self._lib.wick_cuda_model_config(self._h, C.byref(cfg)))
         kv = np.zeros(cfg.n_layers, np.uint32)
         check(self._lib.wick_cuda_model_kv_heads_per_layer(self._h, kv.ctypes.data, cfg.n_layers))
+        arch = self._lib.wick_cuda_model_architecture(self._h).decode()
+        if self.architecture is not None and arch != self.architecture:
+            self.close()
+            raise ValueError(f"{type(self).__name__} is for architecture {self.architecture}, the model is {arch}")
+        types = tuple(self._lib.wick_cuda_model_layer_type(self._h, i).decode() for i in range(cfg.n_layers))
         self._config = ModelConfig(
-            "lfm2", cfg.n_layers, cfg.hidden_size, cfg.intermediate_size, cfg.n_heads, cfg.n_kv_heads, cfg.vocab_size,
-            cfg.max_seq_len, cfg.rope_theta, cfg.rms_norm_eps,
-            tuple("Attention" if k else "GatedConv" for k in kv), cfg.conv_kernel_size, tuple(int(k) for k in kv))
+            arch, cfg.n_layers, cfg.hidden_size, cfg.intermediate_size, cfg.n_heads, cfg.n_kv_heads, cfg.vocab_size,
+            cfg.max_seq_len, cfg.rope_theta, cfg.rms_norm_eps, types, cfg.conv_kernel_size, tuple(int(k) for k in kv))
         self.device = device
 
     @classmethod
-    def from_bytes(cls, data: bytes, context_size: int = 4096, device: int = 0) -> "CudaLfm2Model":
+    def from_bytes(cls, data: bytes, context_size: int = 4096, device: int = 0) -> "CudaModel":
         """WickEngine::from_bytes path (engine.rs:224-363): the GGUF image is in memory."""
         self = cls.__new__(cls)
         self._lib = _lib.load()
@@ -79,15 +92,7 @@ class CudaLfm2Model:
         self._lock = threading.Lock()
         buf = (C.c_uint8 * len(data)).from_buffer_copy(data)
         check(self._lib.wick_cuda_model_create(C.addressof(buf), len(data), context_size, device, C.byref(self._h)))
-        cfg = _lib.Config()
-        check(self._lib.wick_cuda_model_config(self._h, C.byref(cfg)))
-        kv = np.zeros(cfg.n_layers, np.uint32)
-        check(self._lib.wick_cuda_model_kv_heads_per_layer(self._h, kv.ctypes.data, cfg.n_layers))
-        self._config = ModelConfig(
-            "lfm2", cfg.n_layers, cfg.hidden_size, cfg.intermediate_size, cfg.n_heads, cfg.n_kv_heads, cfg.vocab_size,
-            cfg.max_seq_len, cfg.rope_theta, cfg.rms_norm_eps,
-            tuple("Attention" if k else "GatedConv" for k in kv), cfg.conv_kernel_size, tuple(int(k) for k in kv))
-        self.device = device
+        self._read_config(device)
         return self
 
     # ---- lifetime -----------------------------------------------------------
@@ -204,7 +209,7 @@ class CudaLfm2Model:
         return out
 
     def supports_kv_shift(self) -> bool:
-        return True
+        return False
 
     def shift_kv(self, state: InferenceState, n_keep: int, shift: int) -> None:
         """Model::shift_kv (mod.rs:158-170): drop KV cells [n_keep, n_keep + shift), re-rotate the moved K rows."""
@@ -269,64 +274,16 @@ class CudaLfm2Model:
         check(self._lib.wick_cuda_decode_path(self._h, C.byref(v)))
         return "persistent" if v.value else "graph"
 
-    _PREFILL_MODES = {"exact": 0, "tensor": 1, "exact-cuda-cores": 2}
-
-    def prefill_mode(self) -> str:
-        """'exact' (default: bit-exact GEMM, on the tensor cores when the model's sizes allow),
-        'tensor' (fused-chain tcgen05 GEMM, logits equal to f32 rounding per product) or
-        'exact-cuda-cores' (the bit-exact CUDA-core GEMM)."""
-        v = C.c_int32(0)
-        check(self._lib.wick_cuda_prefill_mode(self._h, C.byref(v)))
-        return {n: k for k, n in self._PREFILL_MODES.items()}[v.value]
-
-    def set_prefill_mode(self, mode: str) -> None:
-        if mode not in self._PREFILL_MODES:
-            raise ValueError("prefill mode must be one of " + ", ".join(self._PREFILL_MODES))
-        check(self._lib.wick_cuda_set_prefill_mode(self._h, self._PREFILL_MODES[mode]))
-
-    def prefill_uses_tensor_cores(self) -> bool:
-        v = C.c_int32(0)
-        check(self._lib.wick_cuda_prefill_uses_tensor_cores(self._h, C.byref(v)))
-        return bool(v.value)
-
-    def set_decode_attention(self, mode: str) -> None:
-        """'exact' (default) or 'splitk' (opt-in, not bit-exact): see wick_cuda_set_decode_attention."""
-        check(self._lib.wick_cuda_set_decode_attention(self._h, {"exact": 0, "splitk": 1}[mode]))
-
     def profile_enable(self, on: bool = True) -> None:
         """Per-category device timers of forward_prefill (WICK_PROFILE in wick's GPU backends); clears the totals."""
         check(self._lib.wick_cuda_profile_enable(self._h, 1 if on else 0))
 
     def profile_read(self) -> dict:
         """Milliseconds per kernel category accumulated since profile_enable()."""
-        n = 8
+        n = 9
         ms = (C.c_double * n)()
         check(self._lib.wick_cuda_profile_read(self._h, ms, n))
         return {self._lib.wick_cuda_profile_category_name(i).decode(): float(ms[i]) for i in range(n)}
-
-    def decode_profile(self):
-        """Timeline of the last decode step of the persistent kernel: (kinds [n], ns [n, 4])."""
-        n = C.c_uint32(0)
-        check(self._lib.wick_cuda_decode_profile(self._h, None, None, 0, C.byref(n)))
-        ns = np.zeros((n.value + 4, 4), np.uint64)
-        kinds = np.zeros(n.value + 4, np.int32)
-        check(self._lib.wick_cuda_decode_profile(self._h, ns.ctypes.data, kinds.ctypes.data, n.value + 4, C.byref(n)))
-        self.last_profile_detail = ns[n.value:].reshape(-1)  # stamps of the phase named by WICK_CUDA_PROF_PHASE
-        return kinds[:n.value], ns[:n.value]
-
-    def read_kv(self, layer: int) -> Tuple[np.ndarray, np.ndarray]:
-        kv_dim = self._config.kv_heads_per_layer[layer] * (self._config.hidden_size // self._config.n_heads)
-        rows = self.seq_len
-        k = np.empty((rows, kv_dim), np.float32)
-        v = np.empty((rows, kv_dim), np.float32)
-        check(self._lib.wick_cuda_read_kv(self._h, layer, k.ctypes.data, v.ctypes.data))
-        return k, v
-
-    def read_conv_state(self, layer: int) -> np.ndarray:
-        s = np.empty((self._config.conv_kernel_size - 1, self._config.hidden_size), np.float32)
-        check(self._lib.wick_cuda_read_conv_state(self._h, layer, s.ctypes.data))
-        return s
-
 
     def forward_sample(self, tokens: Sequence[int], pos: int, state: InferenceState, temperature: float, top_k: int, top_p: float,
                        r: float) -> int:
@@ -364,6 +321,15 @@ class CudaLfm2Model:
             check(self._lib.wick_cuda_seq_prefill(self._h, int(seq_id), toks.ctypes.data, len(toks), int(start_pos), logits.ctypes.data))
         return logits
 
+    def seq_prefill_logits(self, seq_id: int, tokens: Sequence[int], start_pos: int, want: Sequence[int]) -> np.ndarray:
+        """seq_prefill that returns logits [len(want), vocab] of the listed places among `tokens`."""
+        toks, places = np.ascontiguousarray(tokens, np.uint32), np.ascontiguousarray(want, np.uint32)
+        logits = np.empty((len(places), self._config.vocab_size), np.float32)
+        with self._lock:
+            check(self._lib.wick_cuda_seq_prefill_logits(self._h, int(seq_id), toks.ctypes.data, len(toks), int(start_pos),
+                                                         places.ctypes.data if len(places) else None, len(places), logits.ctypes.data))
+        return logits
+
     def decode_batch(self, tokens: Sequence[int], seq_ids: Sequence[int]) -> np.ndarray:
         """One greedy step for every listed slot in one pass over the weights: next token per row."""
         toks, ids = np.ascontiguousarray(tokens, np.uint32), np.ascontiguousarray(seq_ids, np.uint32)
@@ -392,6 +358,84 @@ class CudaLfm2Model:
         return out
 
 
-def load_model_cuda(path: str, context_size: int = 4096, device: int = 0) -> CudaLfm2Model:
-    """Counterpart of load_model_metal (model/mod.rs:386-403)."""
-    return CudaLfm2Model(path, context_size, device)
+class CudaLfm2Model(CudaModel):
+    """LFM2 / LFM2.5 from a quantised GGUF file: the `--device cuda` arm of engine::load_text_model
+    (wick/src/engine.rs:1073-1102)."""
+    architecture = "lfm2"
+
+    def supports_kv_shift(self) -> bool:
+        return True
+
+    _PREFILL_MODES = {"exact": 0, "tensor": 1, "exact-cuda-cores": 2}
+
+    def prefill_mode(self) -> str:
+        """'exact' (default: bit-exact GEMM, on the tensor cores when the model's sizes allow),
+        'tensor' (fused-chain tcgen05 GEMM, logits equal to f32 rounding per product) or
+        'exact-cuda-cores' (the bit-exact CUDA-core GEMM)."""
+        v = C.c_int32(0)
+        check(self._lib.wick_cuda_prefill_mode(self._h, C.byref(v)))
+        return {n: k for k, n in self._PREFILL_MODES.items()}[v.value]
+
+    def set_prefill_mode(self, mode: str) -> None:
+        if mode not in self._PREFILL_MODES:
+            raise ValueError("prefill mode must be one of " + ", ".join(self._PREFILL_MODES))
+        check(self._lib.wick_cuda_set_prefill_mode(self._h, self._PREFILL_MODES[mode]))
+
+    def prefill_uses_tensor_cores(self) -> bool:
+        v = C.c_int32(0)
+        check(self._lib.wick_cuda_prefill_uses_tensor_cores(self._h, C.byref(v)))
+        return bool(v.value)
+
+    def set_decode_attention(self, mode: str) -> None:
+        """'exact' (default) or 'splitk' (opt-in, not bit-exact): see wick_cuda_set_decode_attention."""
+        check(self._lib.wick_cuda_set_decode_attention(self._h, {"exact": 0, "splitk": 1}[mode]))
+
+    def decode_profile(self):
+        """Timeline of the last decode step of the persistent kernel: (kinds [n], ns [n, 4])."""
+        n = C.c_uint32(0)
+        check(self._lib.wick_cuda_decode_profile(self._h, None, None, 0, C.byref(n)))
+        ns = np.zeros((n.value + 4, 4), np.uint64)
+        kinds = np.zeros(n.value + 4, np.int32)
+        check(self._lib.wick_cuda_decode_profile(self._h, ns.ctypes.data, kinds.ctypes.data, n.value + 4, C.byref(n)))
+        self.last_profile_detail = ns[n.value:].reshape(-1)  # stamps of the phase named by WICK_CUDA_PROF_PHASE
+        return kinds[:n.value], ns[:n.value]
+
+    def read_kv(self, layer: int) -> Tuple[np.ndarray, np.ndarray]:
+        kv_dim = self._config.kv_heads_per_layer[layer] * (self._config.hidden_size // self._config.n_heads)
+        rows = self.seq_len
+        k = np.empty((rows, kv_dim), np.float32)
+        v = np.empty((rows, kv_dim), np.float32)
+        check(self._lib.wick_cuda_read_kv(self._h, layer, k.ctypes.data, v.ctypes.data))
+        return k, v
+
+    def read_conv_state(self, layer: int) -> np.ndarray:
+        s = np.empty((self._config.conv_kernel_size - 1, self._config.hidden_size), np.float32)
+        check(self._lib.wick_cuda_read_conv_state(self._h, layer, s.ctypes.data))
+        return s
+
+
+class CudaNositarModel(CudaModel):
+    """Nositar from a folder with config.json and model.safetensors: hyper-connection streams over windowed sigmoid
+    attention and channel-decay delta-rule layers.  dtype "bfloat16" (default) or "float32".  The recurrent state cannot be
+    shifted, so there is no n_keep context shift."""
+    architecture = "Nositar"
+
+
+MODEL_CLASSES = {c.architecture: c for c in (CudaLfm2Model, CudaNositarModel)}
+
+
+def model_architecture(path: str) -> str:
+    """Architecture name of a model file or folder: config.json's "architecture", or lfm2 for a GGUF file (the library
+    checks general.architecture when it loads it)."""
+    if os.path.isdir(path):
+        with open(os.path.join(path, "config.json")) as f:
+            return str(json.load(f).get("architecture"))
+    return "lfm2"
+
+
+def load_model_cuda(path: str, context_size: int = 4096, device: int = 0, dtype: str = "default") -> CudaModel:
+    """Counterpart of load_model_metal (model/mod.rs:386-403): the model class is chosen by what is at `path`."""
+    arch = model_architecture(path)
+    if arch not in MODEL_CLASSES:
+        raise ValueError(f"unsupported architecture: {arch} (known: {', '.join(sorted(MODEL_CLASSES))})")
+    return MODEL_CLASSES[arch](path, context_size, device, dtype)

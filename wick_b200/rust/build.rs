@@ -17,6 +17,11 @@ const SOURCES: &[&str] = &[
     "decode_mega.cu",
     "gemm_tc.cu",
     "argmax_noalloc.cu",
+    "kernels_hyper.cu",
+    "kernels_dense.cu",
+    "kernels_mixattn.cu",
+    "kernels_delta.cu",
+    "hybrid.cu",
     "wick_cuda.cu",
 ];
 
