@@ -293,6 +293,48 @@ int32_t wick_cuda_shortconv(const float* proj_dev, const float* conv_w_dev, floa
 /* cpu_argmax (sampler.rs:8-19) of `count` logits -> *out_dev. */
 int32_t wick_cuda_argmax(const float* logits_dev, uint32_t count, uint32_t* out_dev, void* stream);
 
+/* ---- operators of the config.json models ---------------------------------------
+ * `compute` is WICK_CUDA_COMPUTE_BF16 or _F32: the type of the "act" buffers (bfloat16 or f32).  Row pitches (ld*) of act
+ * buffers are multiples of 8 elements, bases 16-byte aligned; columns between the row's length and its length rounded up to 8
+ * are read by dense and must be finite.  Device pointers, asynchronous on `stream`; dense and mix_attention synchronise it
+ * to report expired device waits as WICK_CUDA_ERR_TIMEOUT. */
+
+/* y[n][m] = x[n][k] W[m][k]^T with bfloat16 W (pitch ldw = k rounded up to 8, padding zero).  w_up_dev (optional, same shape):
+ * y = activation(W x) * (W_up x).  softcap > 0: y = softcap tanh(y / softcap).  y is act, or f32 when y_f32 != 0.  path: AUTO, or
+ * one kernel: row streaming (n <= 8), CUDA-core f32, tcgen05 (bfloat16 only). */
+#define WICK_CUDA_DENSE_AUTO 0
+#define WICK_CUDA_DENSE_ROWS 1
+#define WICK_CUDA_DENSE_F32 2
+#define WICK_CUDA_DENSE_TENSOR 3
+#define WICK_CUDA_ACT_RELU 0
+#define WICK_CUDA_ACT_SILU 1
+int32_t wick_cuda_dense(int32_t compute, const void* w_dev, const void* w_up_dev, uint32_t m, uint32_t k, uint32_t ldw, const void* x_dev,
+                        uint32_t ldx, uint32_t n, void* y_dev, uint32_t ldy, int32_t y_f32, int32_t activation, float softcap, int32_t path,
+                        void* stream);
+/* Hyper-connection streams x [n][streams][width] f32: x_t <- sum_s mix[s][t] x_s + out[t] y (when y_dev [n][width] is given, in
+ * place), then h = gain[0] * u / sqrt(mean(u^2) + eps) with u = sum_s in[s] x_s (in_dev NULL: plain sum). */
+int32_t wick_cuda_hyper_norm(int32_t compute, float* x_dev, uint32_t n, uint32_t streams, uint32_t width, const float* y_dev,
+                             const float* mix_dev, const float* out_dev, const float* in_dev, const float* gain_dev, float eps, void* h_dev,
+                             uint32_t ldh, void* stream);
+/* Windowed attention with head-blended sigmoid scores over rows start_pos.. of one sequence.  qkv act [n][ld]: heads*dim q,
+ * kv_heads*dim k, kv_heads*vdim v; q and k are divided by their root mean square per head (q in place), k and v rows are
+ * appended to the caches (act [max_seq][kv_heads*dim], [max_seq][kv_heads*vdim]).  Key j is seen by query i when j <= i and
+ * (size == 0 or i - j < size or j < keep_first).  out act [n][ldo]:
+ * out_h(i) = sum_j sigmoid(bias[h] + sum_g talk[h][g] scale q_g(i) . k_g(j)) v_h(j); talk / bias NULL: identity / zero. */
+int32_t wick_cuda_mix_attention(int32_t compute, void* qkv_dev, uint32_t ld, uint32_t n, uint32_t start_pos, void* k_cache_dev,
+                                void* v_cache_dev, uint32_t max_seq, const float* talk_dev, const float* bias_dev, uint32_t heads,
+                                uint32_t kv_heads, uint32_t dim, uint32_t vdim, float scale, float eps, uint32_t size, uint32_t keep_first,
+                                void* out_dev, uint32_t ldo, void* stream);
+/* Gated delta rule with a decay per head and key channel, over n tokens of one sequence.  proj act [n][ldp]: q, k (kv_heads*dim
+ * each) and v (heads*vdim) channels before their short convolutions (conv_w [channels][taps], last tap = current token), beta
+ * logits [heads] at off_beta; decay f32 [n][heads*dim] and gate f32 [n][heads*vdim] projections.  state f32
+ * [heads][vdim][dim rounded up to 32] and conv_state f32 [taps-1][channels] are read and updated.  out act [n][ldo]. */
+int32_t wick_cuda_channel_delta(int32_t compute, const void* proj_dev, uint32_t ldp, uint32_t off_beta, const float* decay_dev,
+                                const float* gate_dev, const float* conv_w_dev, const float* a_log_dev, const float* dt_bias_dev,
+                                const float* norm_dev, uint32_t n, uint32_t heads, uint32_t kv_heads, uint32_t dim, uint32_t vdim,
+                                uint32_t taps, float eps, float* state_dev, float* conv_state_dev, void* out_dev, uint32_t ldo,
+                                void* stream);
+
 /* Split-K decode attention (opt-in).  The default single-query attention keeps the CPU path's one serial accumulation per
  * output dim over all cached keys (attn_values, cpu.rs:1463-1509), which is bit-exact and, at thousands of keys, slow.
  * WICK_CUDA_DECODE_ATTENTION_SPLITK splits the keys of every head into runs of 256 and merges the runs' (max, sum,
@@ -315,7 +357,7 @@ int32_t wick_cuda_attention_decode_splitk(const float* q_dev, const float* k_cac
  * a CUDA event after each group of kernels of one kind and adds the differences to a running total per category
  * (milliseconds since the last enable).  wick_cuda_profile_category_name(i), i < WICK_CUDA_PROFILE_CATEGORIES, names them:
  * embedding, rmsnorm+quantise, gemm, short-conv, qk-norm+rope+kv-append, attention, activation+quantise,
- * output-norm+logits, recurrence.  (The persistent decode kernel has its own per-phase timeline: wick_cuda_decode_profile.) */
+ * output-norm+logits, recurrence (the last one only for architectures with a recurrence: lfm2 takes and fills 8).  (The persistent decode kernel has its own per-phase timeline: wick_cuda_decode_profile.) */
 #define WICK_CUDA_PROFILE_CATEGORIES 9
 int32_t wick_cuda_profile_enable(wick_cuda_model* m, int32_t on);
 int32_t wick_cuda_profile_read(wick_cuda_model* m, double* ms_out, uint32_t capacity);

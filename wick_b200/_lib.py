@@ -105,6 +105,10 @@ SIGNATURES = {
     "wick_cuda_attention_decode": [_vp, _vp, _vp, _vp, _u32, _u32, _u32, _u32, _vp],
     "wick_cuda_attention_prefill": [_vp, _vp, _vp, _vp, _u32, _u32, _u32, _u32, _u32, _i32, _vp],
     "wick_cuda_shortconv": [_vp, _vp, _vp, _vp, _u32, _u32, _u32, _vp],
+    "wick_cuda_dense": [_i32, _vp, _vp, _u32, _u32, _u32, _vp, _u32, _u32, _vp, _u32, _i32, _i32, _f, _i32, _vp],
+    "wick_cuda_hyper_norm": [_i32, _vp, _u32, _u32, _u32, _vp, _vp, _vp, _vp, _vp, _f, _vp, _u32, _vp],
+    "wick_cuda_mix_attention": [_i32, _vp, _u32, _u32, _u32, _vp, _vp, _u32, _vp, _vp, _u32, _u32, _u32, _u32, _f, _f, _u32, _u32, _vp, _u32, _vp],
+    "wick_cuda_channel_delta": [_i32, _vp, _u32, _u32, _vp, _vp, _vp, _vp, _vp, _vp, _u32, _u32, _u32, _u32, _u32, _u32, _f, _vp, _vp, _vp, _u32, _vp],
     "wick_cuda_argmax": [_vp, _u32, _vp, _vp],
     "wick_cuda_argmax_noalloc": [_vp, _u32, _vp, _vp],
 }

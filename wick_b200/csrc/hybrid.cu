@@ -207,7 +207,7 @@ struct Step {
         if (L.kind == MIX_ATTENTION) {
             launch_qk_rms_append(st, hm.bf16, hm.proj, hm.ldp, n, L.attn, rs);
             mark(PC_QK_ROPE_KV);
-            CU_TRY(launch_mix_attn(st, hm.bf16, hm.proj, hm.ldp, n, L.attn, rs, hm.mixed, hm.ldm, hm.partial, (int)m->cfg.max_seq_len));
+            CU_TRY(launch_mix_attn(st, hm.bf16, hm.proj, hm.ldp, n, L.attn, rs, hm.mixed, hm.ldm, hm.partial, (int)m->cfg.max_seq_len, m->tc_err));
             mark(PC_ATTENTION);
         } else {
             DenseCall c;

@@ -113,7 +113,7 @@ void launch_qk_rms_append(cudaStream_t st, bool bf16, void* qkv, int ld, int n, 
 size_t mix_attn_partial_floats(const MixAttnShape& s, int max_rows);
 bool mix_attn_supported(const MixAttnShape& s);
 cudaError_t launch_mix_attn(cudaStream_t st, bool bf16, const void* q, int ldq, int n, const MixAttnShape& s, const RowState& rs, void* out,
-                            int ldo, float* partial, int max_seq);
+                            int ldo, float* partial, int max_seq, uint32_t* err);
 
 // ── channel-decay delta rule ───────────────────────────────────────────────
 struct DeltaShape {

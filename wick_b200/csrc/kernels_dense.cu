@@ -1,8 +1,7 @@
 // Dense bfloat16 matrices times f32 or bfloat16 activation rows.
 //   k_dense_rows  up to DENSE_ROWS_MAX rows (decode): a warp streams R weight rows with 16-byte loads, every loaded weight
 //                 feeds all the activation rows.  HBM-bound: the weight bytes once.
-//   k_dense_simt  any number of rows, f32 multiply-adds on the CUDA cores: the f32 models' prompts, and shapes the tensor-core
-//                 kernel (gemm_bf16.cu) is not worth starting for.
+//   k_dense_simt  any number of rows, f32 multiply-adds on the CUDA cores: prompts of f32 models (bf16 models use gemm_bf16.cu).
 // Both accumulate in f32 and share the epilogues: plain store, activation(gate) * up, soft cap.
 #include "hybrid_kernels.cuh"
 
@@ -177,6 +176,7 @@ void launch_dense_simt(cudaStream_t st, bool bf16, const DenseCall& c) {
 
 cudaError_t launch_dense(cudaStream_t st, bool bf16, const DenseCall& c) {
     if (c.n <= DENSE_ROWS_MAX) launch_dense_rows(st, bf16, c);
+    else if (bf16) return launch_dense_tc(st, c);
     else launch_dense_simt(st, bf16, c);
     return cudaGetLastError();
 }

@@ -192,7 +192,7 @@ size_t mix_attn_partial_floats(const MixAttnShape& s, int max_rows) {
 }
 
 cudaError_t launch_mix_attn(cudaStream_t st, bool bf16, const void* q, int ldq, int n, const MixAttnShape& s, const RowState& rs, void* out,
-                            int ldo, float* partial, int max_seq) {
+                            int ldo, float* partial, int max_seq, uint32_t* err) {
     if (n <= 0) return cudaSuccess;
     return bf16 ? mix_attn_go<__nv_bfloat16>(st, q, ldq, n, s, rs, out, ldo, partial, max_seq)
                 : mix_attn_go<float>(st, q, ldq, n, s, rs, out, ldo, partial, max_seq);

@@ -1724,8 +1724,9 @@ int32_t wick_cuda_profile_enable(wick_cuda_model* m, int32_t on) {
 
 int32_t wick_cuda_profile_read(wick_cuda_model* m, double* ms_out, uint32_t capacity) {
     W_TRY(check_model(m));
-    if (!ms_out || capacity < WICK_CUDA_PROFILE_CATEGORIES) return fail(WICK_CUDA_ERR_BAD_ARG, "ms_out is NULL or shorter than WICK_CUDA_PROFILE_CATEGORIES");
-    for (int i = 0; i < WICK_CUDA_PROFILE_CATEGORIES; i++) ms_out[i] = m->prof_ms[i];
+    const uint32_t need = m->hybrid ? WICK_CUDA_PROFILE_CATEGORIES : PC_RECURRENCE;  // lfm2 has no recurrence category
+    if (!ms_out || capacity < need) return fail(WICK_CUDA_ERR_BAD_ARG, "ms_out is NULL or shorter than the categories of this architecture");
+    for (uint32_t i = 0; i < std::min<uint32_t>(capacity, WICK_CUDA_PROFILE_CATEGORIES); i++) ms_out[i] = m->prof_ms[i];
     return WICK_CUDA_OK;
 }
 

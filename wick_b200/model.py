@@ -60,6 +60,7 @@ class CudaModel:
     """A loaded model of any architecture behind the C ABI: the methods of `trait Model` plus sequence slots and batching.
     `architecture` of a subclass is the name its model files carry; `load_model_cuda` picks the subclass."""
     architecture: Optional[str] = None
+    _profile_categories = 9
 
     def __init__(self, path: str, context_size: int = 4096, device: int = 0, dtype: str = "default"):
         self._lib = _lib.load()
@@ -280,7 +281,7 @@ class CudaModel:
 
     def profile_read(self) -> dict:
         """Milliseconds per kernel category accumulated since profile_enable()."""
-        n = 9
+        n = self._profile_categories
         ms = (C.c_double * n)()
         check(self._lib.wick_cuda_profile_read(self._h, ms, n))
         return {self._lib.wick_cuda_profile_category_name(i).decode(): float(ms[i]) for i in range(n)}
@@ -362,6 +363,7 @@ class CudaLfm2Model(CudaModel):
     """LFM2 / LFM2.5 from a quantised GGUF file: the `--device cuda` arm of engine::load_text_model
     (wick/src/engine.rs:1073-1102)."""
     architecture = "lfm2"
+    _profile_categories = 8     # no recurrence
 
     def supports_kv_shift(self) -> bool:
         return True

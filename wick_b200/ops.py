@@ -167,6 +167,68 @@ def shortconv(proj: torch.Tensor, conv_w: torch.Tensor, state: torch.Tensor, ker
     return out
 
 
+# ── operators of the config.json models; the activation type is that of the tensors ────────────────────
+_DENSE_PATHS = {"auto": 0, "rows": 1, "f32": 2, "tensor": 3}
+_ACTIVATIONS = {"relu": 0, "silu": 1}
+
+
+def _compute(t: torch.Tensor) -> int:
+    return {torch.bfloat16: 1, torch.float32: 2}[t.dtype]
+
+
+def _opt(t) -> int | None:
+    return None if t is None else _ptr(t)
+
+
+def pad8(t: torch.Tensor) -> torch.Tensor:
+    """Rows of a matrix zero-padded to a multiple of 8 columns."""
+    return torch.nn.functional.pad(t, (0, -t.shape[-1] % 8)).contiguous()
+
+
+def dense(w: torch.Tensor, x: torch.Tensor, w_up: torch.Tensor | None = None, activation: str = "relu", softcap: float = 0.0,
+          out_f32: bool = True, path: str = "auto") -> torch.Tensor:
+    """x [n, k] (bf16 or f32) times bf16 w [m, k] transposed; with w_up: activation(w x) * (w_up x)."""
+    (m, k), n = w.shape, x.shape[0]
+    w8, u8, x8 = pad8(w), None if w_up is None else pad8(w_up), pad8(x)
+    y = torch.empty((n, m), dtype=torch.float32 if out_f32 else x.dtype, device=x.device)
+    check(_lib.load().wick_cuda_dense(_compute(x), _ptr(w8), _opt(u8), m, k, w8.shape[1], _ptr(x8), x8.shape[1], n, _ptr(y), m, int(out_f32),
+                                      _ACTIVATIONS[activation], softcap, _DENSE_PATHS[path], _stream()))
+    return y
+
+
+def hyper_norm(x: torch.Tensor, gain: torch.Tensor, eps: float, w_in=None, y=None, mix=None, w_out=None, dtype=torch.float32) -> torch.Tensor:
+    """Hyper-connection write (in place on x [n, streams, width]), read and RMS norm; returns h [n, width] of `dtype`."""
+    n, s, w = x.shape
+    h = torch.zeros((n, w + -w % 8), dtype=dtype, device=x.device)
+    check(_lib.load().wick_cuda_hyper_norm(_compute(h), _ptr(x), n, s, w, _opt(y), _opt(mix), _opt(w_out), _opt(w_in), _ptr(gain), eps, _ptr(h),
+                                           h.shape[1], _stream()))
+    return h[:, :w]
+
+
+def mix_attention(qkv: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, start_pos: int, heads: int, kv_heads: int, dim: int, vdim: int,
+                  scale: float, eps: float, size: int, keep_first: int, talk=None, bias=None) -> torch.Tensor:
+    """Windowed attention with head-blended sigmoid scores; appends to the caches [max_seq, kv_heads * dim | vdim]."""
+    n = qkv.shape[0]
+    q8 = pad8(qkv)
+    out = torch.zeros((n, heads * vdim + -(heads * vdim) % 8), dtype=qkv.dtype, device=qkv.device)
+    check(_lib.load().wick_cuda_mix_attention(_compute(qkv), _ptr(q8), q8.shape[1], n, start_pos, _ptr(k_cache), _ptr(v_cache), k_cache.shape[0],
+                                              _opt(talk), _opt(bias), heads, kv_heads, dim, vdim, scale, eps, size, keep_first, _ptr(out),
+                                              out.shape[1], _stream()))
+    return out[:, :heads * vdim]
+
+
+def channel_delta(proj: torch.Tensor, off_beta: int, decay: torch.Tensor, gate: torch.Tensor, conv_w: torch.Tensor, a_log: torch.Tensor,
+                  dt_bias: torch.Tensor, norm: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int, eps: float, state: torch.Tensor,
+                  conv_state: torch.Tensor) -> torch.Tensor:
+    """Short convolutions, channel-decay delta rule and gated output norm; state and conv_state are updated."""
+    n = proj.shape[0]
+    out = torch.zeros((n, heads * vdim), dtype=proj.dtype, device=proj.device)
+    check(_lib.load().wick_cuda_channel_delta(_compute(proj), _ptr(proj), proj.shape[1], off_beta, _ptr(decay), _ptr(gate), _ptr(conv_w), _ptr(a_log),
+                                              _ptr(dt_bias), _ptr(norm), n, heads, kv_heads, dim, vdim, conv_w.shape[1], eps, _ptr(state),
+                                              _ptr(conv_state), _ptr(out), heads * vdim, _stream()))
+    return out
+
+
 def argmax(logits: torch.Tensor) -> torch.Tensor:
     out = torch.empty(1, dtype=torch.int32, device=logits.device)
     check(_lib.load().wick_cuda_argmax(_ptr(logits), logits.numel(), _ptr(out), _stream()))

@@ -19,8 +19,10 @@ const SOURCES: &[&str] = &[
     "argmax_noalloc.cu",
     "kernels_hyper.cu",
     "kernels_dense.cu",
+    "gemm_bf16.cu",
     "kernels_mixattn.cu",
     "kernels_delta.cu",
+    "hybrid_ops.cu",
     "hybrid.cu",
     "wick_cuda.cu",
 ];
