@@ -261,6 +261,100 @@ def serving_side_line(m, spec, args, gs, hbm_peak):
     }
 
 
+def time_design(m, vocab, args, prompts, batch):
+    """Prefill, decode at batch 1 and batched decode of a loaded model of any architecture: p50 over repeats, CUDA-event time
+    on the library's stream."""
+    from wick_b200 import gguf_synth as gs
+    from wick_b200.model import InferenceState
+    st, out = InferenceState(), {}
+    for n in prompts:
+        toks = gs.random_prompt(n, vocab, seed=7)
+        for _ in range(2):
+            m.forward_prefill_chunked(toks, 0, st, 0)
+        ms = []
+        for _ in range(PREFILL_REPEATS):
+            m.forward_prefill_chunked(toks, 0, st, 0)
+            ms.append(m.last_chunked_device_ms)
+        out[f"prefill_p{n}_tok_s"] = n / (statistics.median(ms) * 1e-3)
+        m.profile_enable(True)
+        m.forward_prefill_chunked(toks, 0, st, 0)
+        out[f"prefill_p{n}_ms_by_category"] = {k: round(v, 3) for k, v in m.profile_read().items() if v}
+        m.profile_enable(False)
+    for start in (128, 1024):
+        toks = gs.random_prompt(start, vocab, seed=8)
+        ms = []
+        for _ in range(3):
+            m.forward_prefill_chunked(toks, 0, st, 0)
+            m.generate_greedy(1, DECODE_TOKENS, st)
+            ms.append(m.last_elapsed_ms() / DECODE_TOKENS)
+        out[f"decode_at_{start}_ms"] = statistics.median(ms)
+        out[f"decode_at_{start}_tok_s"] = 1e3 / statistics.median(ms)
+    for b in batch:
+        ids = [m.seq_create() for _ in range(b)]
+        for i, s in enumerate(ids):
+            m.seq_prefill(s, gs.random_prompt(256, vocab, seed=100 + i), 0)
+        m.decode_batch_steps([1] * b, ids, 4)
+        m.decode_batch_steps([1] * b, ids, 32)
+        out[f"decode_batch{b}_tok_s"] = 32 * b / (m.last_elapsed_ms() * 1e-3)
+        for s in ids:
+            m.seq_destroy(s)
+    return out
+
+
+def run_nositar(args):
+    """Throughput of the Nositar design at sizes that resemble a real model's layers, beside the closest other model of the
+    library at equal size (LFM2: same width, feed-forward, vocabulary, layer count and attention layers; quantised weights)."""
+    from wick_b200 import gguf_synth as gs
+    from wick_b200 import nositar_synth as ns
+    from wick_b200.model import CudaLfm2Model, CudaNositarModel
+    os.environ.setdefault("WICK_CUDA_MAX_CHUNK", "4096")
+    hbm, kind = measured_peak()
+    int8_peak, _ = int8_peak_tflops()
+    sampler = ClockSampler(int(os.environ.get("LOCAL_RANK", "0")))
+    sampler.start()
+    t0 = time.time()
+    res = {}
+    for name in args.sizes.split(","):
+        spec = ns.SPECS[name]
+        m = CudaNositarModel(ns.cached_model(name), 4608)
+        d = time_design(m, spec.vocab, args, (128, 1024, 4096), (8, 64))
+        m.close()
+        gf = 2.0 * spec.matrix_params_per_layer()
+        for n in (1024, 4096):
+            c = d[f"prefill_p{n}_ms_by_category"]
+            seen = sum(min(i + 1, spec.window + spec.keep_first) for i in range(n))
+            d[f"gemm_p{n}_frac_of_bf16_peak"] = gf * n / (c["gemm"] * 1e-3) / 1e12 / (int8_peak / 2)
+            d[f"attention_p{n}_frac_of_bf16_peak"] = (4.0 * spec.width * seen * len(spec.attn_layers) / (c["attention"] * 1e-3) / 1e12) / (int8_peak / 2)
+            nd = spec.n_layers - len(spec.attn_layers)
+            d[f"recurrence_p{n}_frac_of_f32_peak"] = 8.0 * n * nd * spec.width * (spec.width // spec.delta_heads) / (c["recurrence"] * 1e-3) / 74.4e12
+            d[f"streams_p{n}_frac_of_hbm"] = (n * spec.width * (8 * spec.streams + 6) * (2 * spec.n_layers)) / (c["rmsnorm+quantise"] * 1e-3) / 1e9 / hbm
+        for p in (128, 1024):
+            d[f"decode_at_{p}_frac_of_hbm"] = spec.decode_bytes_per_token(p + DECODE_TOKENS // 2) / (d[f"decode_at_{p}_ms"] * 1e-3) / 1e9 / hbm
+        ls = spec.lfm2()
+        path = os.path.join(os.environ.get("WICK_SYNTH_CACHE", "/tmp/wick_b200_models"), f"{ls.name}.gguf")
+        if not os.path.exists(path):
+            gs.write_lfm2_gguf(path, ls, "q8_0", 0)
+        m = CudaLfm2Model(path, 4608)
+        e = time_design(m, ls.vocab, args, (128, 1024, 4096), (8, 64))
+        m.close()
+        lp = (ls.quant_bytes("q8_0") // 34 * 32) - ls.vocab * ls.hidden
+        for n in (1024, 4096):
+            c = e[f"prefill_p{n}_ms_by_category"]
+            e[f"gemm_p{n}_frac_of_int8_peak"] = 2.0 * lp * n / (c["gemm"] * 1e-3) / 1e12 / int8_peak
+            e[f"attention_p{n}_frac_of_bf16_peak"] = (4.0 * ls.hidden * (n * (n + 1) / 2) * len(ls.attn_layers) / (c["attention"] * 1e-3) / 1e12) / (int8_peak / 2)
+            e[f"norms_p{n}_frac_of_hbm"] = (n * ls.hidden * 13.0 * (2 * ls.n_layers)) / (c["rmsnorm+quantise"] * 1e-3) / 1e9 / hbm
+        for p in (128, 1024):
+            e[f"decode_at_{p}_frac_of_hbm"] = ls.decode_bytes_per_token("q8_0") / (e[f"decode_at_{p}_ms"] * 1e-3) / 1e9 / hbm
+        rnd = lambda x: {k: (round(v, 4) if isinstance(v, float) else v) for k, v in x.items()}  # noqa: E731
+        res[name] = {"nositar_bf16": rnd(d), "lfm2_q8_0_equal_size": rnd(e)}
+    clocks = sampler.stop(t0, time.time())
+    print(json.dumps({"metric": "prefill tok/s @4096, Nositar layers", "value": res[args.sizes.split(",")[-1]]["nositar_bf16"]["prefill_p4096_tok_s"], "unit": "tok/s",
+                      "n_gpus": 1, "higher_is_better": True, "dtype": "bf16", "data": "synthetic", "peaks": {"hbm_gbs": hbm, "bf16_tflops": int8_peak / 2, "source": kind},
+                      "config": {"workload": "6-layer models (2 windowed attention, 4 delta rule), random weights, WICK_CUDA_MAX_CHUNK=" + os.environ["WICK_CUDA_MAX_CHUNK"],
+                                 "l2": "weights and activations larger than L2 for the prompt of 4096"},
+                      "clocks": clocks, "sizes": res}))
+
+
 def workload_config(args, spec):
     return {
         "workload": f"{spec.name} {args.qtype.upper()} bs=1: {PROMPT_TOKENS}-token uniform-random prompt prefill (untimed), "
@@ -284,8 +378,10 @@ def main():
     ap.add_argument("--decode-tokens", type=int, default=DECODE_TOKENS, help="profiling aid; the metric is quoted at 128")
     ap.add_argument("--no-extra", action="store_true", help="skip the prefill / tg512 side measurements")
     ap.add_argument("--no-cpu-baseline", action="store_true")
-    ap.add_argument("--only", default="decode", choices=["decode", "prefill"],
-                    help="profiling aid: 'prefill' times forward_prefill_chunked of --prompt-tokens instead of the headline decode")
+    ap.add_argument("--only", default="decode", choices=["decode", "prefill", "nositar"],
+                    help="profiling aid: 'prefill' times forward_prefill_chunked of --prompt-tokens instead of the headline decode; "
+                         "'nositar' times layers of the Nositar design beside LFM2 layers of equal size (own JSON line)")
+    ap.add_argument("--sizes", default="nositar-w1024,nositar-w2048", help="models of --only nositar")
     ap.add_argument("--prefill-mode", default="exact", choices=["exact", "tensor", "exact-cuda-cores"])
     ap.add_argument("--context", type=int, default=4096, help="context size the model is created with (prompt + decode tokens must fit)")
     ap.add_argument("--ubatch", type=int, default=512, help="prefill chunk of --only prefill (0 = one call); wick's default is 512")
@@ -318,6 +414,10 @@ def main():
         if world > 1:
             dist.barrier()
         torch.cuda.synchronize()
+
+    if args.only == "nositar":
+        run_nositar(args)
+        return
 
     path, spec = model_file(args, rank, world)
     barrier()

@@ -24,7 +24,7 @@ CONFIGS = {
                    width=192, vocab=300, streams=4),
     "d": nm.config([nm.attention(2, 2, 8, 8, 1, 1, 0), nm.delta(1, 1, 8, 8, 1, 9)], width=16, vocab=40, streams=1, softcap=30.0),
 }
-TOL = {"float32": 1e-4, "bfloat16": 8e-2}   # the models are narrow: bfloat16 rounding averages little
+TOL = {"float32": 1e-4, "bfloat16": 0.2}   # worst position; the models are narrow (down to 16), so bfloat16 rounding averages little
 
 
 class Case:
