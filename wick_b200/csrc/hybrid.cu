@@ -205,9 +205,9 @@ struct Step {
         W_TRY(dense(L.proj, hm.h, hm.ldh, hm.proj, hm.ldp, false));
         mark(PC_GEMM);
         if (L.kind == MIX_ATTENTION) {
-            launch_qk_rms_append(st, hm.bf16, hm.proj, hm.ldp, n, L.attn, rs);
+            launch_qk_rms_append(st, hm.bf16, hm.proj, hm.ldp, n, L.attn, rs, hm.attn);
             mark(PC_QK_ROPE_KV);
-            CU_TRY(launch_mix_attn(st, hm.bf16, hm.proj, hm.ldp, n, L.attn, rs, hm.mixed, hm.ldm, hm.partial, (int)m->cfg.max_seq_len, m->tc_err));
+            CU_TRY(launch_mix_attn(st, hm.bf16, hm.proj, hm.ldp, n, L.attn, rs, hm.mixed, hm.ldm, hm.attn, (int)m->cfg.max_seq_len));
             mark(PC_ATTENTION);
         } else {
             DenseCall c;
@@ -356,7 +356,7 @@ int32_t nositar_build(wick_cuda_model* m, const JsonValue& config, const SafeTen
     hm.layers.resize(c.n_layers);
     m->layers.resize(c.n_layers);
     int ldp = 8, ldm = 8, ldf = 8, lda = 8, ldg = 8;
-    size_t partial = 0, wq = 0, wv = 0, wg = 0, wb = 0, wk = 0;
+    size_t partial = 0, fold = 0, wq = 0, wv = 0, wg = 0, wb = 0, wk = 0;
     for (uint32_t i = 0; i < c.n_layers; i++) {
         const JsonValue& lc = list.items[i];
         HybridLayer& L = hm.layers[i];
@@ -368,7 +368,10 @@ int32_t nositar_build(wick_cuda_model* m, const JsonValue& config, const SafeTen
             W_TRY(load_attention(ld, p + "mix.", mc, hm.width, &L, &m->layers[i], act_bytes));
             const MixAttnShape& s = L.attn;
             ldm = std::max(ldm, s.heads * s.vdim);
-            partial = std::max(partial, mix_attn_partial_floats(s, m->max_chunk));
+            size_t pf = 0, fb = 0;
+            mix_attn_scratch(s, hm.bf16, m->max_chunk, &pf, &fb);
+            partial = std::max(partial, pf);
+            fold = std::max(fold, fb);
             c.n_heads = std::max<uint32_t>(c.n_heads, s.heads);
             c.n_kv_heads = std::max<uint32_t>(c.n_kv_heads, s.kv_heads);
         } else if (L.type == "channel_delta" || L.type.rfind("channel_delta_", 0) == 0) {  // one mechanism; the name numbers its size
@@ -429,7 +432,8 @@ int32_t nositar_build(wick_cuda_model* m, const JsonValue& config, const SafeTen
     W_TRY(dev_alloc(m, &hm.y, N * hm.ldw));
     W_TRY(dev_alloc(m, &hm.a, N * hm.lda));
     W_TRY(dev_alloc(m, &hm.gate, N * hm.ldg));
-    W_TRY(dev_alloc(m, &hm.partial, partial));
+    W_TRY(dev_alloc(m, &hm.attn.partial, partial));
+    if (fold) W_TRY(dev_alloc(m, (uint8_t**)&hm.attn.fold, fold));
     W_TRY(dev_alloc(m, &hm.work.q, N * wq));
     W_TRY(dev_alloc(m, &hm.work.k, N * wq));
     W_TRY(dev_alloc(m, &hm.work.v, N * wv));
@@ -440,6 +444,7 @@ int32_t nositar_build(wick_cuda_model* m, const JsonValue& config, const SafeTen
     W_TRY(dev_alloc(m, &hm.rows_dev, N));
     W_TRY(dev_alloc(m, &m->tc_err, 1));
     CU_TRY(cudaMemset(m->tc_err, 0, 4));
+    hm.attn.err = m->tc_err;
     CU_TRY(cudaMallocHost((void**)&hm.h_rows, N * sizeof(int)));
     return WICK_CUDA_OK;
 }

@@ -51,7 +51,7 @@ struct HybridModel {
     void* ff = nullptr;        // act [rows][ldf] activated feed-forward
     float* y = nullptr;        // [rows][ldw] sublayer output
     float *a = nullptr, *gate = nullptr;  // [rows][lda] decay projection, [rows][ldg] gate projection
-    float* partial = nullptr;  // key splits of the attention
+    MixAttnScratch attn;
     DeltaWork work;
     int* rows_dev = nullptr;   // rows of a chunk that get logits
     int* h_rows = nullptr;     // pinned staging of the same

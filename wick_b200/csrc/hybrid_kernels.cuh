@@ -106,14 +106,26 @@ struct MixAttnShape {
     const float* bias = nullptr;  // [H] added to the blended score, or NULL
     int seen(int max_seq) const { return size > 0 && size + keep_first < max_seq ? size + keep_first : max_seq; }
 };
-// Splits qkv [n][ld] (heads*dim q, kv_heads*dim k, kv_heads*vdim v): q and k divided by their root mean square per head, q
-// back in place, k and v rows appended to the caches (act [pos][kv_heads*dim], [pos][kv_heads*vdim]).
-void launch_qk_rms_append(cudaStream_t st, bool bf16, void* qkv, int ld, int n, const MixAttnShape& s, const RowState& rs);
-// out act [n][ldo] (heads*vdim).  partial: mix_attn_partial_floats() floats.
-size_t mix_attn_partial_floats(const MixAttnShape& s, int max_rows);
+// Work memory of one attention layer: mix_attn_scratch() says how much for up to max_rows rows.
+struct MixAttnScratch {
+    float* partial = nullptr;  // key splits
+    void* fold = nullptr;      // folded queries of the tensor-core form (bf16), 16-byte aligned
+    uint32_t* err = nullptr;   // device word for expired waits
+};
+void mix_attn_scratch(const MixAttnShape& s, bool bf16, int max_rows, size_t* partial_floats, size_t* fold_bytes);
 bool mix_attn_supported(const MixAttnShape& s);
-cudaError_t launch_mix_attn(cudaStream_t st, bool bf16, const void* q, int ldq, int n, const MixAttnShape& s, const RowState& rs, void* out,
-                            int ldo, float* partial, int max_seq, uint32_t* err);
+// Splits qkv [n][ld] (heads*dim q, kv_heads*dim k, kv_heads*vdim v): q and k divided by their root mean square per head, k and
+// v rows appended to the caches (act [pos][kv_heads*dim], [pos][kv_heads*vdim]); q back in place or, where the tensor-core form
+// follows, folded into sc.fold.
+void launch_qk_rms_append(cudaStream_t st, bool bf16, void* qkv, int ld, int n, const MixAttnShape& s, const RowState& rs, const MixAttnScratch& sc);
+// out act [n][ldo] (heads*vdim), after launch_qk_rms_append of the same rows.
+cudaError_t launch_mix_attn(cudaStream_t st, bool bf16, const void* qkv, int ld, int n, const MixAttnShape& s, const RowState& rs, void* out,
+                            int ldo, const MixAttnScratch& sc, int max_seq);
+// The tensor-core form (attn_mix_tc.cu): consecutive bf16 tokens of one sequence, sizes that are multiples of 8.
+constexpr int MIX_ATTN_TC_MIN_ROWS = 16;
+bool mix_attn_tc_supported(const MixAttnShape& s);
+void launch_qk_fold_append(cudaStream_t st, const void* qkv, int ld, int n, const MixAttnShape& s, const RowState& rs, void* fold);
+cudaError_t launch_mix_attn_tc(cudaStream_t st, const void* fold, int n, const MixAttnShape& s, const RowState& rs, void* out, int ldo, uint32_t* err);
 
 // ── channel-decay delta rule ───────────────────────────────────────────────
 struct DeltaShape {

@@ -103,14 +103,19 @@ int32_t wick_cuda_mix_attention(int32_t compute, void* qkv_dev, uint32_t ld, uin
         return fail(WICK_CUDA_ERR_BAD_ARG, "mix_attention: inconsistent sizes");
     if (n == 0) return WICK_CUDA_OK;
     cudaStream_t st = (cudaStream_t)stream;
-    Scratch partial, err;
-    CU_TRY(partial.get(st, mix_attn_partial_floats(s, (int)n) * 4));
+    Scratch partial, fold, err;
+    size_t pf = 0, fb = 0;
+    mix_attn_scratch(s, bf16, (int)n, &pf, &fb);
+    CU_TRY(partial.get(st, pf * 4));
+    if (fb) CU_TRY(fold.get(st, fb));
     CU_TRY(err.get(st, 4));
     CU_TRY(cudaMemsetAsync(err.p, 0, 4, st));
     RowState rs;
     rs.s0 = k_cache_dev; rs.s1 = v_cache_dev; rs.start_pos = (int)start_pos;
-    launch_qk_rms_append(st, bf16, qkv_dev, (int)ld, (int)n, s, rs);
-    CU_TRY(launch_mix_attn(st, bf16, qkv_dev, (int)ld, (int)n, s, rs, out_dev, (int)ldo, (float*)partial.p, (int)max_seq, (uint32_t*)err.p));
+    MixAttnScratch sc;
+    sc.partial = (float*)partial.p; sc.fold = fold.p; sc.err = (uint32_t*)err.p;
+    launch_qk_rms_append(st, bf16, qkv_dev, (int)ld, (int)n, s, rs, sc);
+    CU_TRY(launch_mix_attn(st, bf16, qkv_dev, (int)ld, (int)n, s, rs, out_dev, (int)ldo, sc, (int)max_seq));
     uint32_t h = 0;
     CU_TRY(cudaMemcpyAsync(&h, err.p, 4, cudaMemcpyDeviceToHost, st));
     CU_TRY(cudaStreamSynchronize(st));

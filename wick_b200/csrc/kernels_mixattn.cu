@@ -5,7 +5,7 @@
 // key) pair, so a CTA works on all heads of its queries; there is no normaliser, so partial sums over disjoint keys simply
 // add up, and the keys of a query tile can be split over CTAs.
 //
-// k_mix_attn computes in f32 on the CUDA cores and takes any sizes.
+// k_mix_attn computes in f32 on the CUDA cores and takes any sizes; prompts of bf16 models go to attn_mix_tc.cu.
 #include "hybrid_kernels.cuh"
 
 namespace wick {
@@ -176,8 +176,14 @@ cudaError_t mix_attn_go(cudaStream_t st, const void* q, int ldq, int n, const Mi
 
 }  // namespace
 
-void launch_qk_rms_append(cudaStream_t st, bool bf16, void* qkv, int ld, int n, const MixAttnShape& s, const RowState& rs) {
+// The form a launch takes: tensor cores for a prompt portion of a bf16 model whose sizes allow it.
+static bool mix_attn_use_tc(bool bf16, int n, const MixAttnShape& s, const RowState& rs, const MixAttnScratch& sc) {
+    return bf16 && !rs.separate() && n >= MIX_ATTN_TC_MIN_ROWS && sc.fold && mix_attn_tc_supported(s);
+}
+
+void launch_qk_rms_append(cudaStream_t st, bool bf16, void* qkv, int ld, int n, const MixAttnShape& s, const RowState& rs, const MixAttnScratch& sc) {
     if (n <= 0) return;
+    if (mix_attn_use_tc(bf16, n, s, rs, sc)) return launch_qk_fold_append(st, qkv, ld, n, s, rs, sc.fold);
     const unsigned grid = (unsigned)(((size_t)n * (s.heads + 2 * s.kv_heads) + 7) / 8);
     g_kernel_launches++;
     if (bf16) k_qk_rms_append<__nv_bfloat16><<<grid, 256, 0, st>>>((__nv_bfloat16*)qkv, ld, n, s, rs);
@@ -186,16 +192,18 @@ void launch_qk_rms_append(cudaStream_t st, bool bf16, void* qkv, int ld, int n, 
 
 bool mix_attn_supported(const MixAttnShape& s) { return mix_attn_smem(s, 1) <= MA_SMEM_MAX; }
 
-size_t mix_attn_partial_floats(const MixAttnShape& s, int max_rows) {
-    // rows x splits is largest with one query per CTA: splits <= (target + rows - 1) / rows, up to 4 queries per CTA
-    return (size_t)4 * (MA_TARGET_CTAS + max_rows) * s.heads * s.vdim;
+void mix_attn_scratch(const MixAttnShape& s, bool bf16, int max_rows, size_t* partial_floats, size_t* fold_bytes) {
+    // rows x splits: splits <= (target + CTAs - 1) / CTAs with up to 4 queries per CTA
+    *partial_floats = (size_t)4 * (MA_TARGET_CTAS + max_rows) * s.heads * s.vdim;
+    *fold_bytes = bf16 && mix_attn_tc_supported(s) ? (size_t)max_rows * s.heads * s.kv_heads * s.dim * 2 : 0;
 }
 
-cudaError_t launch_mix_attn(cudaStream_t st, bool bf16, const void* q, int ldq, int n, const MixAttnShape& s, const RowState& rs, void* out,
-                            int ldo, float* partial, int max_seq, uint32_t* err) {
+cudaError_t launch_mix_attn(cudaStream_t st, bool bf16, const void* qkv, int ld, int n, const MixAttnShape& s, const RowState& rs, void* out,
+                            int ldo, const MixAttnScratch& sc, int max_seq) {
     if (n <= 0) return cudaSuccess;
-    return bf16 ? mix_attn_go<__nv_bfloat16>(st, q, ldq, n, s, rs, out, ldo, partial, max_seq)
-                : mix_attn_go<float>(st, q, ldq, n, s, rs, out, ldo, partial, max_seq);
+    if (mix_attn_use_tc(bf16, n, s, rs, sc)) return launch_mix_attn_tc(st, sc.fold, n, s, rs, out, ldo, sc.err);
+    return bf16 ? mix_attn_go<__nv_bfloat16>(st, qkv, ld, n, s, rs, out, ldo, sc.partial, max_seq)
+                : mix_attn_go<float>(st, qkv, ld, n, s, rs, out, ldo, sc.partial, max_seq);
 }
 
 }  // namespace wick

@@ -21,6 +21,7 @@ const SOURCES: &[&str] = &[
     "kernels_dense.cu",
     "gemm_bf16.cu",
     "kernels_mixattn.cu",
+    "attn_mix_tc.cu",
     "kernels_delta.cu",
     "hybrid_ops.cu",
     "hybrid.cu",
