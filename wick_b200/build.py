@@ -17,7 +17,7 @@ _HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(_HERE, "csrc")
 LIB_PATH = os.path.join(_HERE, "libwick_cuda.so")
 SOURCES = ["kernels_basic.cu", "kernels_gemv.cu", "kernels_attn.cu", "kernels_q6k.cu", "kernels_batch.cu", "kernels_sample.cu", "tp_comm.cu", "decode_mega.cu", "gemm_tc.cu", "argmax_noalloc.cu",
-           "kernels_hyper.cu", "kernels_dense.cu", "gemm_bf16.cu", "kernels_mixattn.cu", "attn_mix_tc.cu", "kernels_delta.cu", "hybrid_ops.cu", "hybrid.cu", "wick_cuda.cu"]
+           "kernels_hyper.cu", "kernels_dense.cu", "gemm_bf16.cu", "kernels_mixattn.cu", "attn_mix_tc.cu", "kernels_delta.cu", "delta_chunk.cu", "hybrid_ops.cu", "hybrid.cu", "wick_cuda.cu"]
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",

@@ -222,10 +222,14 @@ struct Step {
             DeltaPrepArgs a;
             a.p = hm.proj; a.ldp = hm.ldp; a.off_b = L.off_b; a.a = hm.a; a.lda = hm.lda;
             a.conv_w = L.conv_w; a.A_log = L.A_log; a.dt_bias = L.dt_bias; a.n = n;
-            launch_delta_prep(st, hm.bf16, a, L.delta, rs, hm.work);
-            mark(PC_SHORTCONV);
-            launch_delta_scan(st, n, L.delta, rs, hm.work);
-            launch_delta_out(st, hm.bf16, n, L.delta, hm.work.o, L.out_norm, hm.gate, hm.ldg, hm.mixed, hm.ldm);
+            if (rs.separate()) {
+                launch_delta_step(st, hm.bf16, a, L.delta, rs, L.out_norm, hm.gate, hm.ldg, hm.mixed, hm.ldm);
+            } else {
+                launch_delta_prep(st, hm.bf16, a, L.delta, rs, hm.work);
+                mark(PC_SHORTCONV);
+                launch_delta_scan(st, n, L.delta, rs, hm.work);
+                launch_delta_out(st, hm.bf16, n, L.delta, hm.work.o, L.out_norm, hm.gate, hm.ldg, hm.mixed, hm.ldm);
+            }
             mark(PC_RECURRENCE);
         }
         W_TRY(dense(L.o, hm.mixed, hm.ldm, hm.y, hm.ldw, true));
@@ -356,7 +360,7 @@ int32_t nositar_build(wick_cuda_model* m, const JsonValue& config, const SafeTen
     hm.layers.resize(c.n_layers);
     m->layers.resize(c.n_layers);
     int ldp = 8, ldm = 8, ldf = 8, lda = 8, ldg = 8;
-    size_t partial = 0, fold = 0, wq = 0, wv = 0, wg = 0, wb = 0, wk = 0;
+    size_t partial = 0, fold = 0, wq = 0, wv = 0, wg = 0, wb = 0, wk = 0, wr = 0;
     for (uint32_t i = 0; i < c.n_layers; i++) {
         const JsonValue& lc = list.items[i];
         HybridLayer& L = hm.layers[i];
@@ -386,6 +390,7 @@ int32_t nositar_build(wick_cuda_model* m, const JsonValue& config, const SafeTen
             wv = std::max(wv, (size_t)s.heads * s.vdim);
             wb = std::max(wb, (size_t)s.heads);
             wk = std::max(wk, (size_t)s.kv_heads);
+            wr = std::max(wr, delta_record_floats(s, m->max_chunk));
             c.n_heads = std::max<uint32_t>(c.n_heads, s.heads);
             c.conv_kernel_size = std::max<uint32_t>(c.conv_kernel_size, s.taps);
         } else {
@@ -441,6 +446,7 @@ int32_t nositar_build(wick_cuda_model* m, const JsonValue& config, const SafeTen
     W_TRY(dev_alloc(m, &hm.work.beta, N * wb));
     W_TRY(dev_alloc(m, &hm.work.kq, N * wk));
     W_TRY(dev_alloc(m, &hm.work.o, N * wv));
+    W_TRY(dev_alloc(m, &hm.work.rec, wr));
     W_TRY(dev_alloc(m, &hm.rows_dev, N));
     W_TRY(dev_alloc(m, &m->tc_err, 1));
     CU_TRY(cudaMemset(m->tc_err, 0, 4));

@@ -118,6 +118,7 @@ bool mix_attn_supported(const MixAttnShape& s);
 // v rows appended to the caches (act [pos][kv_heads*dim], [pos][kv_heads*vdim]); q back in place or, where the tensor-core form
 // follows, folded into sc.fold.
 void launch_qk_rms_append(cudaStream_t st, bool bf16, void* qkv, int ld, int n, const MixAttnShape& s, const RowState& rs, const MixAttnScratch& sc);
+// (For separate rows the decode kernel does this itself where the sizes allow it, and this launches nothing.)
 // out act [n][ldo] (heads*vdim), after launch_qk_rms_append of the same rows.
 cudaError_t launch_mix_attn(cudaStream_t st, bool bf16, const void* qkv, int ld, int n, const MixAttnShape& s, const RowState& rs, void* out,
                             int ldo, const MixAttnScratch& sc, int max_seq);
@@ -145,7 +146,12 @@ struct DeltaWork {
     float* beta = nullptr;             // [n][H]
     float* kq = nullptr;               // [n][G] k . q
     float* o = nullptr;                // [n][H*vdim] read-outs
+    float* rec = nullptr;              // chunk records of the prompt form, delta_record_floats(); replaces q, k, g, beta, kq
 };
+// Portions of at least this many tokens of one sequence take the prompt form (delta_chunk.cu), DELTA_CHUNK tokens at a time.
+constexpr int DELTA_CHUNK = 8;
+constexpr int DELTA_CHUNK_MIN_ROWS = 8;
+size_t delta_record_floats(const DeltaShape& s, int n);
 struct DeltaPrepArgs {
     const void* p = nullptr;  // act [n][ldp]: the q | k | v channels at 0.., the beta logits at off_b
     int ldp = 0, off_b = 0;
@@ -158,9 +164,38 @@ struct DeltaPrepArgs {
 void launch_delta_prep(cudaStream_t st, bool bf16, const DeltaPrepArgs& a, const DeltaShape& s, const RowState& rs, const DeltaWork& w);
 // The recurrence: n tokens of one sequence, or one token of each row; state in s0 / p0.
 void launch_delta_scan(cudaStream_t st, int n, const DeltaShape& s, const RowState& rs, const DeltaWork& w);
+// The two steps of the prompt form (called by the launchers above).
+void launch_delta_chunk_prep(cudaStream_t st, bool bf16, const DeltaPrepArgs& a, const DeltaShape& s, const RowState& rs, const DeltaWork& w);
+void launch_delta_chunk_scan(cudaStream_t st, int n, const DeltaShape& s, const RowState& rs, const DeltaWork& w);
 // out act [n][ldo] = rms(o) * norm * sigmoid(gate), gate f32 [n][ldg]
 void launch_delta_out(cudaStream_t st, bool bf16, int n, const DeltaShape& s, const float* o, const float* norm, const float* gate, int ldg,
                       void* out, int ldo);
+
+// One decode token per row: convolutions, decays, the recurrence and the gated norm in one launch (state s0 / p0 and s1 / p1).
+void launch_delta_step(cudaStream_t st, bool bf16, const DeltaPrepArgs& a, const DeltaShape& s, const RowState& rs, const float* norm,
+                       const float* gate, int ldg, void* out, int ldo);
+
+// ── launches that may start before their predecessor has finished ──────────
+// The kernels of a decode step are launched with programmatic stream serialisation: a kernel is brought up while the one before
+// it still runs, touches nothing but weights, and calls pdl_wait() before it reads or writes anything else.  Every kernel
+// launched this way must call pdl_wait() (it is what keeps the whole chain ordered).
+template <class... P, class... A>
+inline cudaError_t launch_pdl(void (*kernel)(P...), dim3 grid, dim3 block, size_t smem, cudaStream_t st, A&&... args) {
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid;
+    cfg.blockDim = block;
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = st;
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = 1;
+    return cudaLaunchKernelEx(&cfg, kernel, P(args)...);
+}
+__device__ __forceinline__ void pdl_launch_next() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
+__device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
+__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
 
 // ── shared device helpers ──────────────────────────────────────────────────
 __device__ __forceinline__ float act_f(float v) { return v; }

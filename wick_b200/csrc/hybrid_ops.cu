@@ -141,9 +141,9 @@ int32_t wick_cuda_channel_delta(int32_t compute, const void* proj_dev, uint32_t 
     const size_t qf = (size_t)n * kv_heads * s.dimp(), gf = (size_t)n * heads * s.dimp(), vf = round_up((int)(heads * vdim), 4) * (size_t)n;
     const size_t bf = round_up((int)heads, 4) * (size_t)n;
     Scratch work;
-    CU_TRY(work.get(st, (2 * qf + gf + 2 * vf + 2 * bf) * 4));
+    CU_TRY(work.get(st, (2 * qf + gf + 2 * vf + 2 * bf + delta_record_floats(s, (int)n)) * 4));
     DeltaWork w;
-    w.q = (float*)work.p; w.k = w.q + qf; w.g = w.k + qf; w.v = w.g + gf; w.o = w.v + vf; w.beta = w.o + vf; w.kq = w.beta + bf;
+    w.q = (float*)work.p; w.k = w.q + qf; w.g = w.k + qf; w.v = w.g + gf; w.o = w.v + vf; w.beta = w.o + vf; w.kq = w.beta + bf; w.rec = w.kq + bf;
     RowState rs;
     rs.s0 = state_dev; rs.s1 = conv_state_dev;
     DeltaPrepArgs a;

@@ -1,3 +1,4 @@
+// Decode rows and short portions of the gated delta rule (prompts: delta_chunk.cu).
 // The gated delta rule with one decay per head and key channel (f32 throughout, as the state is):
 //     S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
 // k_delta_prep   short causal convolutions + silu, unit q and k, decays and step sizes: one warp per (token, group of
@@ -217,6 +218,162 @@ void scan_go(cudaStream_t st, int n, const DeltaShape& s, const RowState& rs, co
     k_delta_scan<R4><<<grid, SCAN_THREADS, smem, st>>>(n, s, rs, sep, w);
 }
 
+// ── one decode token per row ───────────────────────────────────────────────
+// A CTA owns a key head of a row and the heads that use it: convolutions and decays (a thread per channel), unit q and k (one
+// warp), the state's columns (eight lanes each, as above), the gated norm (a warp per head).
+template <class T, int R4, int TAPS>
+__global__ void __launch_bounds__(1024) k_delta_step(const __grid_constant__ DeltaPrepArgs a, const __grid_constant__ DeltaShape s,
+                                                    const __grid_constant__ RowState rs, const float* __restrict__ norm, const float* __restrict__ gate,
+                                                    int ldg, T* __restrict__ out, int ldo) {
+    extern __shared__ __align__(16) float sm[];
+    constexpr int DP = 32 * R4;
+    const int G = s.kv_heads, H = s.heads, D = s.dim, E = s.vdim, rep = H / G, kh = blockIdx.x, j = blockIdx.y, h0 = kh * rep;
+    const int tid = threadIdx.x, nt = blockDim.x, lane = tid & 31, warp = tid >> 5, C = s.channels();
+    const int taps = TAPS > 0 ? TAPS : s.taps;
+    float *q = sm, *k = q + DP, *g = k + DP, *v = g + rep * DP, *o = v + rep * E, *beta = o + rep * E, *kq = beta + rep;
+    pdl_launch_next();
+    pdl_wait();
+    float* state = (float*)rs.st0(j) + (size_t)h0 * E * DP;
+    float* cs = (float*)rs.st1(j);
+    const T* p = (const T*)a.p + (size_t)j * a.ldp;
+    const int convs = 2 * DP + rep * E;
+    for (int i = tid; i < convs + rep * DP + rep; i += nt) {
+        if (i < convs) {
+            int ch = -1;
+            if (i < DP) ch = i < D ? kh * D + i : -1;
+            else if (i < 2 * DP) ch = i - DP < D ? (G + kh) * D + i - DP : -1;
+            else ch = 2 * G * D + h0 * E + i - 2 * DP;
+            float y = 0.0f;
+            if (ch >= 0) {
+                const float* w = a.conv_w + (size_t)ch * taps;
+                const float cur = act_f(p[ch]);
+                if constexpr (TAPS > 0) {
+                    float x[TAPS], wt[TAPS];
+#pragma unroll
+                    for (int t = 0; t < TAPS; t++) {
+                        x[t] = t < TAPS - 1 ? cs[(size_t)t * C + ch] : cur;
+                        wt[t] = w[t];
+                    }
+#pragma unroll
+                    for (int t = 0; t < TAPS; t++) y = fmaf(wt[t], x[t], y);
+#pragma unroll
+                    for (int t = 0; t < TAPS - 1; t++) cs[(size_t)t * C + ch] = x[t + 1];
+                } else {
+                    for (int t = 0; t < taps; t++) {
+                        const float x = t < taps - 1 ? cs[(size_t)t * C + ch] : cur;
+                        y = fmaf(w[t], x, y);
+                        if (t > 0) cs[(size_t)(t - 1) * C + ch] = x;
+                    }
+                }
+                y = silu_f(y);
+            }
+            (i < DP ? q[i] : i < 2 * DP ? k[i - DP] : v[i - 2 * DP]) = y;
+        } else if (i < convs + rep * DP) {
+            const int r = (i - convs) / DP, c = (i - convs) % DP, h = h0 + r;
+            float x = 1.0f;
+            if (c < D) {
+                const float z = a.a[(size_t)j * a.lda + h * D + c] + a.dt_bias[h * D + c];
+                x = expf(-expf(a.A_log[h]) * (fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z)))));
+            }
+            g[r * DP + c] = x;
+        } else {
+            const int r = i - convs - rep * DP;
+            beta[r] = sigmoid_f(act_f(p[a.off_b + h0 + r]));
+        }
+    }
+    __syncthreads();
+    if (warp == 0) {
+        float qq = 0.0f, kk = 0.0f, qk = 0.0f;
+#pragma unroll
+        for (int r = 0; r < R4; r++) {
+            const float a0 = q[r * 32 + lane], b0 = k[r * 32 + lane];
+            qq = fmaf(a0, a0, qq);
+            kk = fmaf(b0, b0, kk);
+            qk = fmaf(a0, b0, qk);
+        }
+        qq = warp_sum(qq);
+        kk = warp_sum(kk);
+        qk = warp_sum(qk);
+        const float qs = 1.0f / sqrtf((float)D) / sqrtf(qq + 1e-6f), ks = 1.0f / sqrtf(kk + 1e-6f);
+#pragma unroll
+        for (int r = 0; r < R4; r++) {
+            q[r * 32 + lane] *= qs;
+            k[r * 32 + lane] *= ks;
+        }
+        if (lane == 0) *kq = qk * qs * ks;
+    }
+    __syncthreads();
+    const int l8 = tid & 7, cols = rep * E;
+    for (int c0 = 0; c0 < cols; c0 += nt / 8) {
+        const int c = c0 + (tid >> 3), r_ = min(c, cols - 1) / E;
+        float* sp = state + (size_t)min(c, cols - 1) * DP;
+        float S[R4][4], r1 = 0.0f, r2 = 0.0f;
+        float4 k4[R4];
+#pragma unroll
+        for (int r = 0; r < R4; r++) {
+            const float4 x = *reinterpret_cast<const float4*>(sp + 32 * r + 4 * l8);
+            S[r][0] = x.x; S[r][1] = x.y; S[r][2] = x.z; S[r][3] = x.w;
+        }
+#pragma unroll
+        for (int r = 0; r < R4; r++) {
+            const float4 q4 = *reinterpret_cast<const float4*>(q + 32 * r + 4 * l8), g4 = *reinterpret_cast<const float4*>(g + r_ * DP + 32 * r + 4 * l8);
+            k4[r] = *reinterpret_cast<const float4*>(k + 32 * r + 4 * l8);
+            S[r][0] *= g4.x; S[r][1] *= g4.y; S[r][2] *= g4.z; S[r][3] *= g4.w;
+            r1 = fmaf(S[r][0], k4[r].x, r1); r2 = fmaf(S[r][0], q4.x, r2);
+            r1 = fmaf(S[r][1], k4[r].y, r1); r2 = fmaf(S[r][1], q4.y, r2);
+            r1 = fmaf(S[r][2], k4[r].z, r1); r2 = fmaf(S[r][2], q4.z, r2);
+            r1 = fmaf(S[r][3], k4[r].w, r1); r2 = fmaf(S[r][3], q4.w, r2);
+        }
+#pragma unroll
+        for (int x = 4; x > 0; x >>= 1) {
+            r1 += __shfl_xor_sync(0xffffffffu, r1, x);
+            r2 += __shfl_xor_sync(0xffffffffu, r2, x);
+        }
+        if (c < cols) {
+            const float u = beta[r_] * (v[c] - r1);
+            if (l8 == 0) o[c] = fmaf(*kq, u, r2);
+#pragma unroll
+            for (int r = 0; r < R4; r++)
+                *reinterpret_cast<float4*>(sp + 32 * r + 4 * l8) = make_float4(fmaf(k4[r].x, u, S[r][0]), fmaf(k4[r].y, u, S[r][1]),
+                                                                              fmaf(k4[r].z, u, S[r][2]), fmaf(k4[r].w, u, S[r][3]));
+        }
+    }
+    __syncthreads();
+    for (int r = warp; r < rep; r += nt / 32) {
+        float ss = 0.0f;
+        for (int i = lane; i < E; i += 32) ss = fmaf(o[r * E + i], o[r * E + i], ss);
+        const float rr = 1.0f / sqrtf(warp_sum(ss) / (float)E + s.eps);
+        for (int i = lane; i < E; i += 32)
+            out[(size_t)j * ldo + (h0 + r) * E + i] = f_act<T>(o[r * E + i] * rr * norm[i] * sigmoid_f(gate[(size_t)j * ldg + (h0 + r) * E + i]));
+    }
+}
+
+template <class T, int R4>
+void step_go(cudaStream_t st, const DeltaPrepArgs& a, const DeltaShape& s, const RowState& rs, const float* norm, const float* gate, int ldg, T* out,
+             int ldo) {
+    const int rep = s.heads / s.kv_heads, cols = rep * s.vdim;
+    const dim3 grid(s.kv_heads, a.n), block((unsigned)std::min(1024, std::max(128, round_up(cols * 8, 128))));
+    const size_t smem = ((size_t)(2 + rep) * 32 * R4 + 2 * cols + rep + 4) * 4;
+    auto k = s.taps == 4 ? k_delta_step<T, R4, 4> : k_delta_step<T, R4, 0>;
+    if (smem > 40 * 1024) cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    launch_pdl(k, grid, block, smem, st, a, s, rs, norm, gate, ldg, out, ldo);
+}
+
+template <class T>
+void step_any(cudaStream_t st, const DeltaPrepArgs& a, const DeltaShape& s, const RowState& rs, const float* norm, const float* gate, int ldg, T* out,
+              int ldo) {
+    switch (s.dimp() / 32) {
+        case 1: return step_go<T, 1>(st, a, s, rs, norm, gate, ldg, out, ldo);
+        case 2: return step_go<T, 2>(st, a, s, rs, norm, gate, ldg, out, ldo);
+        case 3: return step_go<T, 3>(st, a, s, rs, norm, gate, ldg, out, ldo);
+        case 4: return step_go<T, 4>(st, a, s, rs, norm, gate, ldg, out, ldo);
+        case 5: return step_go<T, 5>(st, a, s, rs, norm, gate, ldg, out, ldo);
+        case 6: return step_go<T, 6>(st, a, s, rs, norm, gate, ldg, out, ldo);
+        case 7: return step_go<T, 7>(st, a, s, rs, norm, gate, ldg, out, ldo);
+        default: return step_go<T, 8>(st, a, s, rs, norm, gate, ldg, out, ldo);
+    }
+}
+
 // ── output ─────────────────────────────────────────────────────────────────
 template <class T>
 __global__ void __launch_bounds__(256) k_delta_out(int n, int H, int E, float eps, const float* __restrict__ o, const float* __restrict__ norm,
@@ -235,14 +392,19 @@ __global__ void __launch_bounds__(256) k_delta_out(int n, int H, int E, float ep
 
 }  // namespace
 
+static bool use_chunks(int n, const RowState& rs, const DeltaWork& w) { return !rs.separate() && n >= DELTA_CHUNK_MIN_ROWS && w.rec; }
+
 void launch_delta_prep(cudaStream_t st, bool bf16, const DeltaPrepArgs& a, const DeltaShape& s, const RowState& rs, const DeltaWork& w) {
     if (a.n <= 0) return;
     const bool sep = rs.separate();
     const size_t units = (size_t)a.n * (s.kv_heads + 2 * s.heads);
     const unsigned grid = (unsigned)((units + PREP_WARPS - 1) / PREP_WARPS);
-    g_kernel_launches++;
-    if (bf16) k_delta_prep<__nv_bfloat16><<<grid, PREP_WARPS * 32, 0, st>>>(a, s, rs, sep, w);
-    else k_delta_prep<float><<<grid, PREP_WARPS * 32, 0, st>>>(a, s, rs, sep, w);
+    if (use_chunks(a.n, rs, w)) launch_delta_chunk_prep(st, bf16, a, s, rs, w);
+    else {
+        g_kernel_launches++;
+        if (bf16) k_delta_prep<__nv_bfloat16><<<grid, PREP_WARPS * 32, 0, st>>>(a, s, rs, sep, w);
+        else k_delta_prep<float><<<grid, PREP_WARPS * 32, 0, st>>>(a, s, rs, sep, w);
+    }
     if (!sep && s.taps > 1) {
         const int C = s.channels();
         g_kernel_launches++;
@@ -253,6 +415,7 @@ void launch_delta_prep(cudaStream_t st, bool bf16, const DeltaPrepArgs& a, const
 
 void launch_delta_scan(cudaStream_t st, int n, const DeltaShape& s, const RowState& rs, const DeltaWork& w) {
     if (n <= 0) return;
+    if (use_chunks(n, rs, w)) return launch_delta_chunk_scan(st, n, s, rs, w);
     g_kernel_launches++;
     switch (s.dimp() / 32) {
         case 1: return scan_go<1>(st, n, s, rs, w);
@@ -264,6 +427,14 @@ void launch_delta_scan(cudaStream_t st, int n, const DeltaShape& s, const RowSta
         case 7: return scan_go<7>(st, n, s, rs, w);
         default: return scan_go<8>(st, n, s, rs, w);
     }
+}
+
+void launch_delta_step(cudaStream_t st, bool bf16, const DeltaPrepArgs& a, const DeltaShape& s, const RowState& rs, const float* norm,
+                       const float* gate, int ldg, void* out, int ldo) {
+    if (a.n <= 0) return;
+    g_kernel_launches++;
+    if (bf16) step_any(st, a, s, rs, norm, gate, ldg, (__nv_bfloat16*)out, ldo);
+    else step_any(st, a, s, rs, norm, gate, ldg, (float*)out, ldo);
 }
 
 void launch_delta_out(cudaStream_t st, bool bf16, int n, const DeltaShape& s, const float* o, const float* norm, const float* gate, int ldg,

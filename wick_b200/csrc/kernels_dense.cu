@@ -1,6 +1,6 @@
 // Dense bfloat16 matrices times f32 or bfloat16 activation rows.
-//   k_dense_rows  up to DENSE_ROWS_MAX rows (decode): a warp streams R weight rows with 16-byte loads, every loaded weight
-//                 feeds all the activation rows.  HBM-bound: the weight bytes once.
+//   k_dense_rows  up to DENSE_ROWS_MAX rows (decode): a warp (or several, over parts of k) streams R weight rows with 16-byte
+//                 loads, every loaded weight feeds all the activation rows.  HBM-bound: the weight bytes once.
 //   k_dense_simt  any number of rows, f32 multiply-adds on the CUDA cores: prompts of f32 models (bf16 models use gemm_bf16.cu).
 // Both accumulate in f32 and share the epilogues: plain store, activation(gate) * up, soft cap.
 #include "hybrid_kernels.cuh"
@@ -17,13 +17,15 @@ __device__ __forceinline__ void dense_store(const DenseCall& c, const DenseJob& 
 }
 
 constexpr int ROWS_WARPS = 4;
+constexpr int ROWS_TARGET_WARPS = 148 * 20;
 
-// NB activation rows, R weight rows (of each matrix when gated) per warp.
-template <class T, class O, int NB, int R, bool GATED>
+// NB activation rows, R weight rows (of each matrix when gated) per unit of WK warps, which split the columns of k.
+template <class T, class O, int NB, int R, bool GATED, int WK>
 __global__ void __launch_bounds__(ROWS_WARPS * 32) k_dense_rows(const __grid_constant__ DenseCall c) {
     constexpr int M = GATED ? 2 : 1;
-    const int lane = threadIdx.x & 31;
-    int unit = blockIdx.x * ROWS_WARPS + (threadIdx.x >> 5);
+    __shared__ float red[ROWS_WARPS][M * R * NB];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, part = warp % WK;
+    int unit = (blockIdx.x * ROWS_WARPS + warp) / WK;
     int ji = 0;
     if (!GATED && c.count == 2) {
         const int units0 = (c.job[0].w.m + R - 1) / R;
@@ -33,14 +35,18 @@ __global__ void __launch_bounds__(ROWS_WARPS * 32) k_dense_rows(const __grid_con
         }
     }
     const DenseJob& j = c.job[ji];
-    const int m = j.w.m, ld = j.w.ld, row0 = unit * R;
-    if (row0 >= m) return;
+    const int m = j.w.m, ld = j.w.ld, row0 = unit * R, k0 = (part * 32 + lane) * 8;
     const __nv_bfloat16* wp[M][R];
 #pragma unroll
     for (int q = 0; q < M; q++)
 #pragma unroll
-        for (int r = 0; r < R; r++)  // a row past the end repeats the last one and is not stored
+        for (int r = 0; r < R; r++) {  // a row past the end repeats the last one and is not stored
             wp[q][r] = c.job[ji + q].w.w + (size_t)min(row0 + r, m - 1) * ld;
+            for (int k = k0; k < ld; k += WK * 256)
+                if ((lane & 7) == 0) prefetch_l2(wp[q][r] + k);  // a 128-byte line per eight lanes
+        }
+    pdl_launch_next();
+    pdl_wait();
     float acc[M][R][NB];
 #pragma unroll
     for (int q = 0; q < M; q++)
@@ -50,7 +56,7 @@ __global__ void __launch_bounds__(ROWS_WARPS * 32) k_dense_rows(const __grid_con
             for (int b = 0; b < NB; b++) acc[q][r][b] = 0.0f;
     const T* x = (const T*)j.x;
 #pragma unroll 4
-    for (int k = lane * 8; k < ld; k += 256) {
+    for (int k = k0; k < ld; k += WK * 256) {
         uint4 wv[M][R];
 #pragma unroll
         for (int q = 0; q < M; q++)
@@ -72,30 +78,55 @@ __global__ void __launch_bounds__(ROWS_WARPS * 32) k_dense_rows(const __grid_con
         }
     }
 #pragma unroll
-    for (int r = 0; r < R; r++)
+    for (int q = 0; q < M; q++)
 #pragma unroll
-        for (int b = 0; b < NB; b++) {
-            const float v = warp_sum(acc[0][r][b]);
-            const float u = GATED ? warp_sum(acc[M - 1][r][b]) : 0.0f;
-            if (lane == 0 && row0 + r < m && b < c.n) dense_store<T, O>(c, j, b, row0 + r, v, u);
+        for (int r = 0; r < R; r++)
+#pragma unroll
+            for (int b = 0; b < NB; b++) {
+                const float v = warp_sum(acc[q][r][b]);
+                if (lane == 0) red[warp][(q * R + r) * NB + b] = v;
+            }
+    if constexpr (WK > 1) __syncthreads();
+    else __syncwarp();
+    if (part == 0)
+        for (int i = lane; i < R * NB; i += 32) {
+            const int r = i / NB, b = i % NB;
+            float v = 0.0f, u = 0.0f;
+#pragma unroll
+            for (int p = 0; p < WK; p++) {
+                v += red[warp + p][i];
+                if (GATED) u += red[warp + p][R * NB + i];
+            }
+            if (row0 + r < m && b < c.n) dense_store<T, O>(c, j, b, row0 + r, v, u);
         }
 }
 
-template <class T, class O, int NB, int R>
+template <class T, class O, int NB, int R, bool GATED>
+void dense_rows_wk(cudaStream_t st, const DenseCall& c) {
+    int units = (c.job[0].w.m + R - 1) / R, ld = c.job[0].w.ld;
+    if (!GATED && c.count == 2) {
+        units += (c.job[1].w.m + R - 1) / R;
+        ld = std::max(ld, c.job[1].w.ld);
+    }
+    const int wk = units >= ROWS_TARGET_WARPS || ld <= 256 ? 1 : units * 2 >= ROWS_TARGET_WARPS || ld <= 512 ? 2 : 4;
+    const dim3 grid((unsigned)((units * wk + ROWS_WARPS - 1) / ROWS_WARPS)), block(ROWS_WARPS * 32);
+    if (wk == 1) launch_pdl(k_dense_rows<T, O, NB, R, GATED, 1>, grid, block, 0, st, c);
+    else if (wk == 2) launch_pdl(k_dense_rows<T, O, NB, R, GATED, 2>, grid, block, 0, st, c);
+    else launch_pdl(k_dense_rows<T, O, NB, R, GATED, 4>, grid, block, 0, st, c);
+}
+
+template <class T, class O, int NB>
 void dense_rows_go(cudaStream_t st, const DenseCall& c) {
-    int units = (c.job[0].w.m + R - 1) / R;
-    if (!c.gated && c.count == 2) units += (c.job[1].w.m + R - 1) / R;
-    const unsigned grid = (unsigned)((units + ROWS_WARPS - 1) / ROWS_WARPS);
-    if (c.gated) k_dense_rows<T, O, NB, (R > 1 ? R / 2 : 1), true><<<(unsigned)(((c.job[0].w.m + (R > 1 ? R / 2 : 1) - 1) / (R > 1 ? R / 2 : 1) + ROWS_WARPS - 1) / ROWS_WARPS), ROWS_WARPS * 32, 0, st>>>(c);
-    else k_dense_rows<T, O, NB, R, false><<<grid, ROWS_WARPS * 32, 0, st>>>(c);
+    if (c.gated) dense_rows_wk<T, O, NB, 1, true>(st, c);
+    else dense_rows_wk<T, O, NB, 2, false>(st, c);
 }
 
 template <class T, class O>
 void dense_rows_n(cudaStream_t st, const DenseCall& c) {
-    if (c.n == 1) dense_rows_go<T, O, 1, 2>(st, c);
-    else if (c.n == 2) dense_rows_go<T, O, 2, 2>(st, c);
-    else if (c.n <= 4) dense_rows_go<T, O, 4, 2>(st, c);
-    else dense_rows_go<T, O, 8, 2>(st, c);
+    if (c.n == 1) dense_rows_go<T, O, 1>(st, c);
+    else if (c.n == 2) dense_rows_go<T, O, 2>(st, c);
+    else if (c.n <= 4) dense_rows_go<T, O, 4>(st, c);
+    else dense_rows_go<T, O, 8>(st, c);
 }
 
 // ── f32 tile kernel ────────────────────────────────────────────────────────

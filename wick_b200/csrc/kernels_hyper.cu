@@ -16,13 +16,16 @@ __global__ void __launch_bounds__(HYPER_THREADS) k_hyper_norm(HyperArgs a) {
     __shared__ float prm[HYPER_MAX_STREAMS * (HYPER_MAX_STREAMS + 2)];
     constexpr int SM = S_ ? S_ : HYPER_MAX_STREAMS;
     const int S = S_ ? S_ : a.S, W = a.W, tid = threadIdx.x;
-    const int row = blockIdx.x, src = a.rows ? a.rows[row] : row;
+    const int row = blockIdx.x;
     const bool init = a.embed != nullptr || a.frames != nullptr;
+    pdl_launch_next();
     float* mix = prm;
     float* w_out = prm + S * S;
     float* w_in = w_out + S;
     for (int i = tid; i < S * S + 2 * S; i += HYPER_THREADS)
         prm[i] = i < S * S ? (a.y ? a.mix[i] : 0.0f) : i < S * S + S ? (a.y ? a.out[i - S * S] : 0.0f) : (a.in ? a.in[i - S * S - S] : 1.0f);
+    pdl_wait();
+    const int src = a.rows ? a.rows[row] : row;
     __syncthreads();
     float* x = a.x + (size_t)src * S * W;
     const __nv_bfloat16* e = nullptr;
@@ -127,10 +130,10 @@ static void hyper_v(cudaStream_t st, const HyperArgs& a) {
     const size_t smem = (size_t)round_up(a.W, 4) * 4;
     if (a.W % 4 == 0 && (!a.y || a.ldy % 4 == 0)) {
         if (smem > 40 * 1024) cudaFuncSetAttribute(k_hyper_norm<T, S, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        k_hyper_norm<T, S, 4><<<a.n, HYPER_THREADS, smem, st>>>(a);
+        launch_pdl(k_hyper_norm<T, S, 4>, dim3(a.n), dim3(HYPER_THREADS), smem, st, a);
     } else {
         if (smem > 40 * 1024) cudaFuncSetAttribute(k_hyper_norm<T, S, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        k_hyper_norm<T, S, 1><<<a.n, HYPER_THREADS, smem, st>>>(a);
+        launch_pdl(k_hyper_norm<T, S, 1>, dim3(a.n), dim3(HYPER_THREADS), smem, st, a);
     }
 }
 

@@ -5,7 +5,7 @@
 // key) pair, so a CTA works on all heads of its queries; there is no normaliser, so partial sums over disjoint keys simply
 // add up, and the keys of a query tile can be split over CTAs.
 //
-// k_mix_attn computes in f32 on the CUDA cores and takes any sizes; prompts of bf16 models go to attn_mix_tc.cu.
+// k_mix_attn computes in f32 on the CUDA cores and takes any sizes; k_mix_attn_step is the decode form; prompts of bf16 models go to attn_mix_tc.cu.
 #include "hybrid_kernels.cuh"
 
 namespace wick {
@@ -135,15 +135,148 @@ __global__ void __launch_bounds__(MA_THREADS) k_mix_attn(const T* __restrict__ q
     }
 }
 
-// Adds the key splits of a row in split order.
+// ── one decode token per row ───────────────────────────────────────────────
+// CTA (split, row): the key tiles split, + gridDim.x, ... of the row's visible keys, all heads.  Normalises q itself; the CTA
+// whose tile holds the row's own position also normalises k and appends the k and v rows first.  Sizes multiples of 8.
+constexpr int MS_KT = 16, MS_CHUNKS = 4;  // keys per tile; 8-column pieces of the output per thread
+
+template <class T>
+__device__ __forceinline__ void rms_head(const T* __restrict__ src, int d, float eps, int lane, float* dst_f, T* dst_t) {
+    float ss = 0.0f;
+    for (int i = lane; i < d; i += 32) {
+        const float v = act_f(src[i]);
+        ss = fmaf(v, v, ss);
+    }
+    const float r = 1.0f / sqrtf(warp_sum(ss) / (float)d + eps);
+    for (int i = lane; i < d; i += 32) {
+        const T v = f_act<T>(act_f(src[i]) * r);  // q is rounded like the cached k
+        if (dst_t) dst_t[i] = v;
+        else dst_f[i] = act_f(v);
+    }
+}
+
+template <class T>
+__global__ void __launch_bounds__(MA_THREADS) k_mix_attn_step(const T* __restrict__ qkv, int ld, const __grid_constant__ MixAttnShape s,
+                                                              const __grid_constant__ RowState rs, T* __restrict__ out, int ldo,
+                                                              float* __restrict__ partial) {
+    extern __shared__ __align__(16) float sm[];
+    const int H = s.heads, G = s.kv_heads, D = s.dim, E = s.vdim, rep = H / G, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, j = blockIdx.y;
+    float* qs = sm;                          // [H*D]
+    float* sc = qs + H * D;                  // [H][KT] scores
+    float* wt = sc + H * MS_KT;              // [H][KT] weights
+    float* tk = wt + H * MS_KT;              // [H][H]
+    float* bi = tk + H * H;                  // [H]
+    float* red = bi + round_up(H, 4);        // [groups][H*E] at the end
+    for (int i = tid; i < H * H; i += MA_THREADS) tk[i] = s.talk ? s.talk[i] : (i / H == i % H ? 1.0f : 0.0f);
+    for (int i = tid; i < H; i += MA_THREADS) bi[i] = s.bias ? s.bias[i] : 0.0f;
+    pdl_launch_next();
+    pdl_wait();
+    const int pos = rs.pos(j);
+    const KeyRange kr(s, pos, pos);
+    T* kc = (T*)rs.st0(j);
+    T* vc = (T*)rs.st1(j);
+    const T* row = qkv + (size_t)j * ld;
+    const int tiles = (kr.count + MS_KT - 1) / MS_KT;
+    const bool newest = (tiles - 1) % (int)gridDim.x == (int)blockIdx.x;
+    for (int seg = warp; seg < H + (newest ? G : 0); seg += MA_THREADS / 32)
+        rms_head<T>(row + seg * D, D, s.eps, lane, qs + seg * D, seg < H ? nullptr : kc + (size_t)pos * G * D + (seg - H) * D);
+    if (newest)
+        for (int i = tid; i < G * E; i += MA_THREADS) vc[(size_t)pos * G * E + i] = row[(H + G) * D + i];
+    __syncthreads();
+    const int CH = H * E / 8, groups = CH >= MA_THREADS ? 1 : MA_THREADS / CH;  // key groups of the weighted sum
+    float acc[MS_CHUNKS][8] = {};
+    for (int t = blockIdx.x; t < tiles; t += gridDim.x) {
+        const int t0 = t * MS_KT, cnt = min(MS_KT, kr.count - t0);
+        for (int i = tid; i < H * MS_KT; i += MA_THREADS) {
+            const int key = i % MS_KT, h = i / MS_KT;
+            float a0 = 0.0f, a1 = 0.0f;
+            if (key < cnt) {
+                const T* kp = kc + ((size_t)kr.key(t0 + key) * G + h / rep) * D;
+                const float* qp = qs + h * D;
+#pragma unroll 8
+                for (int d = 0; d < D; d += 8) {
+                    float kv[8];
+                    load8(kp + d, kv);
+#pragma unroll
+                    for (int x = 0; x < 8; x += 2) {
+                        a0 = fmaf(qp[d + x], kv[x], a0);
+                        a1 = fmaf(qp[d + x + 1], kv[x + 1], a1);
+                    }
+                }
+            }
+            sc[i] = (a0 + a1) * s.scale;
+        }
+        __syncthreads();
+        for (int i = tid; i < H * MS_KT; i += MA_THREADS) {
+            const int key = i % MS_KT, h = i / MS_KT;
+            float z = bi[h];
+            for (int g = 0; g < H; g++) z = fmaf(tk[h * H + g], sc[g * MS_KT + key], z);
+            wt[i] = key < cnt ? sigmoid_f(z) : 0.0f;  // every key of the range is visible to the row's position
+        }
+        __syncthreads();
+#pragma unroll
+        for (int x = 0; x < MS_CHUNKS; x++) {
+            const int c = groups > 1 ? (x == 0 && tid < CH * groups ? tid % CH : CH) : tid + x * MA_THREADS, grp = groups > 1 ? tid / CH : 0;
+            if (c < CH) {
+                const int h = c * 8 / E;
+                const T* vp = vc + (size_t)(h / rep) * E + c * 8 % E;
+#pragma unroll 4
+                for (int key = grp; key < cnt; key += groups) {
+                    float v[8];
+                    load8(vp + (size_t)kr.key(t0 + key) * G * E, v);
+                    const float w = wt[h * MS_KT + key];
+#pragma unroll
+                    for (int e = 0; e < 8; e++) acc[x][e] = fmaf(w, v[e], acc[x][e]);
+                }
+            }
+        }
+        __syncthreads();
+    }
+    if (groups > 1) {
+        if (tid < CH * groups)
+#pragma unroll
+            for (int e = 0; e < 8; e++) red[tid * 8 + e] = acc[0][e];
+        __syncthreads();
+        if (tid < CH)
+#pragma unroll
+            for (int e = 0; e < 8; e++) {
+                float a = red[tid * 8 + e];
+                for (int g = 1; g < groups; g++) a += red[(g * CH + tid) * 8 + e];
+                acc[0][e] = a;
+            }
+    }
+    const size_t base = ((size_t)j * gridDim.x + blockIdx.x) * H * E;
+#pragma unroll
+    for (int x = 0; x < MS_CHUNKS; x++) {
+        const int c = tid + x * MA_THREADS;
+        if (c < CH)
+#pragma unroll
+            for (int e = 0; e < 8; e++) {
+                if (partial) partial[base + c * 8 + e] = acc[x][e];
+                else out[(size_t)j * ldo + c * 8 + e] = f_act<T>(acc[x][e]);
+            }
+    }
+}
+
+// Adds the key splits of a row in a fixed order: 32 columns per CTA, eight strided runs of splits, then the runs.
 template <class T>
 __global__ void __launch_bounds__(256) k_mix_attn_sum(const float* __restrict__ partial, int splits, int width, T* __restrict__ out, int ldo) {
-    const int c = blockIdx.x * 256 + threadIdx.x;
-    if (c >= width) return;
+    __shared__ float red[8][32];
+    const int lane = threadIdx.x & 31, run = threadIdx.x >> 5, c = blockIdx.x * 32 + lane;
+    pdl_launch_next();
+    pdl_wait();
     const float* p = partial + (size_t)blockIdx.y * splits * width + c;
     float a = 0.0f;
-    for (int i = 0; i < splits; i++) a += p[(size_t)i * width];
-    out[(size_t)blockIdx.y * ldo + c] = f_act<T>(a);
+    if (c < width)
+#pragma unroll 8
+        for (int i = run; i < splits; i += 8) a += p[(size_t)i * width];
+    red[run][lane] = a;
+    __syncthreads();
+    if (run == 0 && c < width) {
+#pragma unroll
+        for (int i = 1; i < 8; i++) a += red[i][lane];
+        out[(size_t)blockIdx.y * ldo + c] = f_act<T>(a);
+    }
 }
 
 size_t mix_attn_smem(const MixAttnShape& s, int qt) {
@@ -169,7 +302,32 @@ cudaError_t mix_attn_go(cudaStream_t st, const void* q, int ldq, int n, const Mi
     if (splits > 1) {
         const int width = s.heads * s.vdim;
         g_kernel_launches++;
-        k_mix_attn_sum<T><<<dim3((width + 255) / 256, n), 256, 0, st>>>(partial, splits, width, (T*)out, ldo);
+        launch_pdl(k_mix_attn_sum<T>, dim3((width + 31) / 32, n), dim3(256), 0, st, partial, splits, width, (T*)out, ldo);
+    }
+    return cudaGetLastError();
+}
+
+size_t mix_attn_step_smem(const MixAttnShape& s) {
+    const int ch = s.heads * s.vdim / 8, groups = ch >= MA_THREADS || ch == 0 ? 1 : MA_THREADS / ch;
+    return ((size_t)s.heads * (s.dim + 2 * MS_KT) + (size_t)s.heads * s.heads + round_up(s.heads, 4) + (groups > 1 ? (size_t)groups * ch * 8 : 0)) * 4;
+}
+bool mix_attn_step_supported(const MixAttnShape& s) {
+    return s.dim % 8 == 0 && s.vdim % 8 == 0 && s.heads * s.vdim <= 8 * MS_CHUNKS * MA_THREADS && mix_attn_step_smem(s) <= MA_SMEM_MAX;
+}
+
+template <class T>
+cudaError_t mix_attn_step_go(cudaStream_t st, const void* qkv, int ld, int n, const MixAttnShape& s, const RowState& rs, void* out, int ldo,
+                             float* partial, int max_seq) {
+    const size_t smem = mix_attn_step_smem(s);
+    if (smem > 40 * 1024) cudaFuncSetAttribute(k_mix_attn_step<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    const int tiles = (s.seen(max_seq) + MS_KT - 1) / MS_KT + 1;
+    const int splits = std::max(1, std::min({MA_TARGET_CTAS / n, tiles, 2 * MA_MAX_SPLIT}));
+    g_kernel_launches++;
+    launch_pdl(k_mix_attn_step<T>, dim3(splits, n), dim3(MA_THREADS), smem, st, (const T*)qkv, ld, s, rs, (T*)out, ldo, splits > 1 ? partial : nullptr);
+    if (splits > 1) {
+        const int width = s.heads * s.vdim;
+        g_kernel_launches++;
+        launch_pdl(k_mix_attn_sum<T>, dim3((width + 31) / 32, n), dim3(256), 0, st, partial, splits, width, (T*)out, ldo);
     }
     return cudaGetLastError();
 }
@@ -182,7 +340,7 @@ static bool mix_attn_use_tc(bool bf16, int n, const MixAttnShape& s, const RowSt
 }
 
 void launch_qk_rms_append(cudaStream_t st, bool bf16, void* qkv, int ld, int n, const MixAttnShape& s, const RowState& rs, const MixAttnScratch& sc) {
-    if (n <= 0) return;
+    if (n <= 0 || (rs.separate() && mix_attn_step_supported(s))) return;  // k_mix_attn_step does it itself
     if (mix_attn_use_tc(bf16, n, s, rs, sc)) return launch_qk_fold_append(st, qkv, ld, n, s, rs, sc.fold);
     const unsigned grid = (unsigned)(((size_t)n * (s.heads + 2 * s.kv_heads) + 7) / 8);
     g_kernel_launches++;
@@ -201,6 +359,9 @@ void mix_attn_scratch(const MixAttnShape& s, bool bf16, int max_rows, size_t* pa
 cudaError_t launch_mix_attn(cudaStream_t st, bool bf16, const void* qkv, int ld, int n, const MixAttnShape& s, const RowState& rs, void* out,
                             int ldo, const MixAttnScratch& sc, int max_seq) {
     if (n <= 0) return cudaSuccess;
+    if (rs.separate() && mix_attn_step_supported(s))
+        return bf16 ? mix_attn_step_go<__nv_bfloat16>(st, qkv, ld, n, s, rs, out, ldo, sc.partial, max_seq)
+                    : mix_attn_step_go<float>(st, qkv, ld, n, s, rs, out, ldo, sc.partial, max_seq);
     if (mix_attn_use_tc(bf16, n, s, rs, sc)) return launch_mix_attn_tc(st, sc.fold, n, s, rs, out, ldo, sc.err);
     return bf16 ? mix_attn_go<__nv_bfloat16>(st, qkv, ld, n, s, rs, out, ldo, sc.partial, max_seq)
                 : mix_attn_go<float>(st, qkv, ld, n, s, rs, out, ldo, sc.partial, max_seq);

@@ -23,6 +23,7 @@ const SOURCES: &[&str] = &[
     "kernels_mixattn.cu",
     "attn_mix_tc.cu",
     "kernels_delta.cu",
+    "delta_chunk.cu",
     "hybrid_ops.cu",
     "hybrid.cu",
     "wick_cuda.cu",
