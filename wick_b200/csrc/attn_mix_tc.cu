@@ -9,7 +9,7 @@
 // k_mix_attn_tc: a CTA owns 128 queries of one head and walks over tiles of 64 keys (the kept first keys, then the window):
 //   warp 0  lane 0: TMA - q' once (or chunk by chunk when it does not fit), K in chunks of 64 columns, V
 //   warp 1  lane 0: S = q' K^T into one of two tensor-memory buffers, then O += P V of the tile before
-//   warps 2..9    : P = sigmoid(S + bias) masked to the visible keys, rounded to bf16 into shared memory in the 128B-swizzled
+//   warps 2..17   : P = sigmoid(S + bias) masked to the visible keys, rounded to bf16 into shared memory in the 128B-swizzled
 //                   layout of the MMA's A operand; at the end O -> out
 // There is no normaliser and no running maximum, so O is accumulated in tensor memory from the first tile to the last.
 // Every wait is bounded.  Bound: tensor pipe (G-fold redundant score products) and the special-function unit (exp and
@@ -21,7 +21,7 @@ namespace wick {
 
 namespace {
 
-constexpr int MT_Q = 128, MT_K = 64, MT_EPI_WARPS = 8, MT_THREADS = 32 * (2 + MT_EPI_WARPS);
+constexpr int MT_Q = 128, MT_K = 64, MT_EPI_WARPS = 16, MT_THREADS = 32 * (2 + MT_EPI_WARPS);
 constexpr int MT_QCHUNK = MT_Q * 64 * 2, MT_KCHUNK = MT_K * 64 * 2, MT_P = MT_Q * MT_K * 2;
 constexpr int MT_SMEM_MAX = 226 * 1024;
 
@@ -168,8 +168,10 @@ __global__ void __launch_bounds__(MT_THREADS, 1) k_mix_attn_tc(const __grid_cons
             if (ok) umma_commit(smem_u32(o_full));
         }
     } else {
-        const int quarter = warp & 3, half = (warp - 2) >> 2, r = quarter * 32 + lane, qi = p0 + r;
-        const float bias = p.bias ? p.bias[h] : 0.0f;
+        // lanes 32 (warp % 4).. and 16 of the 64 key columns
+        const int quarter = warp & 3, part = (warp - 2) >> 2, r = quarter * 32 + lane, qi = p0 + r;
+        constexpr float LOG2E = 1.4426950408889634f;
+        const float bias = p.bias ? p.bias[h] * -LOG2E : 0.0f;
         const uint32_t lane_base = (uint32_t)(quarter * 32) << 16;
         bool ok = true;
         for (int t = 0; t < tiles; t++) {
@@ -177,8 +179,8 @@ __global__ void __launch_bounds__(MT_THREADS, 1) k_mix_attn_tc(const __grid_cons
             ok = mbar_wait_bounded(smem_u32(&s_full[b]), (t >> 1) & 1, abort, p.err, 28);
             if (!ok) break;
             tc_fence_after();
-            int32_t v[32];
-            tmem_ld32(tmem + lane_base + b * MT_K + half * 32, v);
+            int32_t v[16];
+            tmem_ld16(tmem + lane_base + b * MT_K + part * 16, v);
             tmem_ld_wait();
             tc_fence_before();
             __syncwarp();
@@ -186,30 +188,35 @@ __global__ void __launch_bounds__(MT_THREADS, 1) k_mix_attn_tc(const __grid_cons
             const bool kept = t < kept_tiles;
             const int key0 = (kept ? t * MT_K : lo + (t - kept_tiles) * MT_K);
             const bool all = kept ? key0 + MT_K <= ns : key0 + MT_K - 1 <= p0 && (p.size <= 0 || p1 - key0 < p.size);
-            uint32_t w[16];
+            // sigmoid(z) = 1 / (1 + 2^(-z log2 e))
+            float f[16];
 #pragma unroll
-            for (int c = 0; c < 32; c += 2) {
-                float f[2];
+            for (int c = 0; c < 16; c++) {
+                float e;
+                asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(fmaf(__int_as_float(v[c]), -LOG2E, bias)));
+                asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(f[c]) : "f"(1.0f + e));
+            }
+            if (!all) {
 #pragma unroll
-                for (int e = 0; e < 2; e++) {
-                    const float z = __int_as_float(v[c + e]) + bias;
-                    f[e] = __fdividef(1.0f, 1.0f + __expf(-z));
-                    if (!all) {
-                        const int j = key0 + half * 32 + c + e;
-                        const bool vis = kept ? j < ns : j <= qi && (p.size <= 0 || qi - j < p.size || j < p.keep);
-                        f[e] = vis ? f[e] : 0.0f;
-                    }
+                for (int c = 0; c < 16; c++) {
+                    const int j = key0 + part * 16 + c;
+                    const bool vis = kept ? j < ns : j <= qi && (p.size <= 0 || qi - j < p.size || j < p.keep);
+                    f[c] = vis ? f[c] : 0.0f;
                 }
-                const __nv_bfloat162 q = __floats2bfloat162_rn(f[0], f[1]);
-                w[c >> 1] = *reinterpret_cast<const uint32_t*>(&q);
+            }
+            uint32_t w[8];
+#pragma unroll
+            for (int c = 0; c < 8; c++) {
+                const __nv_bfloat162 q = __floats2bfloat162_rn(f[2 * c], f[2 * c + 1]);
+                w[c] = *reinterpret_cast<const uint32_t*>(&q);
             }
             const int pb = t % p.p_bufs;
             ok = mbar_wait_bounded(smem_u32(&p_empty[pb]), ((t / p.p_bufs) & 1) ^ 1, abort, p.err, 29);
             if (!ok) break;
             uint8_t* prow = sp + pb * MT_P + r * 128;
 #pragma unroll
-            for (int c = 0; c < 4; c++)
-                *reinterpret_cast<uint4*>(prow + (((half * 4 + c) ^ (r & 7)) << 4)) = make_uint4(w[4 * c], w[4 * c + 1], w[4 * c + 2], w[4 * c + 3]);
+            for (int c = 0; c < 2; c++)
+                *reinterpret_cast<uint4*>(prow + (((part * 2 + c) ^ (r & 7)) << 4)) = make_uint4(w[4 * c], w[4 * c + 1], w[4 * c + 2], w[4 * c + 3]);
             asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
             __syncwarp();
             if (lane == 0) mbar_arrive(smem_u32(&p_full[pb]));
@@ -217,7 +224,7 @@ __global__ void __launch_bounds__(MT_THREADS, 1) k_mix_attn_tc(const __grid_cons
         if (ok && mbar_wait_bounded(smem_u32(o_full), 0, abort, p.err, 30)) {
             tc_fence_after();
             __nv_bfloat16* dst = p.out + (size_t)(row0 + r) * p.ldo + h * p.vdim;
-            for (int c0 = half * 16; c0 < p.vdim; c0 += 32) {
+            for (int c0 = part * 16; c0 < p.vdim; c0 += 64) {
                 int32_t v[16];
                 tmem_ld16(tmem_o + lane_base + c0, v);
                 tmem_ld_wait();

@@ -56,6 +56,32 @@ struct Lanes {
 
 __host__ __device__ constexpr int rec_floats(int dp) { return (3 * DC + 1) * dp + 2 * DC * DC + DC; }
 
+// silu after a convolution: an activation, so a bfloat16 model takes the fast forms
+template <class T>
+__device__ __forceinline__ float conv_act(float z) {
+    if constexpr (sizeof(T) == 2) return __fdividef(z, 1.0f + __expf(-z));
+    else return silu_f(z);
+}
+
+// One halving exchange of a transposing sum over the lanes: N values become N / 2, lanes with bit OFF keep the upper half.
+template <int N, int OFF>
+__device__ __forceinline__ void halve(float* x, int lane) {
+    const bool up = lane & OFF;
+#pragma unroll
+    for (int i = 0; i < N / 2; i++) {
+        const float keep = up ? x[i + N / 2] : x[i], send = up ? x[i] : x[i + N / 2];
+        x[i] = keep + __shfl_xor_sync(0xffffffffu, send, OFF);
+    }
+}
+// Sums of 16 values over the lanes: lane l returns that of value l / 2.
+__device__ __forceinline__ float sum16(float* x, int lane) {
+    halve<16, 16>(x, lane);
+    halve<8, 8>(x, lane);
+    halve<4, 4>(x, lane);
+    halve<2, 2>(x, lane);
+    return x[0] + __shfl_xor_sync(0xffffffffu, x[0], 1);
+}
+
 // Convolution + silu of channel ch for the DC tokens from t0 on (tokens >= n: zero).
 template <class T, int TAPS>
 __device__ __forceinline__ void conv_run(const DeltaPrepArgs& a, const float* state, int C, int taps, int t0, int n, int ch, float* y) {
@@ -75,7 +101,7 @@ __device__ __forceinline__ void conv_run(const DeltaPrepArgs& a, const float* st
             float s = 0.0f;
 #pragma unroll
             for (int k = 0; k < TAPS; k++) s = fmaf(wt[k], x[i + k], s);
-            y[i] = t0 + i < n ? silu_f(s) : 0.0f;
+            y[i] = t0 + i < n ? conv_act<T>(s) : 0.0f;
         }
     } else {
 #pragma unroll
@@ -85,7 +111,7 @@ __device__ __forceinline__ void conv_run(const DeltaPrepArgs& a, const float* st
                 const int j = t0 + i - (taps - 1) + k;
                 s = fmaf(w[k], j >= n ? 0.0f : j >= 0 ? act_f(p[(size_t)j * a.ldp]) : state[(size_t)(taps - 1 + j) * C + ch], s);
             }
-            y[i] = t0 + i < n ? silu_f(s) : 0.0f;
+            y[i] = t0 + i < n ? conv_act<T>(s) : 0.0f;
         }
     }
 }
@@ -124,33 +150,38 @@ __global__ void __launch_bounds__(PREP_THREADS) k_delta_chunk_prep(const __grid_
 #pragma unroll
         for (int t = 0; t < DC; t++) k[t][r] = c < D ? y[t] : 0.0f;
     }
-    const float rate = expf(a.A_log[h]), qscale = 1.0f / sqrtf((float)D);
-    float beta[DC];
+    const float rate = expf(a.A_log[h]);
+    float x[2 * DC];
 #pragma unroll
     for (int t = 0; t < DC; t++) {
-        float qq = 0.0f, kk = 0.0f;
+        x[t] = x[DC + t] = 0.0f;
 #pragma unroll
         for (int r = 0; r < R; r++) {
-            qq = fmaf(q[t][r], q[t][r], qq);
-            kk = fmaf(k[t][r], k[t][r], kk);
+            x[t] = fmaf(q[t][r], q[t][r], x[t]);
+            x[DC + t] = fmaf(k[t][r], k[t][r], x[DC + t]);
         }
-        const float qs = qscale / sqrtf(warp_sum(qq) + 1e-6f), ks = 1.0f / sqrtf(warp_sum(kk) + 1e-6f);
-        const bool live = t0 + t < n;
+    }
+    // lane 2t: 1 / |q_t| dim^(1/2), lane 2 (DC + t): 1 / |k_t|
+    const float unit = (lane < 16 ? 1.0f / sqrtf((float)D) : 1.0f) / sqrtf(sum16(x, lane) + 1e-6f);
+    const int my_t = (lane >> 1) & 7;
+    const float beta = t0 + my_t < n ? sigmoid_f(act_f(((const T*)a.p)[(size_t)(t0 + my_t) * a.ldp + a.off_b + h])) : 0.0f;
+#pragma unroll
+    for (int t = 0; t < DC; t++) {
+        const float qs = __shfl_sync(0xffffffffu, unit, 2 * t), ks = __shfl_sync(0xffffffffu, unit, 2 * (DC + t));
 #pragma unroll
         for (int r = 0; r < R; r++) {
             q[t][r] *= qs;
             k[t][r] *= ks;
             const int c = Lanes<R>::channel(lane, r);
             g[t][r] = 1.0f;
-            if (live && c < D) {
+            if (t0 + t < n && c < D) {
                 const float z = a.a[(size_t)(t0 + t) * a.lda + h * D + c] + a.dt_bias[h * D + c];
                 g[t][r] = expf(-rate * (fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z)))));
             }
         }
-        beta[t] = live ? sigmoid_f(act_f(((const T*)a.p)[(size_t)(t0 + t) * a.ldp + a.off_b + h])) : 0.0f;
     }
     float* o = rec + ((size_t)h * ((n + DC - 1) / DC) + chunk) * rec_floats(DP);
-    // k_i . D(j,i) k_j and q_i . D(j,i) k_j, the row products of every (j, i)
+    // beta_i k_i . D(j,i) k_j (stored by columns j) and q_i . D(j,i) k_j (by rows i), zero where token i does not see token j
     float* ab = o + (3 * DC + 1) * DP;
 #pragma unroll
     for (int j = 0; j < DC; j++) {
@@ -158,48 +189,39 @@ __global__ void __launch_bounds__(PREP_THREADS) k_delta_chunk_prep(const __grid_
 #pragma unroll
         for (int r = 0; r < R; r++) w[r] = k[j][r];
 #pragma unroll
-        for (int i = j; i < DC; i++) {
-            float ka = 0.0f, qa = 0.0f;
+        for (int i = 0; i < DC; i++) {
+            x[i] = x[DC + i] = 0.0f;
+            if (i < j) continue;
 #pragma unroll
             for (int r = 0; r < R; r++) {
-                if (i > j) w[r] *= g[i][r];
-                ka = fmaf(k[i][r], w[r], ka);
-                qa = fmaf(q[i][r], w[r], qa);
-            }
-            qa = warp_sum(qa);
-            if (i > j) ka = warp_sum(ka);
-            if (lane == 0) {
-                ab[i * DC + j] = i > j ? beta[i] * ka : 0.0f;
-                ab[DC * DC + i * DC + j] = qa;
+                if (i > j) {
+                    w[r] *= g[i][r];
+                    x[i] = fmaf(k[i][r], w[r], x[i]);
+                }
+                x[DC + i] = fmaf(q[i][r], w[r], x[DC + i]);
             }
         }
+        const float sum = sum16(x, lane) * (lane < 16 ? beta : 1.0f);
+        if ((lane & 1) == 0) ab[lane < 16 ? j * DC + my_t : DC * DC + my_t * DC + j] = sum;
         Lanes<R>::store(o + (2 * DC + j) * DP, lane, w);  // D(j,DC) k_j
     }
+    if (lane < 16 && (lane & 1) == 0) ab[2 * DC * DC + my_t] = beta;
     float cum[R];
 #pragma unroll
     for (int r = 0; r < R; r++) cum[r] = 1.0f;
 #pragma unroll
     for (int t = 0; t < DC; t++) {
-        float x[R], y[R];
+        float ck[R], cq[R];
 #pragma unroll
         for (int r = 0; r < R; r++) {
             cum[r] *= g[t][r];
-            x[r] = cum[r] * k[t][r];
-            y[r] = cum[r] * q[t][r];
+            ck[r] = cum[r] * k[t][r];
+            cq[r] = cum[r] * q[t][r];
         }
-        Lanes<R>::store(o + t * DP, lane, x);
-        Lanes<R>::store(o + (DC + t) * DP, lane, y);
+        Lanes<R>::store(o + t * DP, lane, ck);
+        Lanes<R>::store(o + (DC + t) * DP, lane, cq);
     }
     Lanes<R>::store(o + 3 * DC * DP, lane, cum);
-    if (lane < DC * (DC - 1) / 2) {  // the read-out of token i does not see later tokens
-        int i = 0, j = lane;
-        while (j >= DC - 1 - i) j -= DC - 1 - i++;
-        ab[DC * DC + i * DC + i + 1 + j] = 0.0f;
-        ab[i * DC + i + 1 + j] = 0.0f;
-    }
-#pragma unroll
-    for (int t = 0; t < DC; t++)
-        if (lane == t) ab[2 * DC * DC + t] = beta[t];
 }
 
 __device__ __forceinline__ void cp16(float* dst, const float* src) {
@@ -209,17 +231,6 @@ __device__ __forceinline__ void cp4(float* dst, const float* src) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
 
-// One halving exchange of a transposing sum over the lanes: N values become N / 2, lanes with bit OFF keep the upper half.
-template <int N, int OFF>
-__device__ __forceinline__ void halve(float* x, int lane) {
-    const bool up = lane & OFF;
-#pragma unroll
-    for (int i = 0; i < N / 2; i++) {
-        const float keep = up ? x[i + N / 2] : x[i], send = up ? x[i] : x[i + N / 2];
-        x[i] = keep + __shfl_xor_sync(0xffffffffu, send, OFF);
-    }
-}
-
 constexpr int SCAN_WARPS = 4, SCAN_RING = 3;
 
 // NC = 4 value channels per warp; lane = 4 * token + channel after the transposing sums.
@@ -227,7 +238,7 @@ template <int R>
 __global__ void __launch_bounds__(SCAN_WARPS * 32) k_delta_chunk_scan(int n, const __grid_constant__ DeltaShape s, float* __restrict__ state_all,
                                                                      const float* __restrict__ rec, const float* __restrict__ v, float* __restrict__ out) {
     constexpr int DP = 32 * R, REC = rec_floats(DP), NC = 4, COLS = NC * SCAN_WARPS, SLOT = REC + DC * COLS;
-    static_assert(DC * NC == 32 && REC % 4 == 0, "one (token, channel) pair per lane");
+    static_assert(DC == 8 && DC * NC == 32 && REC % 4 == 0, "one (token, channel) pair per lane");
     extern __shared__ __align__(16) float sm[];
     __shared__ __align__(16) float u_sh[SCAN_WARPS][DC][NC];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.y, H = s.heads, E = s.vdim;
@@ -283,19 +294,30 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) k_delta_chunk_scan(int n, con
         const float* A = rc + (3 * DC + 1) * DP;
         const float* B = A + DC * DC;
         const float rhs = A[2 * DC * DC + my_t] * (rc[REC + my_t * COLS + warp * NC + my_c] - xk[0]);
-        float u[DC];
+        float u[DC], bo[DC];
 #pragma unroll
         for (int t = 0; t < DC; t++) u[t] = __shfl_sync(0xffffffffu, rhs, t * 4 + my_c);
 #pragma unroll
-        for (int t = 1; t < DC; t++)
-#pragma unroll
-            for (int j = 0; j < t; j++) u[t] = fmaf(-A[t * DC + j], u[j], u[t]);
-        float o = xq[0], mine = u[0];
-#pragma unroll
-        for (int j = 0; j < DC; j++) {
-            o = fmaf(B[my_t * DC + j], u[j], o);
-            mine = my_t == j ? u[j] : mine;
+        for (int j = 0; j < DC; j += 4) {
+            const float4 t = *reinterpret_cast<const float4*>(B + my_t * DC + j);
+            bo[j] = t.x; bo[j + 1] = t.y; bo[j + 2] = t.z; bo[j + 3] = t.w;
         }
+        // forward substitution by columns: once u_j is known it leaves every later row
+#pragma unroll
+        for (int j = 0; j < DC - 1; j++) {
+            const float4 a0 = *reinterpret_cast<const float4*>(A + j * DC), a1 = *reinterpret_cast<const float4*>(A + j * DC + 4);
+            const float col[DC] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y, a1.z, a1.w};
+#pragma unroll
+            for (int t = j + 1; t < DC; t++) u[t] = fmaf(-col[t], u[j], u[t]);
+        }
+        float o = xq[0], o1 = 0.0f, mine = u[0];
+#pragma unroll
+        for (int j = 0; j < DC; j += 2) {
+            o = fmaf(bo[j], u[j], o);
+            o1 = fmaf(bo[j + 1], u[j + 1], o1);
+            mine = my_t == j ? u[j] : my_t == j + 1 ? u[j + 1] : mine;
+        }
+        o += o1;
         const int tok = ch * DC + my_t, col = c0 + warp * NC + my_c;
         if (tok < n && col < E) out[(size_t)tok * H * E + h * E + col] = o;
         u_sh[warp][my_t][my_c] = mine;

@@ -35,7 +35,9 @@ struct Loader {
     const SafeTensors& t;
 
     int32_t vec(const std::string& name, const std::vector<int64_t>& shape, float** out) const {
-        const SafeTensor& s = t.get(name, shape);
+        // (a single number may be stored with shape [] or [1])
+        const SafeTensor* one = shape.empty() ? t.find(name) : nullptr;
+        const SafeTensor& s = t.get(name, one && one->shape == std::vector<int64_t>{1} ? one->shape : shape);
         std::vector<float> host(s.elems());
         for (size_t i = 0; i < host.size(); i++) host[i] = bf16_to_f32(s.data + 2 * i);
         return put(host, out);
@@ -79,6 +81,13 @@ struct Loader {
         return (int)s->shape[0];
     }
 };
+
+// A mixer's mechanism: its name without the number that tells several sizes of one mechanism apart ("name", "name_2").
+std::string mechanism(const std::string& type) {
+    const size_t u = type.find_last_of('_');
+    if (u == std::string::npos || u + 1 == type.size() || type.find_first_not_of("0123456789", u + 1) != std::string::npos) return type;
+    return type.substr(0, u);
+}
 
 int32_t load_attention(const Loader& ld, const std::string& p, const JsonValue& mc, int width, HybridLayer* L, Layer* st, size_t act_bytes) {
     MixAttnShape& s = L->attn;
@@ -367,7 +376,8 @@ int32_t nositar_build(wick_cuda_model* m, const JsonValue& config, const SafeTen
         const std::string p = "l" + std::to_string(i) + ".";
         L.type = lc.at("type").str;
         const JsonValue& mc = lc.at("mixer");
-        if (L.type == "attention") {
+        const std::string kind = mechanism(L.type);
+        if (kind == "attention") {
             L.kind = MIX_ATTENTION;
             W_TRY(load_attention(ld, p + "mix.", mc, hm.width, &L, &m->layers[i], act_bytes));
             const MixAttnShape& s = L.attn;
@@ -378,7 +388,7 @@ int32_t nositar_build(wick_cuda_model* m, const JsonValue& config, const SafeTen
             fold = std::max(fold, fb);
             c.n_heads = std::max<uint32_t>(c.n_heads, s.heads);
             c.n_kv_heads = std::max<uint32_t>(c.n_kv_heads, s.kv_heads);
-        } else if (L.type == "channel_delta" || L.type.rfind("channel_delta_", 0) == 0) {  // one mechanism; the name numbers its size
+        } else if (kind == "channel_delta") {
             L.kind = MIX_DELTA;
             W_TRY(load_delta(ld, p + "mix.", mc, hm.width, &L, &m->layers[i]));
             const DeltaShape& s = L.delta;
@@ -400,8 +410,8 @@ int32_t nositar_build(wick_cuda_model* m, const JsonValue& config, const SafeTen
         W_TRY(ld.hyper(p, 1, hm.streams, &L.hc1));
         const JsonValue* mlp = lc.find("mlp");
         if (mlp && mlp->is_object()) {
-            const std::string kind = mlp->at("kind").str;
-            if (kind != "dense") return fail(WICK_CUDA_ERR_BAD_MODEL, "layer " + std::to_string(i) + ": unknown feed-forward kind " + kind);
+            const std::string ff_kind = mlp->at("kind").str;
+            if (ff_kind != "dense") return fail(WICK_CUDA_ERR_BAD_MODEL, "layer " + std::to_string(i) + ": unknown feed-forward kind " + ff_kind);
             const int ff = mlp->count("ff");
             L.has_ff = true;
             W_TRY(ld.matrix(p + "mlp.gate", ff, hm.width, &L.gate));

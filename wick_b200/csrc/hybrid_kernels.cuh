@@ -160,9 +160,10 @@ struct DeltaPrepArgs {
     const float *conv_w = nullptr, *A_log = nullptr, *dt_bias = nullptr;  // [channels][taps], [H], [H*dim]
     int n = 0;
 };
-// Short convolution + silu, unit q and k, decays and step sizes; advances the convolution state (s1 / p1).
+// Consecutive tokens of one sequence: short convolution + silu, unit q and k, decays and step sizes; advances the convolution
+// state (s1).
 void launch_delta_prep(cudaStream_t st, bool bf16, const DeltaPrepArgs& a, const DeltaShape& s, const RowState& rs, const DeltaWork& w);
-// The recurrence: n tokens of one sequence, or one token of each row; state in s0 / p0.
+// Their recurrence; state in s0.
 void launch_delta_scan(cudaStream_t st, int n, const DeltaShape& s, const RowState& rs, const DeltaWork& w);
 // The two steps of the prompt form (called by the launchers above).
 void launch_delta_chunk_prep(cudaStream_t st, bool bf16, const DeltaPrepArgs& a, const DeltaShape& s, const RowState& rs, const DeltaWork& w);

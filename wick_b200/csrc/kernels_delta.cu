@@ -1,14 +1,13 @@
-// Decode rows and short portions of the gated delta rule (prompts: delta_chunk.cu).
 // The gated delta rule with one decay per head and key channel (f32 throughout, as the state is):
 //     S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
-// k_delta_prep   short causal convolutions + silu, unit q and k, decays and step sizes: one warp per (token, group of
-//                channels that is normalised together).
-// k_delta_scan   the recurrence.  The columns of S (value channels) do not depend on each other: eight lanes hold one column,
-//                4 * R4 key channels each, in registers, from the first token of the launch to the last.  The read-out is
-//                folded into the same pass over the column, o = (diag(g) S)^T q + (k . q) u, so that a token costs one
-//                round of cross-lane sums; k . q comes from k_delta_prep.  A block of tokens' q, k, g rows is staged in shared
-//                memory with cp.async, one block ahead.
-// k_delta_out    RMS norm over the value channels of a head, gain, sigmoid gate.
+// for decode steps and portions of a few tokens (prompts: delta_chunk.cu).  The columns of S (value channels) do not depend on
+// each other: eight lanes hold one column, 4 * R4 key channels each.  The read-out is folded into the same pass over the
+// column, o = (diag(g) S)^T q + (k . q) u, so that a token costs one round of cross-lane sums.
+// k_delta_prep   short causal convolutions + silu, unit q and k, k . q, decays and step sizes of consecutive tokens: one warp
+//                per (token, group of channels that is normalised together).
+// k_delta_scan   their recurrence; the state stays in registers, q, k, g rows are staged in shared memory with cp.async.
+// k_delta_step   one decode token per row: all of it, and the gated norm, in one launch.
+// k_delta_out    RMS norm over the value channels of a head, gain, sigmoid gate (also after delta_chunk.cu).
 #include "hybrid_kernels.cuh"
 
 namespace wick {
@@ -19,10 +18,9 @@ namespace {
 constexpr int PREP_WARPS = 8;
 constexpr int PREP_REG = DELTA_MAX_DIM / 32;
 
-// Convolution of channel ch at row j followed by silu; `advance`: also moves the row's own state on (rows are separate
-// sequences then, and this lane owns the channel).
+// Convolution of channel ch at row j followed by silu.
 template <class T>
-__device__ __forceinline__ float conv_silu(const DeltaPrepArgs& a, const DeltaShape& s, float* state, int j, int ch, bool separate) {
+__device__ __forceinline__ float conv_silu(const DeltaPrepArgs& a, const DeltaShape& s, const float* state, int j, int ch) {
     const int t = s.taps, C = s.channels();
     const float* w = a.conv_w + (size_t)ch * t;
     const T* p = (const T*)a.p;
@@ -30,25 +28,20 @@ __device__ __forceinline__ float conv_silu(const DeltaPrepArgs& a, const DeltaSh
     float sum = 0.0f;
     for (int i = 0; i < t - 1; i++) {
         const int src = j - (t - 1 - i);  // row of the launch; negative: kept from before
-        float v;
-        if (separate) v = state[(size_t)i * C + ch];
-        else v = src >= 0 ? act_f(p[(size_t)src * a.ldp + ch]) : state[(size_t)(t - 1 + src) * C + ch];
+        const float v = src >= 0 ? act_f(p[(size_t)src * a.ldp + ch]) : state[(size_t)(t - 1 + src) * C + ch];
         sum = fmaf(w[i], v, sum);
-        if (separate && i > 0) state[(size_t)(i - 1) * C + ch] = v;
     }
-    if (separate && t > 1) state[(size_t)(t - 2) * C + ch] = cur;
     return silu_f(fmaf(w[t - 1], cur, sum));
 }
 
 template <class T>
 __global__ void __launch_bounds__(PREP_WARPS * 32) k_delta_prep(const __grid_constant__ DeltaPrepArgs a, const __grid_constant__ DeltaShape s,
-                                                               const __grid_constant__ RowState rs, bool separate, const __grid_constant__ DeltaWork w) {
+                                                               const float* __restrict__ state, const __grid_constant__ DeltaWork w) {
     const int lane = threadIdx.x & 31;
     const int seg_n = s.kv_heads + 2 * s.heads;
     const size_t unit = (size_t)blockIdx.x * PREP_WARPS + (threadIdx.x >> 5);
     if (unit >= (size_t)a.n * seg_n) return;
     const int j = (int)(unit / seg_n), seg = (int)(unit % seg_n);
-    float* state = (float*)rs.st1(separate ? j : 0);
     const int G = s.kv_heads, H = s.heads, D = s.dim, E = s.vdim, DP = s.dimp();
     if (seg < G) {  // q and k of key head `seg`
         float q[PREP_REG], k[PREP_REG], qq = 0.0f, kk = 0.0f, kq = 0.0f;
@@ -57,8 +50,8 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) k_delta_prep(const __grid_con
             const int i = r * 32 + lane;
             q[r] = k[r] = 0.0f;
             if (i < D) {
-                q[r] = conv_silu<T>(a, s, state, j, seg * D + i, separate);
-                k[r] = conv_silu<T>(a, s, state, j, (G + seg) * D + i, separate);
+                q[r] = conv_silu<T>(a, s, state, j, seg * D + i);
+                k[r] = conv_silu<T>(a, s, state, j, (G + seg) * D + i);
             }
             qq = fmaf(q[r], q[r], qq);
             kk = fmaf(k[r], k[r], kk);
@@ -79,7 +72,7 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) k_delta_prep(const __grid_con
         if (lane == 0) w.kq[(size_t)j * G + seg] = kq;
     } else if (seg < G + H) {  // v of head h
         const int h = seg - G;
-        for (int i = lane; i < E; i += 32) w.v[(size_t)j * H * E + h * E + i] = conv_silu<T>(a, s, state, j, 2 * G * D + h * E + i, separate);
+        for (int i = lane; i < E; i += 32) w.v[(size_t)j * H * E + h * E + i] = conv_silu<T>(a, s, state, j, 2 * G * D + h * E + i);
     } else {  // decays and step size of head h
         const int h = seg - G - H;
         const float rate = expf(a.A_log[h]);
@@ -124,15 +117,14 @@ __host__ __device__ constexpr int scan_tok_floats(int dp) { return 3 * dp + SCAN
 
 // R4 * 4 key channels per lane: dimp = 32 * R4.  Lane l of a column's eight holds channels 32 r + 4 l .. + 3.
 template <int R4>
-__global__ void __launch_bounds__(SCAN_THREADS) k_delta_scan(int n, const __grid_constant__ DeltaShape s, const __grid_constant__ RowState rs,
-                                                            bool separate, const __grid_constant__ DeltaWork w) {
+__global__ void __launch_bounds__(SCAN_THREADS) k_delta_scan(int nt, const __grid_constant__ DeltaShape s, float* __restrict__ state_all,
+                                                            const __grid_constant__ DeltaWork w) {
     extern __shared__ __align__(16) float sm[];
     constexpr int DP = 32 * R4, TOK = scan_tok_floats(DP);
     const int tid = threadIdx.x, l8 = tid & 7, col = tid >> 3;
     const int h = blockIdx.y, G = s.kv_heads, H = s.heads, E = s.vdim;
     const int kh = h / (H / G), c0 = blockIdx.x * SCAN_COLS, c = c0 + col;
-    const int row0 = separate ? blockIdx.z : 0, nt = separate ? 1 : n;
-    float* state = (float*)rs.st0(row0) + ((size_t)h * E + min(c, E - 1)) * DP;
+    float* state = state_all + ((size_t)h * E + min(c, E - 1)) * DP;
     float S[R4][4];
 #pragma unroll
     for (int r = 0; r < R4; r++) {
@@ -145,13 +137,13 @@ __global__ void __launch_bounds__(SCAN_THREADS) k_delta_scan(int n, const __grid
         constexpr int V4 = DP / 4;
         for (int i = tid; i < cnt * 3 * V4; i += SCAN_THREADS) {
             const int t = i / (3 * V4), q = i % (3 * V4), which = q / V4, x = q % V4;
-            const size_t row = (size_t)(row0 + t0 + t);
+            const size_t row = (size_t)(t0 + t);
             const float* src = which == 0 ? w.q + (row * G + kh) * DP : which == 1 ? w.k + (row * G + kh) * DP : w.g + (row * H + h) * DP;
             cp16(dst + t * TOK + which * DP + 4 * x, src + 4 * x);
         }
         for (int i = tid; i < cnt * (SCAN_COLS + 2); i += SCAN_THREADS) {
             const int t = i / (SCAN_COLS + 2), x = i % (SCAN_COLS + 2);
-            const size_t row = (size_t)(row0 + t0 + t);
+            const size_t row = (size_t)(t0 + t);
             if (x < SCAN_COLS) {
                 if (c0 + x < E) cp4(dst + t * TOK + 3 * DP + x, w.v + row * H * E + h * E + c0 + x);
             } else if (x == SCAN_COLS) {
@@ -200,7 +192,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) k_delta_scan(int n, const __grid
                 S[r][2] = fmaf(k4[r].z, u, S[r][2]);
                 S[r][3] = fmaf(k4[r].w, u, S[r][3]);
             }
-            if (l8 == 0 && c < E) w.o[(size_t)(row0 + t0 + t) * H * E + h * E + c] = out;
+            if (l8 == 0 && c < E) w.o[(size_t)(t0 + t) * H * E + h * E + c] = out;
         }
     }
     if (c < E)
@@ -211,11 +203,10 @@ __global__ void __launch_bounds__(SCAN_THREADS) k_delta_scan(int n, const __grid
 
 template <int R4>
 void scan_go(cudaStream_t st, int n, const DeltaShape& s, const RowState& rs, const DeltaWork& w) {
-    const bool sep = rs.separate();
-    const dim3 grid((s.vdim + SCAN_COLS - 1) / SCAN_COLS, s.heads, sep ? n : 1);
+    const dim3 grid((s.vdim + SCAN_COLS - 1) / SCAN_COLS, s.heads);
     const size_t smem = (size_t)2 * SCAN_TB * scan_tok_floats(32 * R4) * 4;
     if (smem > 48 * 1024) cudaFuncSetAttribute(k_delta_scan<R4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    k_delta_scan<R4><<<grid, SCAN_THREADS, smem, st>>>(n, s, rs, sep, w);
+    k_delta_scan<R4><<<grid, SCAN_THREADS, smem, st>>>(n, s, (float*)rs.s0, w);
 }
 
 // ── one decode token per row ───────────────────────────────────────────────
@@ -392,20 +383,19 @@ __global__ void __launch_bounds__(256) k_delta_out(int n, int H, int E, float ep
 
 }  // namespace
 
-static bool use_chunks(int n, const RowState& rs, const DeltaWork& w) { return !rs.separate() && n >= DELTA_CHUNK_MIN_ROWS && w.rec; }
+static bool use_chunks(int n, const DeltaWork& w) { return n >= DELTA_CHUNK_MIN_ROWS && w.rec; }
 
 void launch_delta_prep(cudaStream_t st, bool bf16, const DeltaPrepArgs& a, const DeltaShape& s, const RowState& rs, const DeltaWork& w) {
     if (a.n <= 0) return;
-    const bool sep = rs.separate();
     const size_t units = (size_t)a.n * (s.kv_heads + 2 * s.heads);
     const unsigned grid = (unsigned)((units + PREP_WARPS - 1) / PREP_WARPS);
-    if (use_chunks(a.n, rs, w)) launch_delta_chunk_prep(st, bf16, a, s, rs, w);
+    if (use_chunks(a.n, w)) launch_delta_chunk_prep(st, bf16, a, s, rs, w);
     else {
         g_kernel_launches++;
-        if (bf16) k_delta_prep<__nv_bfloat16><<<grid, PREP_WARPS * 32, 0, st>>>(a, s, rs, sep, w);
-        else k_delta_prep<float><<<grid, PREP_WARPS * 32, 0, st>>>(a, s, rs, sep, w);
+        if (bf16) k_delta_prep<__nv_bfloat16><<<grid, PREP_WARPS * 32, 0, st>>>(a, s, (const float*)rs.s1, w);
+        else k_delta_prep<float><<<grid, PREP_WARPS * 32, 0, st>>>(a, s, (const float*)rs.s1, w);
     }
-    if (!sep && s.taps > 1) {
+    if (s.taps > 1) {
         const int C = s.channels();
         g_kernel_launches++;
         if (bf16) k_delta_conv_state<__nv_bfloat16><<<(C + 255) / 256, 256, 0, st>>>((const __nv_bfloat16*)a.p, a.ldp, a.n, C, s.taps, (float*)rs.s1);
@@ -415,7 +405,7 @@ void launch_delta_prep(cudaStream_t st, bool bf16, const DeltaPrepArgs& a, const
 
 void launch_delta_scan(cudaStream_t st, int n, const DeltaShape& s, const RowState& rs, const DeltaWork& w) {
     if (n <= 0) return;
-    if (use_chunks(n, rs, w)) return launch_delta_chunk_scan(st, n, s, rs, w);
+    if (use_chunks(n, w)) return launch_delta_chunk_scan(st, n, s, rs, w);
     g_kernel_launches++;
     switch (s.dimp() / 32) {
         case 1: return scan_go<1>(st, n, s, rs, w);
