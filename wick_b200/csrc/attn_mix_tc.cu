@@ -310,16 +310,17 @@ bool mt_plan(const MixAttnShape& s, MtParams* p, size_t* smem) {
         p->q_resident = resident;
         const int q = resident ? p->chunks * MT_QCHUNK : 0, ks = MT_KCHUNK + (resident ? 0 : MT_QCHUNK), v = p->vboxes * MT_KCHUNK;
         const int tries[4][2] = {{2, 2}, {2, 1}, {1, 2}, {1, 1}};  // V stages, P buffers
-        for (const auto& t : tries) {
-            const int left = MT_SMEM_MAX - bars - q - t[0] * v - t[1] * MT_P;
-            const int want = resident ? 3 : 4;
-            if (left < want * ks) continue;
-            p->v_stages = t[0];
-            p->p_bufs = t[1];
-            p->k_stages = std::min(left / ks, p->chunks < 4 ? 6 : 8);
-            *smem = (size_t)q + t[0] * v + t[1] * MT_P + p->k_stages * ks + bars;
-            return true;
-        }
+        // enough K chunks in flight to cover a trip to L2 matter more than second V and P buffers
+        for (int want : {6, 3})
+            for (const auto& t : tries) {
+                const int left = MT_SMEM_MAX - bars - q - t[0] * v - t[1] * MT_P;
+                if (left < want * ks) continue;
+                p->v_stages = t[0];
+                p->p_bufs = t[1];
+                p->k_stages = std::min(left / ks, 8);
+                *smem = (size_t)q + t[0] * v + t[1] * MT_P + p->k_stages * ks + bars;
+                return true;
+            }
     }
     return false;
 }

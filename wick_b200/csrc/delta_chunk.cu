@@ -294,30 +294,19 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) k_delta_chunk_scan(int n, con
         const float* A = rc + (3 * DC + 1) * DP;
         const float* B = A + DC * DC;
         const float rhs = A[2 * DC * DC + my_t] * (rc[REC + my_t * COLS + warp * NC + my_c] - xk[0]);
-        float u[DC], bo[DC];
+        float u[DC];
 #pragma unroll
         for (int t = 0; t < DC; t++) u[t] = __shfl_sync(0xffffffffu, rhs, t * 4 + my_c);
 #pragma unroll
-        for (int j = 0; j < DC; j += 4) {
-            const float4 t = *reinterpret_cast<const float4*>(B + my_t * DC + j);
-            bo[j] = t.x; bo[j + 1] = t.y; bo[j + 2] = t.z; bo[j + 3] = t.w;
-        }
-        // forward substitution by columns: once u_j is known it leaves every later row
+        for (int t = 1; t < DC; t++)
 #pragma unroll
-        for (int j = 0; j < DC - 1; j++) {
-            const float4 a0 = *reinterpret_cast<const float4*>(A + j * DC), a1 = *reinterpret_cast<const float4*>(A + j * DC + 4);
-            const float col[DC] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y, a1.z, a1.w};
+            for (int j = 0; j < t; j++) u[t] = fmaf(-A[j * DC + t], u[j], u[t]);
+        float o = xq[0], mine = u[0];
 #pragma unroll
-            for (int t = j + 1; t < DC; t++) u[t] = fmaf(-col[t], u[j], u[t]);
+        for (int j = 0; j < DC; j++) {
+            o = fmaf(B[my_t * DC + j], u[j], o);
+            mine = my_t == j ? u[j] : mine;
         }
-        float o = xq[0], o1 = 0.0f, mine = u[0];
-#pragma unroll
-        for (int j = 0; j < DC; j += 2) {
-            o = fmaf(bo[j], u[j], o);
-            o1 = fmaf(bo[j + 1], u[j + 1], o1);
-            mine = my_t == j ? u[j] : my_t == j + 1 ? u[j + 1] : mine;
-        }
-        o += o1;
         const int tok = ch * DC + my_t, col = c0 + warp * NC + my_c;
         if (tok < n && col < E) out[(size_t)tok * H * E + h * E + col] = o;
         u_sh[warp][my_t][my_c] = mine;
