@@ -89,7 +89,7 @@ int32_t wick_cuda_model_create_from_file(const char* path, uint32_t context_size
 #define WICK_CUDA_COMPUTE_F32 2
 int32_t wick_cuda_model_create_from_path(const char* path, uint32_t context_size, int32_t device, int32_t compute,
                                          wick_cuda_model** out);
-/* Architecture name of the model file ("lfm2", "Nositar") and type name of a layer ("Attention", "GatedConv", or the
+/* Architecture name of the model file ("lfm2", "Nositar", "Novorax") and type name of a layer ("Attention", "GatedConv", or the
  * mixer's name in config.json); "" for a NULL handle or a layer that does not exist. */
 const char* wick_cuda_model_architecture(const wick_cuda_model* m);
 const char* wick_cuda_model_layer_type(const wick_cuda_model* m, uint32_t layer);
@@ -299,8 +299,8 @@ int32_t wick_cuda_argmax(const float* logits_dev, uint32_t count, uint32_t* out_
  * are read by dense and must be finite.  Device pointers, asynchronous on `stream`; dense and mix_attention synchronise it
  * to report expired device waits as WICK_CUDA_ERR_TIMEOUT. */
 
-/* y[n][m] = x[n][k] W[m][k]^T with bfloat16 W (pitch ldw = k rounded up to 8, padding zero).  w_up_dev (optional, same shape):
- * y = activation(W x) * (W_up x).  softcap > 0: y = softcap tanh(y / softcap).  y is act, or f32 when y_f32 != 0.  path: AUTO, or
+/* y[n][m] = activation(x[n][k] W[m][k]^T) with bfloat16 W (pitch ldw = k rounded up to 8, padding zero).  w_up_dev (optional,
+ * same shape): y = activation(W x) * (W_up x).  softcap > 0: y = softcap tanh(y / softcap).  y is act, or f32 when y_f32 != 0.  path: AUTO, or
  * one kernel: row streaming (n <= 8), CUDA-core f32, tcgen05 (bfloat16 only). */
 #define WICK_CUDA_DENSE_AUTO 0
 #define WICK_CUDA_DENSE_ROWS 1
@@ -308,6 +308,8 @@ int32_t wick_cuda_argmax(const float* logits_dev, uint32_t count, uint32_t* out_
 #define WICK_CUDA_DENSE_TENSOR 3
 #define WICK_CUDA_ACT_RELU 0
 #define WICK_CUDA_ACT_SILU 1
+#define WICK_CUDA_ACT_RELU2 2 /* the square of relu */
+#define WICK_CUDA_ACT_NONE 3
 int32_t wick_cuda_dense(int32_t compute, const void* w_dev, const void* w_up_dev, uint32_t m, uint32_t k, uint32_t ldw, const void* x_dev,
                         uint32_t ldx, uint32_t n, void* y_dev, uint32_t ldy, int32_t y_f32, int32_t activation, float softcap, int32_t path,
                         void* stream);

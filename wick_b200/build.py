@@ -8,6 +8,7 @@ from __future__ import annotations
 
 import fcntl
 import os
+import re
 import shutil
 import subprocess
 import sys
@@ -17,7 +18,7 @@ _HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(_HERE, "csrc")
 LIB_PATH = os.path.join(_HERE, "libwick_cuda.so")
 SOURCES = ["kernels_basic.cu", "kernels_gemv.cu", "kernels_attn.cu", "kernels_q6k.cu", "kernels_batch.cu", "kernels_sample.cu", "tp_comm.cu", "decode_mega.cu", "gemm_tc.cu", "argmax_noalloc.cu",
-           "kernels_hyper.cu", "kernels_dense.cu", "gemm_bf16.cu", "kernels_mixattn.cu", "attn_mix_tc.cu", "kernels_delta.cu", "delta_chunk.cu", "hybrid_ops.cu", "hybrid.cu", "wick_cuda.cu"]
+           "kernels_hyper.cu", "kernels_residual.cu", "kernels_dense.cu", "kernels_route.cu", "gemm_bf16.cu", "kernels_mixattn.cu", "attn_mix_tc.cu", "kernels_delta.cu", "delta_chunk.cu", "kernels_latent.cu", "kernels_memory.cu", "hybrid_ops.cu", "hybrid_load.cu", "hybrid.cu", "wick_cuda.cu"]
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
@@ -33,18 +34,32 @@ def _nvcc() -> str:
     raise RuntimeError("nvcc not found")
 
 
-def _inputs() -> tuple[dict, float]:
-    """Modification time of every source, and the newest of what all of them may include (headers, this file)."""
-    srcs = {f: os.path.getmtime(os.path.join(CSRC, f)) for f in SOURCES}
-    shared = [os.path.join(CSRC, f) for f in os.listdir(CSRC) if not f.endswith(".cu")]
-    shared += [os.path.join(_HERE, "..", "include", "wick_cuda.h"), __file__]
-    return srcs, max(os.path.getmtime(f) for f in shared)
+_INCLUDE = re.compile(r'^\s*#include "([^"]+)"', re.M)
+
+
+def _newest(path: str, seen: set) -> float:
+    """Newest modification time of a source and of what it includes from this repository."""
+    seen.add(path)
+    t = os.path.getmtime(path)
+    with open(path) as f:
+        text = f.read()
+    for name in _INCLUDE.findall(text):
+        inc = os.path.normpath(os.path.join(os.path.dirname(path), name))
+        if inc not in seen and os.path.exists(inc):
+            t = max(t, _newest(inc, seen))
+    return t
+
+
+def _inputs() -> dict:
+    """Per source: newest modification time of what its object depends on."""
+    own = os.path.getmtime(__file__)
+    return {f: max(own, _newest(os.path.join(CSRC, f), set())) for f in SOURCES}
 
 
 def build(force: bool = False, verbose: bool = False, extra: List[str] | None = None) -> str:
     """Compiles what is out of date and links; safe to call from several processes at once."""
-    srcs, shared = _inputs()
-    newest = max(shared, *srcs.values())
+    srcs = _inputs()
+    newest = max(srcs.values())
     if not force and os.path.exists(LIB_PATH) and os.path.getmtime(LIB_PATH) >= newest:
         return LIB_PATH
     objdir = os.path.join(_HERE, "build")
@@ -53,10 +68,10 @@ def build(force: bool = False, verbose: bool = False, extra: List[str] | None = 
         fcntl.flock(lock, fcntl.LOCK_EX)
         if not force and os.path.exists(LIB_PATH) and os.path.getmtime(LIB_PATH) >= newest:
             return LIB_PATH  # another process has just done it
-        return _compile(objdir, srcs, shared, force or bool(extra), verbose, extra or [])
+        return _compile(objdir, srcs, force or bool(extra), verbose, extra or [])
 
 
-def _compile(objdir: str, srcs: dict, shared: float, force: bool, verbose: bool, extra: List[str]) -> str:
+def _compile(objdir: str, srcs: dict, force: bool, verbose: bool, extra: List[str]) -> str:
     nvcc = _nvcc()
     env = dict(os.environ)
     # the environment may export CC/CXX pointing at a non-system compiler; nvcc wants the system g++
@@ -66,7 +81,7 @@ def _compile(objdir: str, srcs: dict, shared: float, force: bool, verbose: bool,
     for src in SOURCES:
         obj = os.path.join(objdir, src.replace(".cu", ".o"))
         objs.append(obj)
-        if not force and os.path.exists(obj) and os.path.getmtime(obj) >= max(shared, srcs[src]):
+        if not force and os.path.exists(obj) and os.path.getmtime(obj) >= srcs[src]:
             continue
         part = f"{obj}.{os.getpid()}.part.o"
         cmd = [nvcc, "-ccbin", ccbin, *NVCC_FLAGS, *extra, "-c", os.path.join(CSRC, src), "-o", part]

@@ -315,7 +315,8 @@ __device__ __forceinline__ void quantize_blocks(Ctx& c, const float (&v)[J], int
     // this lane's block
     const int jm = c.lane >> SH;
     // d = amax / 127 and id = 1 / d, both correctly rounded (simd.rs:255-323) but without the generic division
-    // routine: with r = RN(1/127), q0 = RN(a * r) and rem = RN(fma(-q0, 127, a)), fma(rem, r, q0) equals RN(a / 127)
+    // routine, by a multiplication with the rounded reciprocal and a fused correction (Brisebarre, Muller and Raina, Accelerating
+    // Correctly Rounded Floating-Point Division when the Divisor Is Known in Advance): with r = RN(1/127), q0 = RN(a * r) and rem = RN(fma(-q0, 127, a)), fma(rem, r, q0) equals RN(a / 127)
     // for EVERY finite a >= 0 (checked exhaustively over all 2^31 - 2^23 bit patterns on the host, subnormals
     // included); the reciprocal intrinsic is the correctly rounded 1 / d by definition.
     constexpr float R127 = 1.0f / 127.0f;

@@ -8,6 +8,8 @@
 //   warps 2..9    : epilogue; warp w reads lanes 32 (w % 4).. and one half of the columns; the accumulator of the next tile
 //                   fills the other half of tensor memory meanwhile
 // Out-of-range rows and columns arrive as zeros from TMA, so any m, n, k works (row pitches are multiples of 8).
+// With experts, X is sorted by expert and every expert's rows make tiles of their own against its own matrix; the tiles are
+// counted on the device.
 // Every wait is bounded: on expiry the error word is set, all roles leave, tensor memory is freed.
 // Bound: tensor pipe for many tokens, HBM (weight bytes) for few.
 #include "hybrid_kernels.cuh"
@@ -25,9 +27,12 @@ struct GbParams {
     void* y[2];
     int ldy[2], m[2], k[2];
     int tile_start[3];  // tiles of job 0 from 0, of job 1 from tile_start[1], end tile_start[2]
+    bool f32[2];
     int n;
     int act;
-    float softcap;
+    float scale, softcap;
+    int experts;               // > 0: one matrix of m rows per expert, rows of X sorted by expert
+    const int* expert_start;   // [experts + 1]
     uint32_t* err;
 };
 
@@ -42,14 +47,33 @@ struct GbShape {
 };
 
 struct GbTile {
-    int job, m0, n0;
+    int job, m0, n0, n_end, w_row;  // w_row: where rows m0.. are in the weight map
 };
-__device__ __forceinline__ GbTile gb_tile(const GbParams& p, int t, int tiles_n, int bn) {
+// Experts: expert_tiles[e] = tiles before those of expert e.
+template <bool EXPERTS>
+__device__ __forceinline__ GbTile gb_tile(const GbParams& p, int t, int tiles_n, int bn, const int* expert_tiles) {
     GbTile r;
-    r.job = t >= p.tile_start[1] ? 1 : 0;
-    const int local = t - p.tile_start[r.job];
-    r.m0 = local / tiles_n * GB_M;
-    r.n0 = local % tiles_n * bn;
+    if constexpr (EXPERTS) {
+        int lo = 0, hi = p.experts;  // the last e with expert_tiles[e] <= t
+        while (hi - lo > 1) {
+            const int mid = (lo + hi) / 2;
+            if (expert_tiles[mid] <= t) lo = mid;
+            else hi = mid;
+        }
+        const int s0 = p.expert_start[lo], local = t - expert_tiles[lo];
+        r.n_end = p.expert_start[lo + 1];
+        tiles_n = (r.n_end - s0 + bn - 1) / bn;
+        r.job = 0;
+        r.m0 = local / tiles_n * GB_M;
+        r.n0 = s0 + local % tiles_n * bn;
+        r.w_row = lo * p.m[0] + r.m0;
+    } else {
+        r.job = t >= p.tile_start[1] ? 1 : 0;
+        const int local = t - p.tile_start[r.job];
+        r.m0 = r.w_row = local / tiles_n * GB_M;
+        r.n0 = local % tiles_n * bn;
+        r.n_end = p.n;
+    }
     return r;
 }
 
@@ -59,7 +83,7 @@ __device__ __forceinline__ void gb_ld(uint32_t taddr, int32_t* r) {
     else tmem_ld32(taddr, r);
 }
 
-template <int BN, bool DUAL, class O>
+template <int BN, bool DUAL, bool EXPERTS>
 __global__ void __launch_bounds__(GB_THREADS, 1) k_gemm_bf16(const __grid_constant__ GbParams p) {
     using Sh = GbShape<BN, DUAL>;
     extern __shared__ uint8_t gb_raw[];
@@ -69,7 +93,28 @@ __global__ void __launch_bounds__(GB_THREADS, 1) k_gemm_bf16(const __grid_consta
     uint32_t* tmem_word = reinterpret_cast<uint32_t*>(acc_empty + 2);
     volatile uint32_t* abort = tmem_word + 1;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int tiles_n = (p.n + BN - 1) / BN, tiles = p.tile_start[2];
+    const int tiles_n = (p.n + BN - 1) / BN;
+    const int* expert_tiles = nullptr;
+    if constexpr (EXPERTS) {
+        __shared__ int pre[MAX_EXPERTS + 1];
+        const int tiles_m = (p.m[0] + GB_M - 1) / GB_M;
+        if (warp == 1) {  // running sum over the experts, 32 at a time
+            int base = 0;
+            for (int e0 = 0; e0 < p.experts; e0 += 32) {
+                const int e = e0 + lane;
+                int v = e < p.experts ? (p.expert_start[e + 1] - p.expert_start[e] + BN - 1) / BN * tiles_m : 0;
+#pragma unroll
+                for (int o = 1; o < 32; o <<= 1) {
+                    const int u = __shfl_up_sync(0xffffffffu, v, o);
+                    if (lane >= o) v += u;
+                }
+                if (e < p.experts) pre[e + 1] = base + v;
+                base += __shfl_sync(0xffffffffu, v, 31);
+            }
+            if (lane == 0) pre[0] = 0;
+        }
+        expert_tiles = pre;
+    }
     if (threadIdx.x == 0) {
         for (int s = 0; s < Sh::STAGES; s++) {
             mbar_init(smem_u32(&full[s]), 1);
@@ -91,13 +136,14 @@ __global__ void __launch_bounds__(GB_THREADS, 1) k_gemm_bf16(const __grid_consta
     __syncthreads();
     tc_fence_after();
     const uint32_t tmem = *tmem_word;
+    const int tiles = EXPERTS ? expert_tiles[p.experts] : p.tile_start[2];
 
     if (warp == 0) {
         if (lane == 0) {
             uint32_t g = 0;
             bool ok = true;
             for (int t = blockIdx.x; t < tiles && ok; t += gridDim.x) {
-                const GbTile tl = gb_tile(p, t, tiles_n, BN);
+                const GbTile tl = gb_tile<EXPERTS>(p, t, tiles_n, BN, expert_tiles);
                 const int ks = (p.k[tl.job] + GB_K - 1) / GB_K;
                 for (int i = 0; i < ks; i++, g++) {
                     const int s = g % Sh::STAGES;
@@ -105,8 +151,8 @@ __global__ void __launch_bounds__(GB_THREADS, 1) k_gemm_bf16(const __grid_consta
                     if (!ok) break;
                     const uint32_t bar = smem_u32(&full[s]), dst = smem_u32(stages + (size_t)s * Sh::STAGE);
                     mbar_arrive_expect_tx(bar, Sh::STAGE);
-                    tma_load_2d(dst, &p.map_w[tl.job], bar, i * GB_K, tl.m0);
-                    if (DUAL) tma_load_2d(dst + GB_M * GB_K * 2, &p.map_w[1], bar, i * GB_K, tl.m0);
+                    tma_load_2d(dst, &p.map_w[tl.job], bar, i * GB_K, tl.w_row);
+                    if (DUAL) tma_load_2d(dst + GB_M * GB_K * 2, &p.map_w[1], bar, i * GB_K, tl.w_row);
                     tma_load_2d(dst + Sh::A_BYTES, &p.map_x[tl.job], bar, i * GB_K, tl.n0);
                 }
             }
@@ -117,7 +163,7 @@ __global__ void __launch_bounds__(GB_THREADS, 1) k_gemm_bf16(const __grid_consta
             uint32_t g = 0, it = 0;
             bool ok = true;
             for (int t = blockIdx.x; t < tiles && ok; t += gridDim.x, it++) {
-                const GbTile tl = gb_tile(p, t, tiles_n, BN);
+                const GbTile tl = gb_tile<EXPERTS>(p, t, tiles_n, BN, expert_tiles);
                 const int ks = (p.k[tl.job] + GB_K - 1) / GB_K;
                 const uint32_t buf = it & 1, d = tmem + buf * 256;
                 ok = mbar_wait_bounded(smem_u32(&acc_empty[buf]), ((it >> 1) & 1) ^ 1, abort, p.err, 12);
@@ -146,14 +192,14 @@ __global__ void __launch_bounds__(GB_THREADS, 1) k_gemm_bf16(const __grid_consta
         constexpr int HALF = BN / 2, COLS = HALF < 32 ? HALF : 32;
         uint32_t it = 0;
         for (int t = blockIdx.x; t < tiles; t += gridDim.x, it++) {
-            const GbTile tl = gb_tile(p, t, tiles_n, BN);
+            const GbTile tl = gb_tile<EXPERTS>(p, t, tiles_n, BN, expert_tiles);
             const uint32_t buf = it & 1;
             if (!mbar_wait_bounded(smem_u32(&acc_full[buf]), (it >> 1) & 1, abort, p.err, 14)) break;
             tc_fence_after();
             const int row = tl.m0 + quarter * 32 + lane;
             const bool row_ok = row < p.m[tl.job];
             const uint32_t base = tmem + buf * 256 + ((uint32_t)(quarter * 32) << 16) + half * HALF;
-            O* y = (O*)p.y[tl.job] + row;
+            const bool f32 = p.f32[tl.job];
             const int ldy = p.ldy[tl.job];
 #pragma unroll 1
             for (int c0 = 0; c0 < HALF; c0 += COLS) {
@@ -167,14 +213,25 @@ __global__ void __launch_bounds__(GB_THREADS, 1) k_gemm_bf16(const __grid_consta
                     if (lane == 0) mbar_arrive(smem_u32(&acc_empty[buf]));
                 }
                 const int tok0 = tl.n0 + half * HALF + c0;
-                if (row_ok && tok0 < p.n) {
-                    O* dst = y + (size_t)tok0 * ldy;
+                if (row_ok && tok0 < tl.n_end) {
 #pragma unroll
                     for (int c = 0; c < COLS; c++) {
-                        float f = __int_as_float(v[c]);
-                        if constexpr (DUAL) f = activate(f, (Activation)p.act) * __int_as_float(u[c]);
+                        float f = activate(__int_as_float(v[c]), (Activation)p.act);
+                        if constexpr (DUAL) f *= __int_as_float(u[c]);
+                        f *= p.scale;
                         if (p.softcap > 0.0f) f = p.softcap * tanhf(f / p.softcap);
-                        if (tok0 + c < p.n) dst[(size_t)c * ldy] = f_act<O>(f);
+                        v[c] = __float_as_int(f);
+                    }
+                    if (f32) {
+                        float* dst = (float*)p.y[tl.job] + (size_t)tok0 * ldy + row;
+#pragma unroll
+                        for (int c = 0; c < COLS; c++)
+                            if (tok0 + c < tl.n_end) dst[(size_t)c * ldy] = __int_as_float(v[c]);
+                    } else {
+                        __nv_bfloat16* dst = (__nv_bfloat16*)p.y[tl.job] + (size_t)tok0 * ldy + row;
+#pragma unroll
+                        for (int c = 0; c < COLS; c++)
+                            if (tok0 + c < tl.n_end) dst[(size_t)c * ldy] = __float2bfloat16_rn(__int_as_float(v[c]));
                     }
                 }
             }
@@ -190,29 +247,30 @@ __global__ void __launch_bounds__(GB_THREADS, 1) k_gemm_bf16(const __grid_consta
     }
 }
 
-template <int BN, bool DUAL, class O>
+template <int BN, bool DUAL, bool EXPERTS>
 cudaError_t gb_launch(cudaStream_t st, GbParams& p, int jobs, const DenseCall& c, int sms) {
     using Sh = GbShape<BN, DUAL>;
-    const int tiles_n = (c.n + BN - 1) / BN;
+    const int tiles_n = (c.n + BN - 1) / BN, copies = EXPERTS ? c.experts.count : 1;
     int t = 0;
     for (int i = 0; i < 2; i++) {
         p.tile_start[i] = t;
         if (i < jobs) t += (c.job[i].w.m + GB_M - 1) / GB_M * tiles_n;
     }
     p.tile_start[2] = t;
+    if (EXPERTS) t = (c.job[0].w.m + GB_M - 1) / GB_M * (c.n / BN + std::min(c.n, copies));  // no more than this many
     for (int i = 0; i < c.count; i++) {
-        cudaError_t e = encode_bf16_map(c.job[i].w.w, c.job[i].w.m, c.job[i].w.k, c.job[i].w.ld, GB_M, &p.map_w[i]);
+        cudaError_t e = encode_bf16_map(c.job[i].w.w, c.job[i].w.m * copies, c.job[i].w.k, c.job[i].w.ld, GB_M, &p.map_w[i]);
         if (e == cudaSuccess && i < jobs) e = encode_bf16_map(c.job[i].x, c.n, c.job[i].w.k, c.job[i].ldx, BN, &p.map_x[i]);
         if (e != cudaSuccess) return e;
     }
-    static cudaError_t configured = cudaFuncSetAttribute(k_gemm_bf16<BN, DUAL, O>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Sh::SMEM);
+    static cudaError_t configured = cudaFuncSetAttribute(k_gemm_bf16<BN, DUAL, EXPERTS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Sh::SMEM);
     if (configured != cudaSuccess) return configured;
     g_kernel_launches++;
-    k_gemm_bf16<BN, DUAL, O><<<t < sms ? t : sms, GB_THREADS, Sh::SMEM, st>>>(p);
+    k_gemm_bf16<BN, DUAL, EXPERTS><<<t < sms ? t : sms, GB_THREADS, Sh::SMEM, st>>>(p);
     return cudaGetLastError();
 }
 
-template <bool DUAL, class O>
+template <bool DUAL, bool EXPERTS>
 cudaError_t gb_bn(cudaStream_t st, GbParams& p, int jobs, const DenseCall& c, int sms) {
     // Tile width: fewest (waves x time per k step), a step being bound by the MMA (BN / 2 cycles per 16 columns) or by the
     // operands it reads from shared memory (32 + BN / 4 cycles).
@@ -221,7 +279,12 @@ cudaError_t gb_bn(cudaStream_t st, GbParams& p, int jobs, const DenseCall& c, in
     for (int bn : {256, 128, 64, 32}) {
         if (DUAL && bn == 256) continue;
         long tiles = 0;
-        for (int i = 0; i < jobs; i++) tiles += (long)((c.job[i].w.m + GB_M - 1) / GB_M) * ((c.n + bn - 1) / bn);
+        if (EXPERTS) {  // rows spread evenly over the experts, each with a last tile that is half full on average
+            const int used = std::min(c.n, c.experts.count);
+            tiles = (long)((c.job[0].w.m + GB_M - 1) / GB_M) * std::max<long>(used, (long)(c.n / (double)bn + 0.5 * used));
+        } else {
+            for (int i = 0; i < jobs; i++) tiles += (long)((c.job[i].w.m + GB_M - 1) / GB_M) * ((c.n + bn - 1) / bn);
+        }
         const double step = std::max(bn / 2.0, 32 + bn / 4.0) + 4.0;
         const double cost = (double)((tiles + sms - 1) / sms) * step;
         if (!best || cost < best_cost) {
@@ -230,10 +293,10 @@ cudaError_t gb_bn(cudaStream_t st, GbParams& p, int jobs, const DenseCall& c, in
         }
     }
     switch (best) {
-        case 256: if constexpr (!DUAL) return gb_launch<256, DUAL, O>(st, p, jobs, c, sms);
-        case 128: return gb_launch<128, DUAL, O>(st, p, jobs, c, sms);
-        case 64: return gb_launch<64, DUAL, O>(st, p, jobs, c, sms);
-        default: return gb_launch<32, DUAL, O>(st, p, jobs, c, sms);
+        case 256: if constexpr (!DUAL) return gb_launch<256, DUAL, EXPERTS>(st, p, jobs, c, sms);
+        case 128: return gb_launch<128, DUAL, EXPERTS>(st, p, jobs, c, sms);
+        case 64: return gb_launch<64, DUAL, EXPERTS>(st, p, jobs, c, sms);
+        default: return gb_launch<32, DUAL, EXPERTS>(st, p, jobs, c, sms);
     }
 }
 
@@ -241,7 +304,7 @@ cudaError_t gb_bn(cudaStream_t st, GbParams& p, int jobs, const DenseCall& c, in
 
 cudaError_t launch_dense_tc(cudaStream_t st, const DenseCall& c) {
     if (c.n <= 0) return cudaSuccess;
-    if (!c.err) return cudaErrorInvalidValue;
+    if (!c.err || c.blocks || (c.experts && (!c.experts.start || c.experts.count > MAX_EXPERTS || (c.count == 2 && !c.gated)))) return cudaErrorInvalidValue;
     static int sms = 0;
     if (!sms) {
         int dev = 0, v = 0;
@@ -253,17 +316,21 @@ cudaError_t launch_dense_tc(cudaStream_t st, const DenseCall& c) {
     GbParams p{};
     p.n = c.n;
     p.act = c.act;
+    p.scale = c.scale;
     p.softcap = c.softcap;
     p.err = c.err;
+    p.experts = c.experts.count;
+    p.expert_start = c.experts.start;
     const int jobs = c.gated ? 1 : c.count;
     for (int i = 0; i < jobs; i++) {
         p.y[i] = c.job[i].y;
         p.ldy[i] = c.job[i].ldy;
         p.m[i] = c.job[i].w.m;
         p.k[i] = c.job[i].w.k;
+        p.f32[i] = c.job[i].f32;
     }
-    if (c.gated) return c.out_f32 ? gb_bn<true, float>(st, p, jobs, c, sms) : gb_bn<true, __nv_bfloat16>(st, p, jobs, c, sms);
-    return c.out_f32 ? gb_bn<false, float>(st, p, jobs, c, sms) : gb_bn<false, __nv_bfloat16>(st, p, jobs, c, sms);
+    if (c.experts) return c.gated ? gb_bn<true, true>(st, p, jobs, c, sms) : gb_bn<false, true>(st, p, jobs, c, sms);
+    return c.gated ? gb_bn<true, false>(st, p, jobs, c, sms) : gb_bn<false, false>(st, p, jobs, c, sms);
 }
 
 }  // namespace wick

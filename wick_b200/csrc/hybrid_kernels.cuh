@@ -1,5 +1,6 @@
 // Launch wrappers of the kernels behind models that are described by a config.json layer list (hybrid.cu): dense bfloat16
-// matrices, hyper-connection streams, windowed attention with blended sigmoid scores, and the channel-decay delta rule.
+// matrices (plain, block-diagonal, per expert), hyper-connection streams, a plain residual with norms around the sublayers,
+// windowed attention with blended sigmoid scores, latent attention, the channel-decay delta rule and the matrix memory.
 // Sizes and constants are arguments, so that another design can use the same kernels.
 //
 // Activations are token-major.  "act" buffers hold the model's activation type: bfloat16, or f32 for a model created with
@@ -24,32 +25,64 @@ struct DenseWeight {
     const __nv_bfloat16* w = nullptr;
     int m = 0, k = 0, ld = 0;
 };
-enum Activation { ACT_RELU = 0, ACT_SILU = 1 };
+enum Activation { ACT_RELU = 0, ACT_SILU = 1, ACT_RELU2 = 2, ACT_NONE = 3 };
 struct DenseJob {
     DenseWeight w;
     const void* x = nullptr;  // act [n][ldx]
     int ldx = 0;
     void* y = nullptr;        // act or f32 [n][ldy]
     int ldy = 0;
+    bool f32 = false;         // y is f32 whatever the activation type
 };
-// y = x W^T for n rows.  Up to two independent jobs share a launch; or (gated) the two jobs are gate and up matrices of the
-// same shape and input and job[0].y = activation(gate x) * (up x).
+// Block-diagonal matrix: `rows` weight rows per block; block b multiplies columns b * x_step .. of x and fills columns
+// b * y_step .. of y.
+struct DenseBlocks {
+    int rows = 0, x_step = 0, y_step = 0;
+    __host__ __device__ explicit operator bool() const { return rows > 0; }
+};
+// One matrix per expert, stacked (job.w.m rows each).  Few tokens: routed row r belongs to choice r % top of token r / top and
+// its expert is looked up; many tokens: rows are sorted by expert, expert e has rows start[e] .. start[e + 1] - 1.
+struct DenseExperts {
+    int count = 0, top = 1;
+    const int* table = nullptr;  // [vocab][top]
+    const uint32_t* tokens = nullptr;
+    const DecodeCtl* ctl = nullptr;  // the single token of a decode step, when tokens == NULL
+    bool x_per_token = false;    // (lookup) the input row of routed row r is r / top
+    const int* start = nullptr;  // [count + 1]; NULL: lookup
+    __host__ __device__ explicit operator bool() const { return count > 0; }
+};
+// y = act(x W^T) for n rows.  Up to two independent jobs share a launch; or (gated) the two jobs are gate and up matrices of
+// the same shape and input and job[0].y = act(gate x) * (up x).
 struct DenseCall {
     DenseJob job[2];
     int count = 1, n = 0;
-    bool out_f32 = false;   // y is f32 whatever the activation type
     bool gated = false;
-    Activation act = ACT_RELU;
-    float softcap = 0.0f;   // > 0: y = softcap * tanh(y / softcap)
+    Activation act = ACT_NONE;
+    float scale = 1.0f;     // y times this
+    float softcap = 0.0f;   // > 0: then y = softcap * tanh(y / softcap)
+    DenseBlocks blocks;     // one ungated job
+    DenseExperts experts;   // one job, or gated; n counts routed rows
     uint32_t* err = nullptr;  // device word for expired waits of the tensor-core kernel
 };
-// Chooses between the row-streaming kernel (few rows), the tcgen05 kernel (bfloat16) and the f32 kernel.
+// Chooses between the row-streaming kernel (few rows, blocks), the tcgen05 kernel (bfloat16) and the f32 kernel.
 cudaError_t launch_dense(cudaStream_t st, bool bf16, const DenseCall& call);
 // The individual kernels (launch_dense picks one).
-void launch_dense_rows(cudaStream_t st, bool bf16, const DenseCall& call);    // n <= DENSE_ROWS_MAX
+void launch_dense_rows(cudaStream_t st, bool bf16, const DenseCall& call);    // n <= DENSE_ROWS_MAX; any n for blocks and looked-up experts
 void launch_dense_simt(cudaStream_t st, bool bf16, const DenseCall& call);    // any n
 cudaError_t launch_dense_tc(cudaStream_t st, const DenseCall& call);          // bfloat16, tcgen05
 constexpr int DENSE_ROWS_MAX = 8;
+constexpr int MAX_EXPERTS = 1024;
+
+// Sorts the n * top routed rows of a portion by expert, one table per block of the launch:
+// inv[j * top + s] = sorted row of token j's choice s, start[e] = first row of expert e (start[count] = n * top).
+struct RouteJob {
+    const int* table = nullptr;  // [vocab][top]
+    int* inv = nullptr;
+    int* start = nullptr;
+    int experts = 0, top = 1;
+};
+constexpr int MAX_ROUTES = 64;  // tables per launch
+void launch_route(cudaStream_t st, const uint32_t* tokens, int n, const RouteJob* jobs, int count);
 
 // ── where the rows of a launch live ────────────────────────────────────────
 // Either n consecutive tokens of one sequence (positions == NULL: row j is at start_pos + j, state s0 / s1), or one token of
@@ -95,6 +128,40 @@ struct HyperArgs {
 };
 constexpr int HYPER_MAX_STREAMS = 16;
 void launch_hyper_norm(cudaStream_t st, bool bf16, const HyperArgs& a);
+
+// ── one residual stream with norms before and after every sublayer ─────────
+// One launch takes the previous sublayer's output into x and makes the next sublayer's input:
+//   x <- the embedding row or frame                (embed / frames)
+//   x <- x + post * rms(y)                         (post != NULL; y the sum of y_parts rows times y_scale)
+//   x <- y + shift                                 (post == NULL, shift != NULL)
+//   h  = gain * rms(x), or h = [x | x0] with the embedding output x0 (gain == NULL)
+// with rms(z) = z / sqrt(mean(z^2) + eps).
+struct ResidualArgs {
+    const uint32_t* tokens = nullptr;     // where embedding rows come from, for the start and for x0
+    const DecodeCtl* ctl = nullptr;
+    const __nv_bfloat16* embed = nullptr;
+    int ld_embed = 0;
+    const float* frames = nullptr;        // [n][W]
+    bool init = false;                    // x starts as the embedding row / frame
+    float* x = nullptr;                   // [n][W]
+    bool store_x = true;
+    const float* y = nullptr;             // [rows][ldy] f32 output of the previous sublayer
+    int ldy = 0;
+    int y_parts = 1;                      // rows j * y_parts .. of y belong to token j, or (y_rows) rows y_rows[j * y_parts ..]
+    const int* y_rows = nullptr;
+    float y_scale = 1.0f;
+    const float *post = nullptr, *shift = nullptr;  // [W]
+    const float* gain = nullptr;          // [W]
+    float eps = 0.0f;
+    const int* rows = nullptr;            // if set, output row i comes from token rows[i] (x is then not written)
+    void* h = nullptr;                    // act [..][ldh]
+    int ldh = 0;
+    int h_parts = 1;                      // with h_rows: h of token j goes to rows h_rows[j * h_parts ..]
+    const int* h_rows = nullptr;
+    float* normed = nullptr;              // optional f32 copy of the last row's h [W]
+    int n = 0, W = 0;
+};
+void launch_residual_norm(cudaStream_t st, bool bf16, const ResidualArgs& a);
 
 // ── windowed attention with blended sigmoid scores ─────────────────────────
 struct MixAttnShape {
@@ -168,13 +235,81 @@ void launch_delta_scan(cudaStream_t st, int n, const DeltaShape& s, const RowSta
 // The two steps of the prompt form (called by the launchers above).
 void launch_delta_chunk_prep(cudaStream_t st, bool bf16, const DeltaPrepArgs& a, const DeltaShape& s, const RowState& rs, const DeltaWork& w);
 void launch_delta_chunk_scan(cudaStream_t st, int n, const DeltaShape& s, const RowState& rs, const DeltaWork& w);
-// out act [n][ldo] = rms(o) * norm * sigmoid(gate), gate f32 [n][ldg]
-void launch_delta_out(cudaStream_t st, bool bf16, int n, const DeltaShape& s, const float* o, const float* norm, const float* gate, int ldg,
-                      void* out, int ldo);
+// out act [n][ldo] = rms(o) * norm * sigmoid(gate) per head of E values: o f32 [n][H * E], head h's weights at norm + h *
+// norm_step, gate f32 or act [n][ldg]
+void launch_gated_head_norm(cudaStream_t st, bool bf16, int n, int H, int E, float eps, const float* o, const float* norm, int norm_step,
+                            const void* gate, bool gate_f32, int ldg, void* out, int ldo);
 
 // One decode token per row: convolutions, decays, the recurrence and the gated norm in one launch (state s0 / p0 and s1 / p1).
 void launch_delta_step(cudaStream_t st, bool bf16, const DeltaPrepArgs& a, const DeltaShape& s, const RowState& rs, const float* norm,
                        const float* gate, int ldg, void* out, int ldo);
+
+// ── latent attention ───────────────────────────────────────────────────────
+// Queries come through a latent of q_rank, keys and values through a latent of kv_rank that all heads share, beside rot_dim
+// key columns that carry the position.  Only the normalised latent and the rotated key part are cached, one row per position:
+//   [c: kv_rank, up to a multiple of 8 | rotated part: rot_dim, up to a multiple of 8]   (padding zero)
+// A query may be taken to the latent's side, q_c = W_uk^T q, so that its score is one product with a cache row and the weighted
+// sum of cache rows gives the value through W_uv ("absorbed"; decode, short portions, f32); or keys and values of the visible
+// positions are computed from the cache (prompts).  Softmax has one more entry per head, `sink`, without a value.
+struct LatentShape {
+    int heads = 0, dim = 0, rot_dim = 0, rot_dims = 0, vdim = 0, q_rank = 0, kv_rank = 0;
+    int size = 0;                  // sliding window (0: none): key j is seen by i when i - j < size
+    float scale = 1.0f, eps = 0.0f;
+    const float* sink = nullptr;   // [H]
+    const float2* rope = nullptr;  // [positions][rot_dims / 2] cos, sin of the first rot_dims of the rot_dim columns, in pairs
+    const float *q_norm = nullptr, *kv_norm = nullptr;
+    __host__ __device__ int ldc() const { return round_up(kv_rank, 8) + round_up(rot_dim, 8); }  // cache row
+    __host__ __device__ int off_rot() const { return round_up(kv_rank, 8); }
+    // a query row: per head [dim, up to a multiple of 8 | rot_dim, up to a multiple of 8]
+    __host__ __device__ int q_off_rot() const { return round_up(dim, 8); }
+    __host__ __device__ int q_pitch() const { return round_up(dim, 8) + round_up(rot_dim, 8); }
+    __host__ __device__ int off_kv() const { return round_up(q_rank, 8); }  // of the projections' row: [c_q | c, rotated part]
+    int seen(int max_seq) const { return size > 0 && size < max_seq ? size : max_seq; }
+};
+// Rows of p act [n][ldp]: c_q normalised in place, c normalised and the rotated part turned into the cache (state s0 / p0).
+void launch_latent_append(cudaStream_t st, bool bf16, void* p, int ldp, int n, const LatentShape& s, const RowState& rs);
+// Absorbed attention: qc act [n][H][ldc] (q taken to the latent's side in the first kv_rank columns of a head), q act [n][ldq]
+// (the rotated columns are read from here).  o act [n][H][ldo_h]: weighted sums of latents.  partial: latent_scratch() floats.
+size_t latent_scratch(const LatentShape& s, int max_rows);
+bool latent_supported(const LatentShape& s);
+cudaError_t launch_latent_attn(cudaStream_t st, bool bf16, const void* qc, const void* q, int ldq, int n, const LatentShape& s, const RowState& rs,
+                               void* o, int ldo_h, float* partial, int max_seq);
+
+// ── matrix memory ──────────────────────────────────────────────────────────
+// Per head, with log gates i, f and a running maximum m (log domain):
+//   m' = max(f + m, i);  S <- exp(f + m - m') S + exp(i - m') k v^T;  z likewise with v = 1
+//   o = S^T q / (max(|z . q|, exp(-m')) + 1e-6)
+// The state holds S^T and z together: s0 f32 [H][vdim + 1][dimp], z being the last row; s1 f32 [H]: m.
+struct MemoryShape {
+    int heads = 0, dim = 0, vdim = 0;
+    float cap = 1.0f, eps = 0.0f;
+    const float *i_bias = nullptr, *f_bias = nullptr, *norm = nullptr;  // [H], [H], [H * vdim]
+    __host__ __device__ int dimp() const { return round_up(dim, 32); }
+    __host__ __device__ int rows() const { return vdim + 1; }
+    size_t state_floats() const { return (size_t)heads * rows() * dimp(); }
+};
+constexpr int MEMORY_CHUNK = 64;
+constexpr int MEMORY_MAX_DIM = 4096;  // of keys and of values
+// Work memory for n tokens of one sequence.
+struct MemoryWork {
+    double *a = nullptr, *g = nullptr;                   // [H][n]: log weight of token j in token t's sum = a[t] + g[j] (same chunk)
+    float *carry = nullptr, *write = nullptr, *m = nullptr;  // [H][n]: weight of the chunk's first state; of token j in the next; m
+    float* keep = nullptr;                               // [H][chunks]: weight of the chunk's first state in the next
+    float* S = nullptr;                                  // [chunks][H][vdim + 1][dimp] states at the chunks' starts
+    float* o = nullptr;                                  // [n][H * vdim] read-outs
+};
+// Projections: q | k | v | g act columns of a row of p (ldp) in this order, gates f32 [n][ldi]: H input, then H forget logits.
+struct MemoryArgs {
+    const void* p = nullptr;
+    int ldp = 0;
+    const float* gates = nullptr;
+    int ldi = 0, n = 0;
+};
+// Consecutive tokens of one sequence: read-outs, normalised and gated, to out act [n][ldo].
+cudaError_t launch_memory_prompt(cudaStream_t st, bool bf16, const MemoryArgs& a, const MemoryShape& s, const RowState& rs, const MemoryWork& w,
+                                 void* out, int ldo);
+// One decode token per row.
+void launch_memory_step(cudaStream_t st, bool bf16, const MemoryArgs& a, const MemoryShape& s, const RowState& rs, void* out, int ldo);
 
 // ── launches that may start before their predecessor has finished ──────────
 // The kernels of a decode step are launched with programmatic stream serialisation: a kernel is brought up while the one before
@@ -225,7 +360,11 @@ __device__ __forceinline__ void load8(const float* p, float* f) {
 }
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
-__device__ __forceinline__ float activate(float z, Activation a) { return a == ACT_RELU ? fmaxf(z, 0.0f) : silu_f(z); }
+__device__ __forceinline__ float activate(float z, Activation a) {
+    if (a == ACT_SILU) return silu_f(z);
+    const float r = fmaxf(z, 0.0f);
+    return a == ACT_RELU ? r : a == ACT_RELU2 ? r * r : z;
+}
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -37,7 +37,7 @@ int32_t wick_cuda_dense(int32_t compute, const void* w_dev, const void* w_up_dev
     const uint32_t k8 = (k + 7) / 8 * 8;
     if (!m || !k || ldw % 8 || ldx % 8 || ldw != k8 || ldx < k8 || ldy < m || !aligned16(w_dev) || !aligned16(x_dev) || (w_up_dev && !aligned16(w_up_dev)))
         return fail(WICK_CUDA_ERR_BAD_ARG, "dense: ldw must be k rounded up to 8, ldx a multiple of 8 and at least that, ldy >= m, 16-byte aligned bases");
-    if (activation != ACT_RELU && activation != ACT_SILU) return fail(WICK_CUDA_ERR_BAD_ARG, "dense: unknown activation");
+    if (activation < ACT_RELU || activation > ACT_NONE) return fail(WICK_CUDA_ERR_BAD_ARG, "dense: unknown activation");
     if (n == 0) return WICK_CUDA_OK;
     if (path < 0 || path > 3 || (path == WICK_CUDA_DENSE_ROWS && n > (uint32_t)DENSE_ROWS_MAX) || (path == WICK_CUDA_DENSE_TENSOR && !bf16))
         return fail(WICK_CUDA_ERR_BAD_ARG, "dense: this path does not take these arguments");
@@ -50,7 +50,7 @@ int32_t wick_cuda_dense(int32_t compute, const void* w_dev, const void* w_up_dev
     c.job[0].w.m = (int)m; c.job[0].w.k = (int)k; c.job[0].w.ld = (int)ldw;
     c.job[0].x = x_dev; c.job[0].ldx = (int)ldx; c.job[0].y = y_dev; c.job[0].ldy = (int)ldy;
     c.n = (int)n;
-    c.out_f32 = y_f32 != 0 || !bf16;
+    c.job[0].f32 = y_f32 != 0 || !bf16;
     c.softcap = softcap;
     c.act = (Activation)activation;
     c.err = (uint32_t*)err.p;
@@ -151,7 +151,7 @@ int32_t wick_cuda_channel_delta(int32_t compute, const void* proj_dev, uint32_t 
     a.conv_w = conv_w_dev; a.A_log = a_log_dev; a.dt_bias = dt_bias_dev; a.n = (int)n;
     launch_delta_prep(st, bf16, a, s, rs, w);
     launch_delta_scan(st, (int)n, s, rs, w);
-    launch_delta_out(st, bf16, (int)n, s, w.o, norm_dev, gate_dev, (int)(heads * vdim), out_dev, (int)ldo);
+    launch_gated_head_norm(st, bf16, (int)n, s.heads, s.vdim, s.eps, w.o, norm_dev, 0, gate_dev, true, (int)(heads * vdim), out_dev, (int)ldo);
     CU_TRY(cudaGetLastError());
     return WICK_CUDA_OK;
 }

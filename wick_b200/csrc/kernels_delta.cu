@@ -7,7 +7,7 @@
 //                per (token, group of channels that is normalised together).
 // k_delta_scan   their recurrence; the state stays in registers, q, k, g rows are staged in shared memory with cp.async.
 // k_delta_step   one decode token per row: all of it, and the gated norm, in one launch.
-// k_delta_out    RMS norm over the value channels of a head, gain, sigmoid gate (also after delta_chunk.cu).
+// k_gated_head_norm  RMS norm over the value channels of a head, weights, sigmoid gate (also after delta_chunk.cu, kernels_memory.cu).
 #include "hybrid_kernels.cuh"
 
 namespace wick {
@@ -366,9 +366,9 @@ void step_any(cudaStream_t st, const DeltaPrepArgs& a, const DeltaShape& s, cons
 }
 
 // ── output ─────────────────────────────────────────────────────────────────
-template <class T>
-__global__ void __launch_bounds__(256) k_delta_out(int n, int H, int E, float eps, const float* __restrict__ o, const float* __restrict__ norm,
-                                                   const float* __restrict__ gate, int ldg, T* __restrict__ out, int ldo) {
+template <class T, class TG>
+__global__ void __launch_bounds__(256) k_gated_head_norm(int n, int H, int E, float eps, const float* __restrict__ o, const float* __restrict__ norm, int norm_step,
+                                                         const TG* __restrict__ gate, int ldg, T* __restrict__ out, int ldo) {
     const int lane = threadIdx.x & 31;
     const size_t unit = (size_t)blockIdx.x * 8 + (threadIdx.x >> 5);
     if (unit >= (size_t)n * H) return;
@@ -378,7 +378,7 @@ __global__ void __launch_bounds__(256) k_delta_out(int n, int H, int E, float ep
     for (int i = lane; i < E; i += 32) ss = fmaf(src[i], src[i], ss);
     const float r = 1.0f / sqrtf(warp_sum(ss) / (float)E + eps);
     for (int i = lane; i < E; i += 32)
-        out[(size_t)j * ldo + h * E + i] = f_act<T>(src[i] * r * norm[i] * sigmoid_f(gate[(size_t)j * ldg + h * E + i]));
+        out[(size_t)j * ldo + h * E + i] = f_act<T>(src[i] * r * norm[h * norm_step + i] * sigmoid_f(act_f(gate[(size_t)j * ldg + h * E + i])));
 }
 
 }  // namespace
@@ -427,13 +427,15 @@ void launch_delta_step(cudaStream_t st, bool bf16, const DeltaPrepArgs& a, const
     else step_any(st, a, s, rs, norm, gate, ldg, (float*)out, ldo);
 }
 
-void launch_delta_out(cudaStream_t st, bool bf16, int n, const DeltaShape& s, const float* o, const float* norm, const float* gate, int ldg,
-                      void* out, int ldo) {
+void launch_gated_head_norm(cudaStream_t st, bool bf16, int n, int H, int E, float eps, const float* o, const float* norm, int norm_step,
+                            const void* gate, bool gate_f32, int ldg, void* out, int ldo) {
     if (n <= 0) return;
-    const unsigned grid = (unsigned)(((size_t)n * s.heads + 7) / 8);
+    const unsigned grid = (unsigned)(((size_t)n * H + 7) / 8);
+    using B = __nv_bfloat16;
     g_kernel_launches++;
-    if (bf16) k_delta_out<__nv_bfloat16><<<grid, 256, 0, st>>>(n, s.heads, s.vdim, s.eps, o, norm, gate, ldg, (__nv_bfloat16*)out, ldo);
-    else k_delta_out<float><<<grid, 256, 0, st>>>(n, s.heads, s.vdim, s.eps, o, norm, gate, ldg, (float*)out, ldo);
+    if (!bf16) k_gated_head_norm<float, float><<<grid, 256, 0, st>>>(n, H, E, eps, o, norm, norm_step, (const float*)gate, ldg, (float*)out, ldo);
+    else if (gate_f32) k_gated_head_norm<B, float><<<grid, 256, 0, st>>>(n, H, E, eps, o, norm, norm_step, (const float*)gate, ldg, (B*)out, ldo);
+    else k_gated_head_norm<B, B><<<grid, 256, 0, st>>>(n, H, E, eps, o, norm, norm_step, (const B*)gate, ldg, (B*)out, ldo);
 }
 
 }  // namespace wick

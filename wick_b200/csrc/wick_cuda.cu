@@ -940,6 +940,7 @@ struct ArchEntry {
 const ArchEntry ARCHITECTURES[] = {
     {"lfm2", &LFM2_FAMILY, lfm2_build, nullptr},
     {"Nositar", &HYBRID_FAMILY, nullptr, nositar_build},
+    {"Novorax", &HYBRID_FAMILY, nullptr, novorax_build},
 };
 const ArchEntry* find_architecture(const std::string& name) {
     for (const ArchEntry& a : ARCHITECTURES)
@@ -1275,7 +1276,7 @@ int32_t wick_cuda_model_config(const wick_cuda_model* m, wick_cuda_config* out) 
 const char* wick_cuda_model_architecture(const wick_cuda_model* m) { return m ? m->arch.c_str() : ""; }
 
 const char* wick_cuda_model_layer_type(const wick_cuda_model* m, uint32_t layer) {
-    if (!m || layer >= m->layers.size()) return "";
+    if (!m || layer >= m->cfg.n_layers) return "";
     if (m->hybrid) return hybrid_layer_type(m, (int)layer);
     return m->layers[layer].is_attn ? "Attention" : "GatedConv";
 }
@@ -1283,7 +1284,10 @@ const char* wick_cuda_model_layer_type(const wick_cuda_model* m, uint32_t layer)
 int32_t wick_cuda_model_kv_heads_per_layer(const wick_cuda_model* m, uint32_t* out, uint32_t n) {
     W_TRY(check_model(m));
     if (!out || n != m->cfg.n_layers) return fail(WICK_CUDA_ERR_BAD_ARG, "out is NULL or n != n_layers");
-    for (uint32_t i = 0; i < n; i++) out[i] = m->layers[i].is_attn ? m->layers[i].n_kv : 0;
+    for (uint32_t i = 0; i < n; i++) {
+        const Layer& L = m->layers[m->hybrid ? hybrid_first_run(m, (int)i) : (int)i];
+        out[i] = L.is_attn ? L.n_kv : 0;
+    }
     return WICK_CUDA_OK;
 }
 

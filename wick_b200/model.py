@@ -423,7 +423,15 @@ class CudaNositarModel(CudaModel):
     architecture = "Nositar"
 
 
-MODEL_CLASSES = {c.architecture: c for c in (CudaLfm2Model, CudaNositarModel)}
+class CudaNovoraxModel(CudaModel):
+    """Novorax from a folder with config.json and model.safetensors: latent attention with a sink over a sliding window and
+    matrix-memory (mLSTM) layers, dense or table-routed expert feed-forwards, norms before and after every sublayer, and a group
+    of layers that may run several times.  dtype "bfloat16" (default) or "float32".  The recurrent state cannot be shifted, and
+    experts are chosen by token id, so there is no n_keep context shift and, with experts, no embedding input."""
+    architecture = "Novorax"
+
+
+MODEL_CLASSES = {c.architecture: c for c in (CudaLfm2Model, CudaNositarModel, CudaNovoraxModel)}
 
 
 def model_architecture(path: str) -> str:

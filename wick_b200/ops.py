@@ -169,7 +169,7 @@ def shortconv(proj: torch.Tensor, conv_w: torch.Tensor, state: torch.Tensor, ker
 
 # ── operators of the config.json models; the activation type is that of the tensors ────────────────────
 _DENSE_PATHS = {"auto": 0, "rows": 1, "f32": 2, "tensor": 3}
-_ACTIVATIONS = {"relu": 0, "silu": 1}
+_ACTIVATIONS = {"relu": 0, "silu": 1, "relu2": 2, "none": 3}
 
 
 def _compute(t: torch.Tensor) -> int:
@@ -185,9 +185,11 @@ def pad8(t: torch.Tensor) -> torch.Tensor:
     return torch.nn.functional.pad(t, (0, -t.shape[-1] % 8)).contiguous()
 
 
-def dense(w: torch.Tensor, x: torch.Tensor, w_up: torch.Tensor | None = None, activation: str = "relu", softcap: float = 0.0,
+def dense(w: torch.Tensor, x: torch.Tensor, w_up: torch.Tensor | None = None, activation: str | None = None, softcap: float = 0.0,
           out_f32: bool = True, path: str = "auto") -> torch.Tensor:
-    """x [n, k] (bf16 or f32) times bf16 w [m, k] transposed; with w_up: activation(w x) * (w_up x)."""
+    """activation(x [n, k] (bf16 or f32) times bf16 w [m, k] transposed); with w_up: activation(w x) * (w_up x).  The activation is
+    none by default, with w_up relu."""
+    activation = activation or ("none" if w_up is None else "relu")
     (m, k), n = w.shape, x.shape[0]
     w8, u8, x8 = pad8(w), None if w_up is None else pad8(w_up), pad8(x)
     y = torch.empty((n, m), dtype=torch.float32 if out_f32 else x.dtype, device=x.device)
