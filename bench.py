@@ -355,6 +355,63 @@ def run_nositar(args):
                       "clocks": clocks, "sizes": res}))
 
 
+def run_novorax(args):
+    """Throughput of the Novorax design at sizes that resemble a real model's layers, beside the closest other model of the
+    library at equal size (Nositar: same width, layer count, attention layers, window, vocabulary and active feed-forward
+    parameters)."""
+    from wick_b200 import nositar_synth as ns
+    from wick_b200 import novorax_synth as vs
+    from wick_b200.model import CudaNositarModel, CudaNovoraxModel
+    os.environ.setdefault("WICK_CUDA_MAX_CHUNK", "4096")
+    hbm, kind = measured_peak()
+    bf16_peak = int8_peak_tflops()[0] / 2
+    sampler = ClockSampler(int(os.environ.get("LOCAL_RANK", "0")))
+    sampler.start()
+    t0 = time.time()
+    res = {}
+    sizes = [s for s in args.sizes.split(",") if s in vs.SPECS] or list(vs.SPECS)
+    rnd = lambda x: {k: (round(v, 4) if isinstance(v, float) else v) for k, v in x.items()}  # noqa: E731
+    for name in sizes:
+        spec = vs.SPECS[name]
+        m = CudaNovoraxModel(vs.cached_model(name), 4608)
+        d = time_design(m, spec.vocab, args, (128, 1024, 4096), (8, 64))
+        m.close()
+        runs = spec.runs()
+        na = sum(i in spec.attn_layers for i in runs)
+        for n in (1024, 4096):
+            c = d[f"prefill_p{n}_ms_by_category"]
+            seen = sum(min(i + 1, spec.window) for i in range(n))
+            d[f"gemm_p{n}_frac_of_bf16_peak"] = 2.0 * spec.matrix_params_per_run() * n / (c["gemm"] * 1e-3) / 1e12 / bf16_peak
+            d[f"attention_p{n}_frac_of_bf16_peak"] = 2.0 * spec.heads * (spec.dim + spec.rot_dim + spec.vdim) * seen * na / (c["attention"] * 1e-3) / 1e12 / bf16_peak
+            # multiply-adds of the token-by-token form: k v^T into the state, q out of it
+            d[f"recurrence_p{n}_frac_of_f32_peak"] = 4.0 * n * (len(runs) - na) * spec.mem_heads * spec.mem_dim * (spec.mem_vdim + 1) / (c["recurrence"] * 1e-3) / 74.4e12
+            d[f"residual_p{n}_frac_of_hbm"] = n * spec.width * 14.0 * 2 * len(runs) / (c["rmsnorm+quantise"] * 1e-3) / 1e9 / hbm
+        for p in (128, 1024):
+            d[f"decode_at_{p}_frac_of_hbm"] = spec.decode_bytes_per_token(p + DECODE_TOKENS // 2) / (d[f"decode_at_{p}_ms"] * 1e-3) / 1e9 / hbm
+        other = name.replace("novorax", "nositar")
+        os_ = ns.SPECS[other]
+        m = CudaNositarModel(ns.cached_model(other), 4608)
+        e = time_design(m, os_.vocab, args, (128, 1024, 4096), (8, 64))
+        m.close()
+        for n in (1024, 4096):
+            c = e[f"prefill_p{n}_ms_by_category"]
+            seen = sum(min(i + 1, os_.window + os_.keep_first) for i in range(n))
+            nd = os_.n_layers - len(os_.attn_layers)
+            e[f"gemm_p{n}_frac_of_bf16_peak"] = 2.0 * os_.matrix_params_per_layer() * n / (c["gemm"] * 1e-3) / 1e12 / bf16_peak
+            e[f"attention_p{n}_frac_of_bf16_peak"] = 4.0 * os_.width * seen * len(os_.attn_layers) / (c["attention"] * 1e-3) / 1e12 / bf16_peak
+            e[f"recurrence_p{n}_frac_of_f32_peak"] = 8.0 * n * nd * os_.width * (os_.width // os_.delta_heads) / (c["recurrence"] * 1e-3) / 74.4e12
+            e[f"streams_p{n}_frac_of_hbm"] = n * os_.width * (8 * os_.streams + 6) * 2 * os_.n_layers / (c["rmsnorm+quantise"] * 1e-3) / 1e9 / hbm
+        for p in (128, 1024):
+            e[f"decode_at_{p}_frac_of_hbm"] = os_.decode_bytes_per_token(p + DECODE_TOKENS // 2) / (e[f"decode_at_{p}_ms"] * 1e-3) / 1e9 / hbm
+        res[name] = {"novorax_bf16": rnd(d), "nositar_bf16_equal_size": rnd(e)}
+    clocks = sampler.stop(t0, time.time())
+    print(json.dumps({"metric": "prefill tok/s @4096, Novorax layers", "value": res[sizes[-1]]["novorax_bf16"]["prefill_p4096_tok_s"], "unit": "tok/s",
+                      "n_gpus": 1, "higher_is_better": True, "dtype": "bf16", "data": "synthetic", "peaks": {"hbm_gbs": hbm, "bf16_tflops": bf16_peak, "source": kind},
+                      "config": {"workload": "6-layer models (2 latent attention, 4 matrix memory; 2 of them with 16 experts, 2 chosen), random weights, WICK_CUDA_MAX_CHUNK="
+                                 + os.environ["WICK_CUDA_MAX_CHUNK"], "l2": "weights and activations larger than L2 for the prompt of 4096"},
+                      "clocks": clocks, "sizes": res}))
+
+
 def workload_config(args, spec):
     return {
         "workload": f"{spec.name} {args.qtype.upper()} bs=1: {PROMPT_TOKENS}-token uniform-random prompt prefill (untimed), "
@@ -378,10 +435,11 @@ def main():
     ap.add_argument("--decode-tokens", type=int, default=DECODE_TOKENS, help="profiling aid; the metric is quoted at 128")
     ap.add_argument("--no-extra", action="store_true", help="skip the prefill / tg512 side measurements")
     ap.add_argument("--no-cpu-baseline", action="store_true")
-    ap.add_argument("--only", default="decode", choices=["decode", "prefill", "nositar"],
+    ap.add_argument("--only", default="decode", choices=["decode", "prefill", "nositar", "novorax"],
                     help="profiling aid: 'prefill' times forward_prefill_chunked of --prompt-tokens instead of the headline decode; "
-                         "'nositar' times layers of the Nositar design beside LFM2 layers of equal size (own JSON line)")
-    ap.add_argument("--sizes", default="nositar-w1024,nositar-w2048", help="models of --only nositar")
+                         "'nositar' times layers of the Nositar design beside LFM2 layers of equal size, 'novorax' layers of the Novorax design "
+                         "beside Nositar layers (own JSON lines)")
+    ap.add_argument("--sizes", default="nositar-w1024,nositar-w2048", help="models of --only nositar / novorax")
     ap.add_argument("--prefill-mode", default="exact", choices=["exact", "tensor", "exact-cuda-cores"])
     ap.add_argument("--context", type=int, default=4096, help="context size the model is created with (prompt + decode tokens must fit)")
     ap.add_argument("--ubatch", type=int, default=512, help="prefill chunk of --only prefill (0 = one call); wick's default is 512")
@@ -415,8 +473,8 @@ def main():
             dist.barrier()
         torch.cuda.synchronize()
 
-    if args.only == "nositar":
-        run_nositar(args)
+    if args.only in ("nositar", "novorax"):
+        (run_nositar if args.only == "nositar" else run_novorax)(args)
         return
 
     path, spec = model_file(args, rank, world)

@@ -112,7 +112,7 @@ def test_architecture_registry(tmp_path):
     cfg = nm.config([nm.delta(2, 1, 8, 8, 3, 0)], **SMALL)
     p = _folder(tmp_path, cfg)
     assert model.model_architecture(p) == "Nositar"
-    assert set(model.MODEL_CLASSES) == {"lfm2", "Nositar"}
+    assert set(model.MODEL_CLASSES) == {"lfm2", "Nositar", "Novorax"}
     assert model.MODEL_CLASSES["Nositar"] is model.CudaNositarModel
     json.dump({"architecture": "Unheard"}, open(os.path.join(p, "config.json"), "w"))
     with pytest.raises(ValueError, match="Unheard"):

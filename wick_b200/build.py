@@ -27,6 +27,10 @@ NVCC_FLAGS = [
 ]
 
 
+# sources of many large kernels: their code generation runs on several threads
+SPLIT = {"delta_chunk.cu": ["--split-compile=0"]}
+
+
 def _nvcc() -> str:
     for cand in (os.environ.get("NVCC"), shutil.which("nvcc"), "/usr/local/cuda/bin/nvcc"):
         if cand and os.path.exists(cand):
@@ -84,7 +88,7 @@ def _compile(objdir: str, srcs: dict, force: bool, verbose: bool, extra: List[st
         if not force and os.path.exists(obj) and os.path.getmtime(obj) >= srcs[src]:
             continue
         part = f"{obj}.{os.getpid()}.part.o"
-        cmd = [nvcc, "-ccbin", ccbin, *NVCC_FLAGS, *extra, "-c", os.path.join(CSRC, src), "-o", part]
+        cmd = [nvcc, "-ccbin", ccbin, *NVCC_FLAGS, *SPLIT.get(src, []), *extra, "-c", os.path.join(CSRC, src), "-o", part]
         if verbose:
             cmd.insert(1, "-Xptxas=-v")
         procs.append((cmd, part, obj, subprocess.Popen(cmd, env=env, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)))

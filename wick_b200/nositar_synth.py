@@ -90,42 +90,54 @@ SPECS: Dict[str, NositarSpec] = {
 }
 
 
-def write_model(folder: str, spec: NositarSpec, seed: int = 0) -> str:
+def write_folder(folder: str, config: dict, shapes: Dict[str, Tuple[int, ...]], draw, seed: int = 0) -> str:
+    """config.json and model.safetensors with the tensors that draw(name, shape, generator) returns: int32 ones as such, the rest
+    rounded to bfloat16."""
     import torch
     gen = torch.Generator("cuda").manual_seed(seed)
     os.makedirs(folder, exist_ok=True)
-    shapes = spec.shapes()
+    is_int = {name: name.endswith(".table") for name in shapes}
     head, at = {}, 0
     for name, s in shapes.items():
-        n = 2
+        n = 4 if is_int[name] else 2
         for d in s:
             n *= d
-        head[name] = {"dtype": "BF16", "shape": list(s), "data_offsets": [at, at + n]}
+        head[name] = {"dtype": "I32" if is_int[name] else "BF16", "shape": list(s), "data_offsets": [at, at + n]}
         at += n
     h = json.dumps(head).encode()
     tmp = os.path.join(folder, f"model.{os.getpid()}.part")
     with open(tmp, "wb") as f:
         f.write(struct.pack("<Q", len(h)) + h)
         for name, s in shapes.items():
-            t = torch.randn(s, generator=gen, device="cuda")
-            last = name.split(".")[-1]
-            if len(s) == 2 and last not in ("talk", "mix", "conv"):
-                t *= s[1] ** -0.5
-            elif last in ("talk", "mix"):
-                t = 0.2 * t / s[0] ** 0.5 + torch.eye(s[0], device="cuda")
-            elif last == "in":
-                t = 0.1 * t + 1.0 / s[0]
-            elif last == "pb":
-                t = 0.3 * t - 5.0
-            elif last in ("A_log", "dt_bias"):
-                t = 0.5 * t - 2.0
-            elif last != "conv" and name != "embed":
-                t = 0.1 * t + 1.0
-            f.write(t.to(torch.bfloat16).cpu().view(torch.int16).numpy().tobytes())
+            t = draw(name, s, gen)
+            f.write((t.to(torch.int32).cpu() if is_int[name] else t.to(torch.bfloat16).cpu().view(torch.int16)).numpy().tobytes())
     os.replace(tmp, os.path.join(folder, "model.safetensors"))
     with open(os.path.join(folder, "config.json"), "w") as f:
-        json.dump(spec.config(), f)
+        json.dump(config, f)
     return folder
+
+
+def draw_weight(name, s, gen):
+    import torch
+    t = torch.randn(s, generator=gen, device="cuda")
+    last = name.split(".")[-1]
+    if len(s) == 2 and last not in ("talk", "mix", "conv"):
+        t *= s[1] ** -0.5
+    elif last in ("talk", "mix"):
+        t = 0.2 * t / s[0] ** 0.5 + torch.eye(s[0], device="cuda")
+    elif last == "in":
+        t = 0.1 * t + 1.0 / s[0]
+    elif last == "pb":
+        t = 0.3 * t - 5.0
+    elif last in ("A_log", "dt_bias"):
+        t = 0.5 * t - 2.0
+    elif last != "conv" and name != "embed":
+        t = 0.1 * t + 1.0
+    return t
+
+
+def write_model(folder: str, spec: NositarSpec, seed: int = 0) -> str:
+    return write_folder(folder, spec.config(), spec.shapes(), draw_weight, seed)
 
 
 def cached_model(name: str, seed: int = 0) -> str:
