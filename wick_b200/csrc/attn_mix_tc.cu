@@ -37,17 +37,6 @@ struct MtParams {
     uint32_t* err;
 };
 
-// MN-major operand tile (keys down, 64-column boxes of `box_bytes`), 128B swizzle.
-__device__ __forceinline__ unsigned long long umma_desc_mn_sw128(uint32_t smem_addr, uint32_t box_bytes) {
-    unsigned long long d = 0;
-    d |= (unsigned long long)((smem_addr >> 4) & 0x3FFF);
-    d |= (unsigned long long)(box_bytes >> 4) << 16;   // next 64 columns
-    d |= (unsigned long long)(1024 >> 4) << 32;        // next 8 keys
-    d |= 1ull << 46;
-    d |= 2ull << 61;
-    return d;
-}
-
 __global__ void __launch_bounds__(MT_THREADS, 1) k_mix_attn_tc(const __grid_constant__ MtParams p) {
     extern __shared__ uint8_t mt_raw[];
     uint8_t* sm = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(mt_raw) + 1023) & ~(uintptr_t)1023);
@@ -127,7 +116,7 @@ __global__ void __launch_bounds__(MT_THREADS, 1) k_mix_attn_tc(const __grid_cons
     } else if (warp == 1) {
         if (lane == 0) {
             const uint32_t idesc_s = umma_bf16_idesc(MT_Q, MT_K);
-            const uint32_t idesc_o = umma_bf16_idesc(MT_Q, round_up(p.vdim, 16)) | (1u << 16);  // B (V) is MN-major
+            const uint32_t idesc_o = umma_bf16_idesc(MT_Q, round_up(p.vdim, 16)) | UMMA_B_MN;  // V
             uint32_t g = 0;
             bool ok = !p.q_resident || mbar_wait_bounded(smem_u32(q_full), 0, abort, p.err, 23);
             for (int t = 0; t <= tiles && ok; t++) {

@@ -215,6 +215,13 @@ struct Step {
         launch_latent_append(m->stream, hm.bf16, hm.proj, hm.ldp, n, s, rs);
         mark(PC_QK_ROPE_KV);
         W_TRY(dense(L.uq, hm.proj, hm.ldp, hm.q, hm.ldq, false));
+        if (L.ukv.w && !rs.separate() && n >= LATENT_TC_MIN_ROWS) {
+            CU_TRY(launch_latent_kv(m->stream, n, s, rs, L.ukv, hm.kv, m->tc_err));
+            mark(PC_GEMM);
+            CU_TRY(launch_latent_attn_tc(m->stream, hm.q, hm.ldq, n, s, rs, hm.kv, hm.mixed, hm.ldm, m->tc_err));
+            mark(PC_ATTENTION);
+            return WICK_CUDA_OK;
+        }
         W_TRY(blocks(L.uk_t, s.kv_rank, hm.q, hm.ldq, s.q_pitch(), hm.qc, s.heads * s.ldc(), s.ldc()));
         mark(PC_GEMM);
         CU_TRY(launch_latent_attn(m->stream, hm.bf16, hm.qc, hm.q, hm.ldq, n, s, rs, hm.oc, s.off_rot(), hm.latent_partial, (int)m->cfg.max_seq_len));
@@ -391,7 +398,7 @@ int32_t hybrid_alloc_scratch(wick_cuda_model* m) {
     const size_t act_bytes = hm.bf16 ? 2 : 4, N = (size_t)m->max_chunk;
     const int streams = std::max(hm.streams, 1);
     int ldp = 8, ldm = 8, ldf = 8, lda = 0, ldg = 0, ldq = 0, ldc = 0, ldi = 0;
-    size_t partial = 0, fold = 0, wq = 0, wv = 0, wg = 0, wb = 0, wk = 0, wr = 0, lp = 0, mh = 0, mS = 0, mo = 0;
+    size_t kv = 0, partial = 0, fold = 0, wq = 0, wv = 0, wg = 0, wb = 0, wk = 0, wr = 0, lp = 0, mh = 0, mS = 0, mo = 0;
     const size_t chunks = (N + MEMORY_CHUNK - 1) / MEMORY_CHUNK;
     for (const HybridLayer& L : hm.layers) {
         ldp = std::max(ldp, L.proj.m);
@@ -420,6 +427,7 @@ int32_t hybrid_alloc_scratch(wick_cuda_model* m) {
             ldq = std::max(ldq, s.heads * s.q_pitch());
             ldc = std::max(ldc, s.heads * s.ldc());
             lp = std::max(lp, latent_scratch(s, m->max_chunk));
+            if (L.ukv.w) kv = std::max(kv, latent_tc_keys(s, m->max_chunk, (int)c.max_seq_len) * latent_tc_cols(s));
             c.n_heads = std::max<uint32_t>(c.n_heads, s.heads);
             c.n_kv_heads = std::max<uint32_t>(c.n_kv_heads, 1);
         } else {
@@ -484,6 +492,7 @@ int32_t hybrid_alloc_scratch(wick_cuda_model* m) {
         W_TRY(act(&hm.qc, N * hm.ldc));
         W_TRY(act(&hm.oc, N * hm.ldc));
         W_TRY(dev_alloc(m, &hm.latent_partial, lp));
+        if (kv) W_TRY(act(&hm.kv, kv));
     }
     if (mh) {
         W_TRY(dev_alloc(m, &hm.gates, N * hm.ldi));

@@ -7,6 +7,8 @@
 #include <vector>
 
 #include "hybrid_kernels.cuh"
+#include "latent_kernels.cuh"
+#include "memory_kernels.cuh"
 #include "model_internal.cuh"
 #include "safetensors.hpp"
 
@@ -37,6 +39,7 @@ struct HybridLayer {
     DenseWeight a2, g2;  // low-rank up projections of the decay and the output gate
     float *conv_w = nullptr, *A_log = nullptr, *dt_bias = nullptr, *out_norm = nullptr;
     DenseWeight uq, uk_t, uv;  // latent: queries; per head to the latent's side [kv_rank][dim]; values [vdim][kv_rank]
+    DenseWeight ukv;           // keys and values of the prompt form (empty where that does not apply)
     DenseWeight gates;
     FeedForwardKind ff = FF_NONE;
     Activation act = ACT_RELU;
@@ -82,6 +85,7 @@ struct HybridModel {
     float* y = nullptr;        // [rows (x max_top)][ldw] sublayer output
     float *a = nullptr, *gate = nullptr;  // [rows][lda] decay projection, [rows][ldg] gate projection
     void *q = nullptr, *qc = nullptr, *oc = nullptr;  // act [rows][ldq], [rows][ldc]: latent queries, on the latent's side, read-outs
+    void* kv = nullptr;        // act: keys and values that a portion sees
     float* gates = nullptr;    // [rows][ldi] input and forget gate logits
     float* latent_partial = nullptr;
     MixAttnScratch attn;

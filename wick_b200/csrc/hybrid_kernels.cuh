@@ -244,73 +244,6 @@ void launch_gated_head_norm(cudaStream_t st, bool bf16, int n, int H, int E, flo
 void launch_delta_step(cudaStream_t st, bool bf16, const DeltaPrepArgs& a, const DeltaShape& s, const RowState& rs, const float* norm,
                        const float* gate, int ldg, void* out, int ldo);
 
-// ── latent attention ───────────────────────────────────────────────────────
-// Queries come through a latent of q_rank, keys and values through a latent of kv_rank that all heads share, beside rot_dim
-// key columns that carry the position.  Only the normalised latent and the rotated key part are cached, one row per position:
-//   [c: kv_rank, up to a multiple of 8 | rotated part: rot_dim, up to a multiple of 8]   (padding zero)
-// A query may be taken to the latent's side, q_c = W_uk^T q, so that its score is one product with a cache row and the weighted
-// sum of cache rows gives the value through W_uv ("absorbed"; decode, short portions, f32); or keys and values of the visible
-// positions are computed from the cache (prompts).  Softmax has one more entry per head, `sink`, without a value.
-struct LatentShape {
-    int heads = 0, dim = 0, rot_dim = 0, rot_dims = 0, vdim = 0, q_rank = 0, kv_rank = 0;
-    int size = 0;                  // sliding window (0: none): key j is seen by i when i - j < size
-    float scale = 1.0f, eps = 0.0f;
-    const float* sink = nullptr;   // [H]
-    const float2* rope = nullptr;  // [positions][rot_dims / 2] cos, sin of the first rot_dims of the rot_dim columns, in pairs
-    const float *q_norm = nullptr, *kv_norm = nullptr;
-    __host__ __device__ int ldc() const { return round_up(kv_rank, 8) + round_up(rot_dim, 8); }  // cache row
-    __host__ __device__ int off_rot() const { return round_up(kv_rank, 8); }
-    // a query row: per head [dim, up to a multiple of 8 | rot_dim, up to a multiple of 8]
-    __host__ __device__ int q_off_rot() const { return round_up(dim, 8); }
-    __host__ __device__ int q_pitch() const { return round_up(dim, 8) + round_up(rot_dim, 8); }
-    __host__ __device__ int off_kv() const { return round_up(q_rank, 8); }  // of the projections' row: [c_q | c, rotated part]
-    int seen(int max_seq) const { return size > 0 && size < max_seq ? size : max_seq; }
-};
-// Rows of p act [n][ldp]: c_q normalised in place, c normalised and the rotated part turned into the cache (state s0 / p0).
-void launch_latent_append(cudaStream_t st, bool bf16, void* p, int ldp, int n, const LatentShape& s, const RowState& rs);
-// Absorbed attention: qc act [n][H][ldc] (q taken to the latent's side in the first kv_rank columns of a head), q act [n][ldq]
-// (the rotated columns are read from here).  o act [n][H][ldo_h]: weighted sums of latents.  partial: latent_scratch() floats.
-size_t latent_scratch(const LatentShape& s, int max_rows);
-bool latent_supported(const LatentShape& s);
-cudaError_t launch_latent_attn(cudaStream_t st, bool bf16, const void* qc, const void* q, int ldq, int n, const LatentShape& s, const RowState& rs,
-                               void* o, int ldo_h, float* partial, int max_seq);
-
-// ── matrix memory ──────────────────────────────────────────────────────────
-// Per head, with log gates i, f and a running maximum m (log domain):
-//   m' = max(f + m, i);  S <- exp(f + m - m') S + exp(i - m') k v^T;  z likewise with v = 1
-//   o = S^T q / (max(|z . q|, exp(-m')) + 1e-6)
-// The state holds S^T and z together: s0 f32 [H][vdim + 1][dimp], z being the last row; s1 f32 [H]: m.
-struct MemoryShape {
-    int heads = 0, dim = 0, vdim = 0;
-    float cap = 1.0f, eps = 0.0f;
-    const float *i_bias = nullptr, *f_bias = nullptr, *norm = nullptr;  // [H], [H], [H * vdim]
-    __host__ __device__ int dimp() const { return round_up(dim, 32); }
-    __host__ __device__ int rows() const { return vdim + 1; }
-    size_t state_floats() const { return (size_t)heads * rows() * dimp(); }
-};
-constexpr int MEMORY_CHUNK = 64;
-constexpr int MEMORY_MAX_DIM = 4096;  // of keys and of values
-// Work memory for n tokens of one sequence.
-struct MemoryWork {
-    double *a = nullptr, *g = nullptr;                   // [H][n]: log weight of token j in token t's sum = a[t] + g[j] (same chunk)
-    float *carry = nullptr, *write = nullptr, *m = nullptr;  // [H][n]: weight of the chunk's first state; of token j in the next; m
-    float* keep = nullptr;                               // [H][chunks]: weight of the chunk's first state in the next
-    float* S = nullptr;                                  // [chunks][H][vdim + 1][dimp] states at the chunks' starts
-    float* o = nullptr;                                  // [n][H * vdim] read-outs
-};
-// Projections: q | k | v | g act columns of a row of p (ldp) in this order, gates f32 [n][ldi]: H input, then H forget logits.
-struct MemoryArgs {
-    const void* p = nullptr;
-    int ldp = 0;
-    const float* gates = nullptr;
-    int ldi = 0, n = 0;
-};
-// Consecutive tokens of one sequence: read-outs, normalised and gated, to out act [n][ldo].
-cudaError_t launch_memory_prompt(cudaStream_t st, bool bf16, const MemoryArgs& a, const MemoryShape& s, const RowState& rs, const MemoryWork& w,
-                                 void* out, int ldo);
-// One decode token per row.
-void launch_memory_step(cudaStream_t st, bool bf16, const MemoryArgs& a, const MemoryShape& s, const RowState& rs, void* out, int ldo);
-
 // ── launches that may start before their predecessor has finished ──────────
 // The kernels of a decode step are launched with programmatic stream serialisation: a kernel is brought up while the one before
 // it still runs, touches nothing but weights, and calls pdl_wait() before it reads or writes anything else.  Every kernel

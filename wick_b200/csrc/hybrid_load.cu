@@ -251,6 +251,17 @@ int32_t load_latent(const Loader& ld, const std::string& p, const JsonValue& mc,
         W_TRY(ld.put_matrix(host, H * C, s.dim, &L->uk_t));
     }
     W_TRY(ld.matrix(p + "uv", H * s.vdim, C, &L->uv));
+    if (ld.m->hybrid->bf16 && latent_tc_supported(s)) {  // keys and values of the prompt form
+        const int d8 = round_up(s.dim, 8), v8 = round_up(s.vdim, 8);
+        const SafeTensor &tk = ld.t.get(p + "uk", {H * s.dim, C}), &tv = ld.t.get(p + "uv", {H * s.vdim, C});
+        const size_t l = round_up(C, 8);
+        std::vector<uint16_t> host((size_t)latent_tc_cols(s) * l, 0);
+        for (int h = 0; h < H; h++) {
+            for (int d = 0; d < s.dim; d++) memcpy(&host[((size_t)h * d8 + d) * l], tk.data + (size_t)(h * s.dim + d) * C * 2, (size_t)C * 2);
+            for (int d = 0; d < s.vdim; d++) memcpy(&host[((size_t)H * d8 + h * v8 + d) * l], tv.data + (size_t)(h * s.vdim + d) * C * 2, (size_t)C * 2);
+        }
+        W_TRY(ld.put_matrix(host, latent_tc_cols(s), C, &L->ukv));
+    }
     W_TRY(ld.matrix(p + "o", width, H * s.vdim, &L->o));
     float *sink = nullptr, *qn = nullptr, *kn = nullptr;
     W_TRY(ld.vec(p + "sink", {H}, &sink));

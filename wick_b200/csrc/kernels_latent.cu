@@ -5,7 +5,7 @@
 // k_latent_attn    CTA (key split, row, group of heads): scores of a tile of cache rows, running softmax, weighted sum of the
 //                  tile's latents; f32 on the CUDA cores, any sizes.  A group's heads share every cache row that is read.
 // k_latent_sum     merges the key splits of a row and adds the sink's share of the denominator.
-#include "hybrid_kernels.cuh"
+#include "latent_kernels.cuh"
 
 namespace wick {
 

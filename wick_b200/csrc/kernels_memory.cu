@@ -14,7 +14,7 @@
 //   k_memory_out     per (chunk, head, tile of value channels): q S_0 and the chunk's own (q k^T) v, divided
 // The row of z rides along as one more value channel that is 1 for every token.
 // k_memory_step is the decode form: everything for one token of a (row, head), with the gated norm.
-#include "hybrid_kernels.cuh"
+#include "memory_kernels.cuh"
 
 namespace wick {
 

@@ -38,6 +38,13 @@ __device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap* map
         : "memory");
 }
 
+__device__ __forceinline__ void tma_load_3d(uint32_t dst, const CUtensorMap* map, uint32_t bar, int x, int y, int z) {
+    asm volatile(
+        "cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];" ::"r"(dst),
+        "l"((unsigned long long)map), "r"(bar), "r"(x), "r"(y), "r"(z)
+        : "memory");
+}
+
 // K-major operand tile, rows of 128 bytes, 128B swizzle: 8-row atoms 1024 bytes apart.
 __device__ __forceinline__ unsigned long long umma_desc_sw128(uint32_t smem_addr) {
     unsigned long long d = 0;
@@ -84,6 +91,14 @@ __device__ __forceinline__ void tmem_ld8(uint32_t taddr, int32_t* r) {
         : "r"(taddr)
         : "memory");
 }
+__device__ __forceinline__ void tmem_st16(uint32_t taddr, const int32_t* r) {
+    asm volatile(
+        "tcgen05.st.sync.aligned.32x32b.x16.b32 [%16], "
+        "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15};" ::"r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]),
+        "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(taddr)
+        : "memory");
+}
+__device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 __device__ __forceinline__ void tmem_ld_wait() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
 // cuTensorMapEncodeTiled through the runtime's entry-point lookup (the library does not link libcuda), NULL if absent.
 typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
@@ -101,6 +116,18 @@ inline EncodeTiledFn encode_tiled_fn() {
     });
     return fn;
 }
+
+// MN-major operand tile (k index down the rows, boxes of 64 columns = 128 bytes and `box_bytes`), 128B swizzle.
+__device__ __forceinline__ unsigned long long umma_desc_mn_sw128(uint32_t smem_addr, uint32_t box_bytes) {
+    unsigned long long d = 0;
+    d |= (unsigned long long)((smem_addr >> 4) & 0x3FFF);
+    d |= (unsigned long long)(box_bytes >> 4) << 16;   // next 64 columns
+    d |= (unsigned long long)(1024 >> 4) << 32;        // next 8 rows
+    d |= 1ull << 46;
+    d |= 2ull << 61;
+    return d;
+}
+constexpr uint32_t UMMA_A_MN = 1u << 15, UMMA_B_MN = 1u << 16;  // flags of the instruction descriptor
 
 // Wait with a limit of the order of a second (try_wait itself suspends for a while); false once it is reached or another
 // role of the CTA has given up.  Every lane of a warp may run the same wait.
@@ -139,6 +166,22 @@ inline cudaError_t encode_bf16_map(const void* base, int rows, int cols, int ld,
     cuuint32_t box[2] = {64, (cuuint32_t)box_rows};
     cuuint32_t estr[2] = {1, 1};
     CUresult r = fn(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
+                    CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                    CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    return r == CUDA_SUCCESS ? cudaSuccess : cudaErrorInvalidValue;
+}
+
+// The same for rows of `groups` pieces of `cols` columns, `pitch` elements apart (a multiple of 8): box of 64 columns of one
+// piece x box_rows rows, zero beyond the piece's columns.  Coordinates: column, piece, row.
+inline cudaError_t encode_bf16_map3(const void* base, int rows, int groups, int cols, int pitch, int ld, int box_rows, CUtensorMap* out) {
+    EncodeTiledFn fn = encode_tiled_fn();
+    if (!fn) return cudaErrorNotSupported;
+    if (((uintptr_t)base & 15) || ld % 8 || pitch % 8) return cudaErrorMisalignedAddress;
+    cuuint64_t dims[3] = {(cuuint64_t)cols, (cuuint64_t)groups, (cuuint64_t)rows};
+    cuuint64_t strides[2] = {(cuuint64_t)pitch * 2, (cuuint64_t)ld * 2};
+    cuuint32_t box[3] = {64, 1, (cuuint32_t)box_rows};
+    cuuint32_t estr[3] = {1, 1, 1};
+    CUresult r = fn(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr,
                     CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
                     CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     return r == CUDA_SUCCESS ? cudaSuccess : cudaErrorInvalidValue;
