@@ -18,7 +18,7 @@ _HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(_HERE, "csrc")
 LIB_PATH = os.path.join(_HERE, "libwick_cuda.so")
 SOURCES = ["kernels_basic.cu", "kernels_gemv.cu", "kernels_attn.cu", "kernels_q6k.cu", "kernels_batch.cu", "kernels_sample.cu", "tp_comm.cu", "decode_mega.cu", "gemm_tc.cu", "argmax_noalloc.cu",
-           "kernels_hyper.cu", "kernels_residual.cu", "kernels_dense.cu", "kernels_route.cu", "gemm_bf16.cu", "kernels_mixattn.cu", "attn_mix_tc.cu", "kernels_delta.cu", "delta_chunk.cu", "kernels_latent.cu", "attn_latent_tc.cu", "kernels_memory.cu", "hybrid_ops.cu", "hybrid_load.cu", "hybrid.cu", "wick_cuda.cu"]
+           "kernels_hyper.cu", "kernels_residual.cu", "kernels_dense.cu", "kernels_route.cu", "gemm_bf16.cu", "kernels_mixattn.cu", "attn_mix_tc.cu", "kernels_delta.cu", "delta_chunk.cu", "kernels_latent.cu", "attn_latent_step.cu", "attn_latent_tc.cu", "kernels_memory.cu", "hybrid_ops.cu", "hybrid_load.cu", "hybrid.cu", "wick_cuda.cu"]
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
@@ -54,16 +54,24 @@ def _newest(path: str, seen: set) -> float:
     return t
 
 
+def _read(path: str) -> str:
+    try:
+        with open(path) as f:
+            return f.read()
+    except OSError:
+        return ""
+
+
 def _inputs() -> dict:
     """Per source: newest modification time of what its object depends on."""
-    own = os.path.getmtime(__file__)
-    return {f: max(own, _newest(os.path.join(CSRC, f), set())) for f in SOURCES}
+    return {f: _newest(os.path.join(CSRC, f), set()) for f in SOURCES}
 
 
 def build(force: bool = False, verbose: bool = False, extra: List[str] | None = None) -> str:
     """Compiles what is out of date and links; safe to call from several processes at once."""
     srcs = _inputs()
     newest = max(srcs.values())
+    newest = max(newest, os.path.getmtime(__file__))
     if not force and os.path.exists(LIB_PATH) and os.path.getmtime(LIB_PATH) >= newest:
         return LIB_PATH
     objdir = os.path.join(_HERE, "build")
@@ -85,15 +93,16 @@ def _compile(objdir: str, srcs: dict, force: bool, verbose: bool, extra: List[st
     for src in SOURCES:
         obj = os.path.join(objdir, src.replace(".cu", ".o"))
         objs.append(obj)
-        if not force and os.path.exists(obj) and os.path.getmtime(obj) >= srcs[src]:
+        flags = " ".join([*NVCC_FLAGS, *SPLIT.get(src, []), *extra])
+        if not force and os.path.exists(obj) and os.path.getmtime(obj) >= srcs[src] and _read(obj + ".flags") == flags:
             continue
         part = f"{obj}.{os.getpid()}.part.o"
         cmd = [nvcc, "-ccbin", ccbin, *NVCC_FLAGS, *SPLIT.get(src, []), *extra, "-c", os.path.join(CSRC, src), "-o", part]
         if verbose:
             cmd.insert(1, "-Xptxas=-v")
-        procs.append((cmd, part, obj, subprocess.Popen(cmd, env=env, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)))
+        procs.append((cmd, part, obj, flags, subprocess.Popen(cmd, env=env, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)))
     failed = None
-    for cmd, part, obj, p in procs:
+    for cmd, part, obj, flags, p in procs:
         out, _ = p.communicate()
         if verbose or p.returncode:
             sys.stderr.write(out)
@@ -101,6 +110,8 @@ def _compile(objdir: str, srcs: dict, force: bool, verbose: bool, extra: List[st
             failed = failed or cmd
         else:
             os.replace(part, obj)
+            with open(obj + ".flags", "w") as f:
+                f.write(flags)
     if failed:
         raise RuntimeError("nvcc failed: " + " ".join(failed))
     part = f"{LIB_PATH}.{os.getpid()}.part"

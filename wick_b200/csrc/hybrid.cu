@@ -224,7 +224,7 @@ struct Step {
         }
         W_TRY(blocks(L.uk_t, s.kv_rank, hm.q, hm.ldq, s.q_pitch(), hm.qc, s.heads * s.ldc(), s.ldc()));
         mark(PC_GEMM);
-        CU_TRY(launch_latent_attn(m->stream, hm.bf16, hm.qc, hm.q, hm.ldq, n, s, rs, hm.oc, s.off_rot(), hm.latent_partial, (int)m->cfg.max_seq_len));
+        CU_TRY(launch_latent_attn(m->stream, hm.bf16, hm.qc, hm.q, hm.ldq, n, s, rs, hm.oc, s.off_rot(), hm.latent, (int)m->cfg.max_seq_len));
         mark(PC_ATTENTION);
         W_TRY(blocks(L.uv, s.vdim, hm.oc, s.heads * s.off_rot(), s.off_rot(), hm.mixed, hm.ldm, s.vdim));
         return WICK_CUDA_OK;
@@ -426,7 +426,7 @@ int32_t hybrid_alloc_scratch(wick_cuda_model* m) {
             const LatentShape& s = L.latent;
             ldq = std::max(ldq, s.heads * s.q_pitch());
             ldc = std::max(ldc, s.heads * s.ldc());
-            lp = std::max(lp, latent_scratch(s, m->max_chunk));
+            lp = std::max(lp, latent_scratch(s, hm.bf16, m->max_chunk, (int)c.max_seq_len));
             if (L.ukv.w) kv = std::max(kv, latent_tc_keys(s, m->max_chunk, (int)c.max_seq_len) * latent_tc_cols(s));
             c.n_heads = std::max<uint32_t>(c.n_heads, s.heads);
             c.n_kv_heads = std::max<uint32_t>(c.n_kv_heads, 1);
@@ -491,7 +491,7 @@ int32_t hybrid_alloc_scratch(wick_cuda_model* m) {
         W_TRY(act(&hm.q, N * hm.ldq));
         W_TRY(act(&hm.qc, N * hm.ldc));
         W_TRY(act(&hm.oc, N * hm.ldc));
-        W_TRY(dev_alloc(m, &hm.latent_partial, lp));
+        W_TRY(dev_alloc(m, &hm.latent.partial, lp));
         if (kv) W_TRY(act(&hm.kv, kv));
     }
     if (mh) {
@@ -512,7 +512,7 @@ int32_t hybrid_alloc_scratch(wick_cuda_model* m) {
     W_TRY(dev_alloc(m, &hm.rows_dev, N));
     W_TRY(dev_alloc(m, &m->tc_err, 1));
     CU_TRY(cudaMemset(m->tc_err, 0, 4));
-    hm.attn.err = m->tc_err;
+    hm.attn.err = hm.latent.err = m->tc_err;
     CU_TRY(cudaMallocHost((void**)&hm.h_rows, N * sizeof(int)));
     return WICK_CUDA_OK;
 }

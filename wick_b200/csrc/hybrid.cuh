@@ -87,7 +87,7 @@ struct HybridModel {
     void *q = nullptr, *qc = nullptr, *oc = nullptr;  // act [rows][ldq], [rows][ldc]: latent queries, on the latent's side, read-outs
     void* kv = nullptr;        // act: keys and values that a portion sees
     float* gates = nullptr;    // [rows][ldi] input and forget gate logits
-    float* latent_partial = nullptr;
+    LatentScratch latent;
     MixAttnScratch attn;
     DeltaWork work;
     MemoryWork memory;

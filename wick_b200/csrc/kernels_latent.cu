@@ -5,6 +5,7 @@
 // k_latent_attn    CTA (key split, row, group of heads): scores of a tile of cache rows, running softmax, weighted sum of the
 //                  tile's latents; f32 on the CUDA cores, any sizes.  A group's heads share every cache row that is read.
 // k_latent_sum     merges the key splits of a row and adds the sink's share of the denominator.
+// bfloat16 models take attn_latent_step.cu for the splits of a few tokens and attn_latent_tc.cu for prompts.
 #include "latent_kernels.cuh"
 
 namespace wick {
@@ -13,26 +14,28 @@ namespace {
 
 constexpr int LA_THREADS = 256, LA_KT = 32, LA_HEADS = 8;
 constexpr int LA_TARGET_CTAS = 296, LA_MAX_SPLIT = 64;
+constexpr int LA_STEP_ROWS = 128;  // rows per launch of the tensor-core form, for the size of its partial records
 constexpr size_t LA_SMEM_MAX = 200 * 1024;
 
+constexpr int AP_THREADS = 256;
+
 template <class T>
-__global__ void __launch_bounds__(128) k_latent_append(T* __restrict__ p, int ldp, const __grid_constant__ LatentShape s, const __grid_constant__ RowState rs) {
-    __shared__ float red[2][4];
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, j = blockIdx.x;
+__global__ void __launch_bounds__(AP_THREADS) k_latent_append(T* __restrict__ p, int ldp, const __grid_constant__ LatentShape s, const __grid_constant__ RowState rs) {
+    extern __shared__ float row[];  // c_q | c | rotated part
+    __shared__ float red[2][AP_THREADS / 32];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, j = blockIdx.x, Q = s.q_rank, C = s.kv_rank, skip = s.off_kv() - Q;
     pdl_launch_next();
     pdl_wait();
     const int pos = rs.pos(j);
     T* cq = p + (size_t)j * ldp;
-    const T* c = cq + s.off_kv();
     T* dst = (T*)rs.st0(j) + (size_t)pos * s.ldc();
     float qq = 0.0f, cc = 0.0f;
-    for (int i = tid; i < s.q_rank; i += 128) {
-        const float v = act_f(cq[i]);
-        qq = fmaf(v, v, qq);
-    }
-    for (int i = tid; i < s.kv_rank; i += 128) {
-        const float v = act_f(c[i]);
-        cc = fmaf(v, v, cc);
+#pragma unroll 4
+    for (int i = tid; i < Q + C + s.rot_dim; i += AP_THREADS) {
+        const float v = act_f(cq[i < Q ? i : i + skip]);
+        row[i] = v;
+        if (i < Q) qq = fmaf(v, v, qq);
+        else if (i < Q + C) cc = fmaf(v, v, cc);
     }
     qq = warp_sum(qq);
     cc = warp_sum(cc);
@@ -41,21 +44,28 @@ __global__ void __launch_bounds__(128) k_latent_append(T* __restrict__ p, int ld
         red[1][warp] = cc;
     }
     __syncthreads();
-    const float rq = 1.0f / sqrtf((red[0][0] + red[0][1] + red[0][2] + red[0][3]) / (float)s.q_rank + s.eps);
-    const float rc = 1.0f / sqrtf((red[1][0] + red[1][1] + red[1][2] + red[1][3]) / (float)s.kv_rank + s.eps);
-    for (int i = tid; i < s.q_rank; i += 128) cq[i] = f_act<T>(act_f(cq[i]) * rq * s.q_norm[i]);
+    qq = cc = 0.0f;
+#pragma unroll
+    for (int i = 0; i < AP_THREADS / 32; i++) {
+        qq += red[0][i];
+        cc += red[1][i];
+    }
+    const float rq = 1.0f / sqrtf(qq / (float)Q + s.eps), rc = 1.0f / sqrtf(cc / (float)C + s.eps);
+#pragma unroll 4
+    for (int i = tid; i < Q; i += AP_THREADS) cq[i] = f_act<T>(row[i] * rq * s.q_norm[i]);
     const int off = s.off_rot(), ldc = s.ldc();
-    for (int i = tid; i < ldc; i += 128) {
+    const float* r = row + Q + C;
+#pragma unroll 4
+    for (int i = tid; i < ldc; i += AP_THREADS) {
         float v = 0.0f;
-        if (i < s.kv_rank) {
-            v = act_f(c[i]) * rc * s.kv_norm[i];
+        if (i < C) {
+            v = row[Q + i] * rc * s.kv_norm[i];
         } else if (i >= off && i - off < s.rot_dim) {
             const int d = i - off;
-            const T* r = c + s.kv_rank;
-            v = act_f(r[d]);
+            v = r[d];
             if (d < s.rot_dims) {
                 const float2 cs = s.rope[(size_t)pos * (s.rot_dims / 2) + d / 2];
-                v = d % 2 == 0 ? v * cs.x - act_f(r[d + 1]) * cs.y : v * cs.x + act_f(r[d - 1]) * cs.y;
+                v = d % 2 == 0 ? v * cs.x - r[d + 1] * cs.y : v * cs.x + r[d - 1] * cs.y;
             }
         }
         dst[i] = f_act<T>(v);
@@ -162,36 +172,45 @@ __global__ void __launch_bounds__(LA_THREADS) k_latent_attn(const T* __restrict_
     }
 }
 
-// A CTA per (head, row).
+// A CTA per (head, row).  split_keys > 0: split i holds keys i * split_keys .. of the row, those past its last key are not there.
 template <class T>
-__global__ void __launch_bounds__(128) k_latent_sum(const float* __restrict__ partial, int splits, const __grid_constant__ LatentShape s, T* __restrict__ o, int ldo_h) {
-    const int C = s.kv_rank, h = blockIdx.x, H = s.heads, j = blockIdx.y, tid = threadIdx.x;
-    __shared__ float w[LA_MAX_SPLIT];
+__global__ void __launch_bounds__(256) k_latent_sum(const float* __restrict__ partial, int splits, int split_keys, const __grid_constant__ LatentShape s,
+                                                    const __grid_constant__ RowState rs, T* __restrict__ o, int ldo_h) {
+    const int C = s.kv_rank, h = blockIdx.x, H = s.heads, j = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    __shared__ float w[LATENT_MAX_SPLIT], red[2][8];
     pdl_launch_next();
     pdl_wait();
     const float* p = partial + ((size_t)j * H + h) * splits * (C + 2);
-    if (tid < 32) {
-        const float sink = s.sink[h];
-        float mx = sink;
-        for (int i = tid; i < splits; i += 32) mx = fmaxf(mx, p[(size_t)i * (C + 2) + C]);
-#pragma unroll
-        for (int x = 16; x > 0; x >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, x));
-        float den = 0.0f;
-        for (int i = tid; i < splits; i += 32) {
-            const float f = expf(p[(size_t)i * (C + 2) + C] - mx);
-            w[i] = f;
-            den = fmaf(f, p[(size_t)i * (C + 2) + C + 1], den);
-        }
-        den = warp_sum(den) + expf(sink - mx);
-        for (int i = tid; i < splits; i += 32) w[i] /= den;
+    int used = splits;
+    if (split_keys > 0) {
+        const int pos = rs.pos(j);
+        used = (pos - first_key(s, pos) + split_keys) / split_keys;
     }
+    // (log weights and the sink in units of log2 where the splits were made by the tensor-core form)
+    const float unit = split_keys > 0 ? 1.4426950408889634f : 1.0f, sink = s.sink[h] * unit;
+    float top = tid < used ? p[(size_t)tid * (C + 2) + C] : -INFINITY, sum = tid < used ? p[(size_t)tid * (C + 2) + C + 1] : 0.0f;
+    float mx = fmaxf(top, sink);
+#pragma unroll
+    for (int x = 16; x > 0; x >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, x));
+    if (lane == 0) red[0][warp] = mx;
     __syncthreads();
-    for (int c = tid; c < ldo_h; c += 128) {
+#pragma unroll
+    for (int i = 0; i < 8; i++) mx = fmaxf(mx, red[0][i]);
+    const float f = split_keys > 0 ? exp2f(top - mx) : expf(top - mx);
+    sum = warp_sum(sum * f);
+    if (lane == 0) red[1][warp] = sum;
+    if (tid < used) w[tid] = f;
+    __syncthreads();
+    float den = split_keys > 0 ? exp2f(sink - mx) : expf(sink - mx);
+#pragma unroll
+    for (int i = 0; i < 8; i++) den += red[1][i];
+    const float inv = 1.0f / den;
+    for (int c = tid; c < ldo_h; c += 256) {
         float a = 0.0f;
         if (c < C)
 #pragma unroll 8
-            for (int i = 0; i < splits; i++) a = fmaf(w[i], p[(size_t)i * (C + 2) + c], a);
-        o[((size_t)j * H + h) * ldo_h + c] = f_act<T>(a);
+            for (int i = 0; i < used; i++) a = fmaf(w[i], p[(size_t)i * (C + 2) + c], a);
+        o[((size_t)j * H + h) * ldo_h + c] = f_act<T>(a * inv);
     }
 }
 
@@ -205,6 +224,7 @@ int latent_splits(const LatentShape& s, int rows, int max_seq) {
 template <class T>
 cudaError_t latent_attn_go(cudaStream_t st, const void* qc, const void* q, int ldq, int n, const LatentShape& s, const RowState& rs, void* o, int ldo_h,
                            float* partial, int max_seq) {
+    static_assert(LA_MAX_SPLIT <= LATENT_MAX_SPLIT && LATENT_MAX_SPLIT <= 256, "a thread per split");
     const size_t smem = latent_smem(s);
     if (smem > 40 * 1024) {
         const cudaError_t e = cudaFuncSetAttribute(k_latent_attn<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -216,33 +236,58 @@ cudaError_t latent_attn_go(cudaStream_t st, const void* qc, const void* q, int l
                ldo_h, splits > 1 ? partial : nullptr);
     if (splits > 1) {
         g_kernel_launches++;
-        launch_pdl(k_latent_sum<T>, dim3(s.heads, n), dim3(128), 0, st, partial, splits, s, (T*)o, ldo_h);
+        launch_pdl(k_latent_sum<T>, dim3(s.heads, n), dim3(256), 0, st, partial, splits, 0, s, rs, (T*)o, ldo_h);
     }
     return cudaGetLastError();
 }
 
 }  // namespace
 
-bool latent_supported(const LatentShape& s) { return latent_smem(s) <= LA_SMEM_MAX; }
+bool latent_supported(const LatentShape& s) { return latent_smem(s) <= LA_SMEM_MAX && (size_t)(s.q_rank + s.kv_rank + s.rot_dim) * 4 <= LA_SMEM_MAX; }
 
-size_t latent_scratch(const LatentShape& s, int max_rows) {
+static int step_splits(const LatentShape& s, int max_seq) { return (s.seen(max_seq) + LATENT_STEP_KEYS - 1) / LATENT_STEP_KEYS; }
+
+size_t latent_scratch(const LatentShape& s, bool bf16, int max_rows, int max_seq) {
     const int groups = (s.heads + LA_HEADS - 1) / LA_HEADS;
     // rows * splits: splits <= target / (rows * groups), at least one
-    return (size_t)std::max(LA_TARGET_CTAS / groups + 1, max_rows) * s.heads * (s.kv_rank + 2);
+    size_t records = (size_t)std::max(LA_TARGET_CTAS / groups + 1, max_rows);
+    if (bf16 && latent_step_supported(s, max_seq)) records = (size_t)std::min(max_rows, LA_STEP_ROWS) * step_splits(s, max_seq);
+    return records * s.heads * (s.kv_rank + 2);
 }
 
 void launch_latent_append(cudaStream_t st, bool bf16, void* p, int ldp, int n, const LatentShape& s, const RowState& rs) {
     if (n <= 0) return;
+    const size_t smem = (size_t)(s.q_rank + s.kv_rank + s.rot_dim) * 4;
     g_kernel_launches++;
-    if (bf16) launch_pdl(k_latent_append<__nv_bfloat16>, dim3(n), dim3(128), 0, st, (__nv_bfloat16*)p, ldp, s, rs);
-    else launch_pdl(k_latent_append<float>, dim3(n), dim3(128), 0, st, (float*)p, ldp, s, rs);
+    auto go = [&](auto kernel, auto* rows) {
+        if (smem > 40 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        launch_pdl(kernel, dim3(n), dim3(AP_THREADS), smem, st, rows, ldp, s, rs);
+    };
+    if (bf16) go(k_latent_append<__nv_bfloat16>, (__nv_bfloat16*)p);
+    else go(k_latent_append<float>, (float*)p);
 }
 
 cudaError_t launch_latent_attn(cudaStream_t st, bool bf16, const void* qc, const void* q, int ldq, int n, const LatentShape& s, const RowState& rs,
-                               void* o, int ldo_h, float* partial, int max_seq) {
+                               void* o, int ldo_h, const LatentScratch& sc, int max_seq) {
     if (n <= 0) return cudaSuccess;
-    return bf16 ? latent_attn_go<__nv_bfloat16>(st, qc, q, ldq, n, s, rs, o, ldo_h, partial, max_seq)
-                : latent_attn_go<float>(st, qc, q, ldq, n, s, rs, o, ldo_h, partial, max_seq);
+    if (!bf16) return latent_attn_go<float>(st, qc, q, ldq, n, s, rs, o, ldo_h, sc.partial, max_seq);
+    using B = __nv_bfloat16;
+    if (!latent_step_supported(s, max_seq)) return latent_attn_go<B>(st, qc, q, ldq, n, s, rs, o, ldo_h, sc.partial, max_seq);
+    const int splits = step_splits(s, max_seq);
+    for (int r0 = 0; r0 < n; r0 += LA_STEP_ROWS) {
+        const int rows = std::min(LA_STEP_ROWS, n - r0);
+        RowState part = rs;
+        if (part.p0) part.p0 += r0;
+        if (part.positions) part.positions += r0;
+        part.start_pos += r0;
+        const cudaError_t e = launch_latent_step(st, (const B*)qc + (size_t)r0 * s.heads * s.ldc(), (const B*)q + (size_t)r0 * ldq, ldq, rows, s, part, sc.partial,
+                                                 splits, sc.err);
+        if (e != cudaSuccess) return e;
+        g_kernel_launches++;
+        launch_pdl(k_latent_sum<B>, dim3(s.heads, rows), dim3(256), 0, st, sc.partial, splits, LATENT_STEP_KEYS, s, part,
+                   (B*)o + (size_t)r0 * s.heads * ldo_h, ldo_h);
+    }
+    return cudaGetLastError();
 }
 
 }  // namespace wick

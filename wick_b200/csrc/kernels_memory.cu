@@ -14,9 +14,13 @@
 //   k_memory_out     per (chunk, head, tile of value channels): q S_0 and the chunk's own (q k^T) v, divided
 // The row of z rides along as one more value channel that is 1 for every token.
 // k_memory_step is the decode form: everything for one token of a (row, head), with the gated norm.
+#include <cooperative_groups.h>
+
 #include "memory_kernels.cuh"
 
 namespace wick {
+
+namespace cg = cooperative_groups;
 
 namespace {
 
@@ -281,15 +285,21 @@ __global__ void __launch_bounds__(256) k_memory_out(const T* __restrict__ p, int
 }
 
 // ── one decode token per row ───────────────────────────────────────────────
-// CTA (head, row): a warp per state row (value channel, or z), lanes over the key channels.
+// A cluster of CTAs per (head, row), each with a share of the state's rows (value channels, z last): a warp per state row, lanes
+// over the key channels.  The CTAs exchange z . q and the sums of squares of their read-outs through distributed shared memory.
+constexpr int MS_MAX_CLUSTER = 8;
+
 template <class T>
-__global__ void __launch_bounds__(1024) k_memory_step(const __grid_constant__ MemoryArgs a, const __grid_constant__ MemoryShape s, const __grid_constant__ RowState rs,
-                                                      T* __restrict__ out, int ldo) {
+__global__ void __launch_bounds__(512) k_memory_step(const __grid_constant__ MemoryArgs a, const __grid_constant__ MemoryShape s, const __grid_constant__ RowState rs,
+                                                     T* __restrict__ out, int ldo) {
     extern __shared__ __align__(16) float sm[];
-    const int H = s.heads, D = s.dim, E = s.vdim, DP = s.dimp(), h = blockIdx.x, j = blockIdx.y;
+    cg::cluster_group cluster = cg::this_cluster();
+    const int CL = (int)cluster.num_blocks(), rank = (int)cluster.block_rank();
+    const int H = s.heads, D = s.dim, E = s.vdim, DP = s.dimp(), h = blockIdx.x / CL, j = blockIdx.y;
     const int tid = threadIdx.x, nt = blockDim.x, lane = tid & 31, warp = tid >> 5, warps = nt / 32;
-    float *q = sm, *k = q + DP, *o = k + DP;  // o: [vdim + 1]
-    __shared__ float red[32];
+    const int share = (E + 1 + CL - 1) / CL, r0 = rank * share, r1 = min(r0 + share, E + 1);
+    float *q = sm, *k = q + DP, *o = k + DP;  // o: [share]
+    __shared__ float red[16], parts[2];       // parts: sum of squares of this CTA's read-outs, z . q (of the CTA that has z)
     pdl_launch_next();
     pdl_wait();
     const T* p = (const T*)a.p + (size_t)j * a.ldp;
@@ -304,9 +314,9 @@ __global__ void __launch_bounds__(1024) k_memory_step(const __grid_constant__ Me
         k[i] = i < D ? act_f(p[H * D + h * D + i]) * write : 0.0f;
     }
     __syncthreads();
-    if (tid == 0) *ms = m;  // (everyone has read it)
-#pragma unroll 2
-    for (int r = warp; r <= E; r += warps) {
+    float ss = 0.0f;
+#pragma unroll 4
+    for (int r = r0 + warp; r < r1; r += warps) {
         const float v = r < E ? act_f(p[2 * H * D + h * E + r]) : 1.0f;
         float* row = st + (size_t)r * DP;
         float acc = 0.0f;
@@ -318,23 +328,53 @@ __global__ void __launch_bounds__(1024) k_memory_step(const __grid_constant__ Me
             *reinterpret_cast<float4*>(row + i) = x;
         }
         acc = warp_sum(acc);
-        if (lane == 0) o[r] = acc;
+        if (lane == 0) {
+            if (r < E) o[r - r0] = acc;
+            else parts[1] = acc;
+        }
+        if (r < E) ss = fmaf(acc, acc, ss);
     }
-    __syncthreads();
-    const float den = fmaxf(fabsf(o[E]), expf(-m)) + 1e-6f;
-    float ss = 0.0f;
-    for (int i = tid; i < E; i += nt) {
-        const float v = o[i] / den;
-        ss = fmaf(v, v, ss);
-    }
-    ss = warp_sum(ss);
     if (lane == 0) red[warp] = ss;
     __syncthreads();
+    if (tid == 0) {
+        ss = 0.0f;
+        for (int i = 0; i < warps; i++) ss += red[i];
+        parts[0] = ss;
+    }
+    cluster.sync();
+    if (rank == 0 && tid == 0) *ms = m;  // (everyone has read it)
     ss = 0.0f;
-    for (int i = 0; i < warps; i++) ss += red[i];
-    const float r = 1.0f / sqrtf(ss / (float)E + s.eps);
-    for (int i = tid; i < E; i += nt)
-        out[(size_t)j * ldo + h * E + i] = f_act<T>(o[i] / den * r * s.norm[h * E + i] * sigmoid_f(act_f(p[2 * H * D + H * E + h * E + i])));
+    for (int i = 0; i < CL; i++) ss += *cluster.map_shared_rank(&parts[0], i);
+    const float zq = *cluster.map_shared_rank(&parts[1], E / share);
+    cluster.sync();  // a CTA's shared memory stays until everyone has read it
+    const float den = fmaxf(fabsf(zq), expf(-m)) + 1e-6f, inv = 1.0f / den;
+    const float r = inv / sqrtf(ss * inv * inv / (float)E + s.eps);
+    for (int i = r0 + tid; i < min(r1, E); i += nt)
+        out[(size_t)j * ldo + h * E + i] = f_act<T>(o[i - r0] * r * s.norm[h * E + i] * sigmoid_f(act_f(p[2 * H * D + H * E + h * E + i])));
+}
+
+template <class T>
+void memory_step_go(cudaStream_t st, const MemoryArgs& a, const MemoryShape& s, const RowState& rs, T* out, int ldo) {
+    int cl = 1;  // enough CTAs to keep the memory busy, at least 16 state rows each
+    while (cl < MS_MAX_CLUSTER && s.heads * a.n * cl < 148 && s.rows() / (2 * cl) >= 16) cl *= 2;
+    const int share = (s.rows() + cl - 1) / cl;
+    const int threads = std::min(512, std::max(128, round_up(share * 8, 128)));
+    const size_t smem = ((size_t)2 * s.dimp() + share) * 4;
+    if (smem > 40 * 1024) cudaFuncSetAttribute(k_memory_step<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(s.heads * cl, a.n);
+    cfg.blockDim = dim3(threads);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = st;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    attr[1].id = cudaLaunchAttributeClusterDimension;
+    attr[1].val.clusterDim.x = cl;
+    attr[1].val.clusterDim.y = attr[1].val.clusterDim.z = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = 2;
+    cudaLaunchKernelEx(&cfg, k_memory_step<T>, a, s, rs, out, ldo);
 }
 
 template <class T>
@@ -366,10 +406,8 @@ cudaError_t launch_memory_prompt(cudaStream_t st, bool bf16, const MemoryArgs& a
 void launch_memory_step(cudaStream_t st, bool bf16, const MemoryArgs& a, const MemoryShape& s, const RowState& rs, void* out, int ldo) {
     if (a.n <= 0) return;
     g_kernel_launches++;
-    const int threads = std::min(1024, std::max(128, round_up((s.vdim + 1) * 8, 128)));
-    const size_t smem = ((size_t)2 * s.dimp() + s.rows()) * 4;
-    if (bf16) launch_pdl(k_memory_step<__nv_bfloat16>, dim3(s.heads, a.n), dim3(threads), smem, st, a, s, rs, (__nv_bfloat16*)out, ldo);
-    else launch_pdl(k_memory_step<float>, dim3(s.heads, a.n), dim3(threads), smem, st, a, s, rs, (float*)out, ldo);
+    if (bf16) memory_step_go(st, a, s, rs, (__nv_bfloat16*)out, ldo);
+    else memory_step_go(st, a, s, rs, (float*)out, ldo);
 }
 
 }  // namespace wick

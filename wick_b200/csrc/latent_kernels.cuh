@@ -1,5 +1,4 @@
 // Launch wrappers of latent attention.
-//
 #pragma once
 #include "hybrid_kernels.cuh"
 
@@ -28,12 +27,22 @@ struct LatentShape {
 };
 // Rows of p act [n][ldp]: c_q normalised in place, c normalised and the rotated part turned into the cache (state s0 / p0).
 void launch_latent_append(cudaStream_t st, bool bf16, void* p, int ldp, int n, const LatentShape& s, const RowState& rs);
-// Absorbed attention: qc act [n][H][ldc] (q taken to the latent's side in the first kv_rank columns of a head), q act [n][ldq]
-// (the rotated columns are read from here).  o act [n][H][ldo_h]: weighted sums of latents.  partial: latent_scratch() floats.
-size_t latent_scratch(const LatentShape& s, int max_rows);
+// Absorbed attention: qc act [n][H][ldc] (q taken to the latent's side in the first kv_rank columns of a head, zero up to
+// off_rot), q act [n][ldq] (the rotated columns are read from here, before the rotation).  o act [n][H][ldo_h]: weighted sums of
+// latents.
+struct LatentScratch {
+    float* partial = nullptr;  // key splits: latent_scratch() floats
+    uint32_t* err = nullptr;   // device word for expired waits
+};
+size_t latent_scratch(const LatentShape& s, bool bf16, int max_rows, int max_seq);
 bool latent_supported(const LatentShape& s);
 cudaError_t launch_latent_attn(cudaStream_t st, bool bf16, const void* qc, const void* q, int ldq, int n, const LatentShape& s, const RowState& rs,
-                               void* o, int ldo_h, float* partial, int max_seq);
+                               void* o, int ldo_h, const LatentScratch& sc, int max_seq);
+// Its tensor-core form (attn_latent_step.cu), bf16: a split per LATENT_STEP_KEYS keys.
+constexpr int LATENT_STEP_KEYS = 64, LATENT_MAX_SPLIT = 256;
+bool latent_step_supported(const LatentShape& s, int max_seq);
+cudaError_t launch_latent_step(cudaStream_t st, const void* qc, const void* q, int ldq, int n, const LatentShape& s, const RowState& rs, float* partial,
+                               int splits, uint32_t* err);
 
 // The prompt form (attn_latent_tc.cu): consecutive bf16 tokens of one sequence; keys and values of the visible positions come
 // from the cache through ukv, whose rows are [H][dim, up to a multiple of 8] keys, then [H][vdim, up to a multiple of 8] values.
