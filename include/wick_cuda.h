@@ -296,8 +296,8 @@ int32_t wick_cuda_argmax(const float* logits_dev, uint32_t count, uint32_t* out_
 /* ---- operators of the config.json models ---------------------------------------
  * `compute` is WICK_CUDA_COMPUTE_BF16 or _F32: the type of the "act" buffers (bfloat16 or f32).  Row pitches (ld*) of act
  * buffers are multiples of 8 elements, bases 16-byte aligned; columns between the row's length and its length rounded up to 8
- * are read by dense and must be finite.  Device pointers, asynchronous on `stream`; dense and mix_attention synchronise it
- * to report expired device waits as WICK_CUDA_ERR_TIMEOUT. */
+ * are read by dense and must be finite.  Device pointers, asynchronous on `stream`; the ones that may wait on the device
+ * (dense, mix_attention, latent_attention, matrix_memory) synchronise it to report expired device waits as WICK_CUDA_ERR_TIMEOUT. */
 
 /* y[n][m] = activation(x[n][k] W[m][k]^T) with bfloat16 W (pitch ldw = k rounded up to 8, padding zero).  w_up_dev (optional,
  * same shape): y = activation(W x) * (W_up x).  softcap > 0: y = softcap tanh(y / softcap).  y is act, or f32 when y_f32 != 0.  path: AUTO, or
@@ -336,6 +336,43 @@ int32_t wick_cuda_channel_delta(int32_t compute, const void* proj_dev, uint32_t 
                                 const float* norm_dev, uint32_t n, uint32_t heads, uint32_t kv_heads, uint32_t dim, uint32_t vdim,
                                 uint32_t taps, float eps, float* state_dev, float* conv_state_dev, void* out_dev, uint32_t ldo,
                                 void* stream);
+
+/* One residual stream x [n][width] f32 with norms around the sublayers.  With y_dev (f32 rows of `width`; token j's output is the
+ * sum of rows j * y_parts .., or of rows y_rows_dev[j * y_parts] .., times y_scale): x <- x + post * rms(y), or, with shift_dev
+ * instead of post_dev, x <- y + shift.  Then h = gain * rms(x), or [x | x0] (gain_dev NULL, x0_dev f32 [n][width]), to row j of h,
+ * or to rows h_rows_dev[j * h_parts] ...  rms(z) = z / sqrt(mean(z^2) + eps). */
+int32_t wick_cuda_residual_norm(int32_t compute, float* x_dev, uint32_t n, uint32_t width, const float* y_dev, uint32_t y_parts,
+                                const int32_t* y_rows_dev, float y_scale, const float* post_dev, const float* shift_dev,
+                                const float* gain_dev, const float* x0_dev, float eps, void* h_dev, uint32_t ldh, uint32_t h_parts,
+                                const int32_t* h_rows_dev, void* stream);
+/* Latent attention with a sink over rows start_pos.. of one sequence.  p act [n][ldp]: the query latent (q_rank, normalised in
+ * place with weights q_norm), then, at q_rank rounded up to 8, the key / value latent (kv_rank) and rot_dim rotated columns.
+ * cache act [max_seq][kv_rank up to 8 | rot_dim up to 8] is appended to.  bfloat16 weights, pitches rounded up to 8:
+ *   uq [heads][dim up to 8 | rot_dim up to 8][q_rank]   queries (rows in the gaps zero)
+ *   uk_t [heads][kv_rank][dim], uv [heads][vdim][kv_rank]   keys (transposed) and values from the latent
+ *   ukv [heads][dim up to 8] keys, then [heads][vdim up to 8] values, [kv_rank]   for the prompt form (optional)
+ * rope f32 [max_seq][rot_dims / 2][cos, sin] turns neighbouring pairs of the first rot_dims rotated columns.  Key j is seen by
+ * query i when j <= i and (size == 0 or i - j < size).  Softmax of scale * q . k with one more entry `sink` [heads] that has no
+ * value.  form: AUTO, or one of the two (PROMPT: bfloat16, tcgen05).  out act [n][ldo]: heads * vdim. */
+#define WICK_CUDA_LATENT_AUTO 0
+#define WICK_CUDA_LATENT_ABSORBED 1
+#define WICK_CUDA_LATENT_PROMPT 2
+int32_t wick_cuda_latent_attention(int32_t compute, void* p_dev, uint32_t ldp, uint32_t n, uint32_t start_pos, void* cache_dev,
+                                   uint32_t max_seq, const void* uq_dev, const void* uk_t_dev, const void* uv_dev, const void* ukv_dev,
+                                   const float* sink_dev, const float* q_norm_dev, const float* kv_norm_dev, const float* rope_dev,
+                                   uint32_t heads, uint32_t dim, uint32_t rot_dim, uint32_t rot_dims, uint32_t vdim, uint32_t q_rank,
+                                   uint32_t kv_rank, uint32_t size, float scale, float eps, int32_t form, void* out_dev, uint32_t ldo,
+                                   void* stream);
+/* Matrix memory with exponential gates over n tokens of one sequence.  p act [n][ldp]: q | k (heads * dim each) | v | output gate
+ * (heads * vdim each); gates f32 [n][ldi]: input, then forget gate logits (heads each).  Per head i = cap tanh((in + i_bias) /
+ * cap), f = logsigmoid(cap tanh((fg + f_bias) / cap)), m' = max(f + m, i), S <- exp(f + m - m') S + exp(i - m') k v^T, z likewise
+ * with v = 1, o = S^T q dim^(-1/2) / (max(|z . q dim^(-1/2)|, exp(-m')) + 1e-6); out act [n][ldo] = rms(o) norm sigmoid(gate).  state
+ * f32 [heads][vdim + 1][dim rounded up to 32] (z last) and m f32 [heads] are read and updated.  step != 0: token by token with
+ * the decode kernel. */
+int32_t wick_cuda_matrix_memory(int32_t compute, const void* p_dev, uint32_t ldp, const float* gates_dev, uint32_t ldi, uint32_t n,
+                                uint32_t heads, uint32_t dim, uint32_t vdim, float cap, float eps, const float* i_bias_dev,
+                                const float* f_bias_dev, const float* norm_dev, float* state_dev, float* m_dev, int32_t step,
+                                void* out_dev, uint32_t ldo, void* stream);
 
 /* Split-K decode attention (opt-in).  The default single-query attention keeps the CPU path's one serial accumulation per
  * output dim over all cached keys (attn_values, cpu.rs:1463-1509), which is bit-exact and, at thousands of keys, slow.

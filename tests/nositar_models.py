@@ -64,17 +64,20 @@ def make_weights(cfg, seed=0, rank=10):
 
 
 def write_model(folder, cfg, weights):
-    """Writes the folder; returns the weights as the file holds them (f64 of the bfloat16 values)."""
+    """Writes the folder; returns the weights as the file holds them (f64 of the bfloat16 values; integer tables as they are)."""
     os.makedirs(folder, exist_ok=True)
     with open(os.path.join(folder, "config.json"), "w") as f:
         json.dump(cfg, f)
     head, blobs, at, back = {}, [], 0, {}
     for name, a in weights.items():
-        a = np.asarray(a, np.float32)
-        bits = to_bf16(a).reshape(a.shape)
-        back[name] = bf16_f64(bits.reshape(-1)).reshape(a.shape)
-        raw = bits.tobytes()
-        head[name] = {"dtype": "BF16", "shape": list(a.shape), "data_offsets": [at, at + len(raw)]}
+        a = np.asarray(a)
+        if a.dtype.kind == "i":
+            back[name], raw, kind = a, a.astype("<i4").tobytes(), "I32"
+        else:
+            bits = to_bf16(a).reshape(a.shape)
+            back[name] = bf16_f64(bits.reshape(-1)).reshape(a.shape)
+            raw, kind = bits.tobytes(), "BF16"
+        head[name] = {"dtype": kind, "shape": list(a.shape), "data_offsets": [at, at + len(raw)]}
         blobs.append(raw)
         at += len(raw)
     h = json.dumps(head).encode()

@@ -109,6 +109,10 @@ SIGNATURES = {
     "wick_cuda_hyper_norm": [_i32, _vp, _u32, _u32, _u32, _vp, _vp, _vp, _vp, _vp, _f, _vp, _u32, _vp],
     "wick_cuda_mix_attention": [_i32, _vp, _u32, _u32, _u32, _vp, _vp, _u32, _vp, _vp, _u32, _u32, _u32, _u32, _f, _f, _u32, _u32, _vp, _u32, _vp],
     "wick_cuda_channel_delta": [_i32, _vp, _u32, _u32, _vp, _vp, _vp, _vp, _vp, _vp, _u32, _u32, _u32, _u32, _u32, _u32, _f, _vp, _vp, _vp, _u32, _vp],
+    "wick_cuda_residual_norm": [_i32, _vp, _u32, _u32, _vp, _u32, _vp, _f, _vp, _vp, _vp, _vp, _f, _vp, _u32, _u32, _vp, _vp],
+    "wick_cuda_latent_attention": [_i32, _vp, _u32, _u32, _u32, _vp, _u32, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _u32, _u32, _u32, _u32, _u32, _u32, _u32, _u32,
+                                   _f, _f, _i32, _vp, _u32, _vp],
+    "wick_cuda_matrix_memory": [_i32, _vp, _u32, _vp, _u32, _u32, _u32, _u32, _u32, _f, _f, _vp, _vp, _vp, _vp, _vp, _i32, _vp, _u32, _vp],
     "wick_cuda_argmax": [_vp, _u32, _vp, _vp],
     "wick_cuda_argmax_noalloc": [_vp, _u32, _vp, _vp],
 }

@@ -238,7 +238,7 @@ struct Step {
         MemoryArgs a;
         a.p = hm.proj; a.ldp = hm.ldp; a.gates = hm.gates; a.ldi = hm.ldi; a.n = n;
         if (rs.separate()) launch_memory_step(m->stream, hm.bf16, a, L.memory, rs, hm.mixed, hm.ldm);
-        else CU_TRY(launch_memory_prompt(m->stream, hm.bf16, a, L.memory, rs, hm.memory, hm.mixed, hm.ldm));
+        else CU_TRY(launch_memory_prompt(m->stream, hm.bf16, a, L.memory, rs, memory_work(L.memory, hm.bf16, n, hm.memory, m->tc_err), hm.mixed, hm.ldm));
         mark(PC_RECURRENCE);
         return WICK_CUDA_OK;
     }
@@ -398,8 +398,7 @@ int32_t hybrid_alloc_scratch(wick_cuda_model* m) {
     const size_t act_bytes = hm.bf16 ? 2 : 4, N = (size_t)m->max_chunk;
     const int streams = std::max(hm.streams, 1);
     int ldp = 8, ldm = 8, ldf = 8, lda = 0, ldg = 0, ldq = 0, ldc = 0, ldi = 0;
-    size_t kv = 0, partial = 0, fold = 0, wq = 0, wv = 0, wg = 0, wb = 0, wk = 0, wr = 0, lp = 0, mh = 0, mS = 0, mo = 0;
-    const size_t chunks = (N + MEMORY_CHUNK - 1) / MEMORY_CHUNK;
+    size_t kv = 0, partial = 0, fold = 0, wq = 0, wv = 0, wg = 0, wb = 0, wk = 0, wr = 0, lp = 0, mem = 0;
     for (const HybridLayer& L : hm.layers) {
         ldp = std::max(ldp, L.proj.m);
         ldm = std::max(ldm, L.o.k);
@@ -433,9 +432,7 @@ int32_t hybrid_alloc_scratch(wick_cuda_model* m) {
         } else {
             const MemoryShape& s = L.memory;
             ldi = std::max(ldi, 2 * s.heads);
-            mh = std::max(mh, (size_t)s.heads);
-            mS = std::max(mS, s.state_floats());
-            mo = std::max(mo, (size_t)s.heads * s.vdim);
+            mem = std::max(mem, memory_work_bytes(s, hm.bf16, m->max_chunk));
             c.n_heads = std::max<uint32_t>(c.n_heads, s.heads);
         }
         if (L.ff != FF_NONE) {
@@ -494,16 +491,9 @@ int32_t hybrid_alloc_scratch(wick_cuda_model* m) {
         W_TRY(dev_alloc(m, &hm.latent.partial, lp));
         if (kv) W_TRY(act(&hm.kv, kv));
     }
-    if (mh) {
+    if (mem) {
         W_TRY(dev_alloc(m, &hm.gates, N * hm.ldi));
-        W_TRY(dev_alloc(m, &hm.memory.a, N * mh));
-        W_TRY(dev_alloc(m, &hm.memory.g, N * mh));
-        W_TRY(dev_alloc(m, &hm.memory.carry, N * mh));
-        W_TRY(dev_alloc(m, &hm.memory.write, N * mh));
-        W_TRY(dev_alloc(m, &hm.memory.m, N * mh));
-        W_TRY(dev_alloc(m, &hm.memory.keep, chunks * mh));
-        W_TRY(dev_alloc(m, &hm.memory.S, chunks * mS));
-        W_TRY(dev_alloc(m, &hm.memory.o, N * mo));
+        W_TRY(dev_alloc(m, (uint8_t**)&hm.memory, mem));
     }
     for (RouteJob& r : hm.routes) {
         W_TRY(dev_alloc(m, &r.inv, N * r.top));

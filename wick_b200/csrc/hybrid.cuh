@@ -90,7 +90,7 @@ struct HybridModel {
     LatentScratch latent;
     MixAttnScratch attn;
     DeltaWork work;
-    MemoryWork memory;
+    void* memory = nullptr;    // work memory of the matrix memory
     int* rows_dev = nullptr;   // rows of a chunk that get logits
     int* h_rows = nullptr;     // pinned staging of the same
     ~HybridModel();

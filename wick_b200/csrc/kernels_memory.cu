@@ -16,6 +16,8 @@
 // k_memory_step is the decode form: everything for one token of a (row, head), with the gated norm.
 #include <cooperative_groups.h>
 
+#include <type_traits>
+
 #include "memory_kernels.cuh"
 
 namespace wick {
@@ -391,6 +393,35 @@ cudaError_t memory_prompt_go(cudaStream_t st, const MemoryArgs& a, const MemoryS
 }
 
 }  // namespace
+
+// One walk over the parts of the work memory: sizes, or (base given) pointers.
+static size_t carve(const MemoryShape& s, int n, uint8_t* base, MemoryWork* w) {
+    const size_t N = (size_t)n, H = s.heads, chunks = (N + MC - 1) / MC;
+    size_t at = 0;
+    auto take = [&](auto** out, size_t count) {
+        *out = (std::remove_reference_t<decltype(*out)>)(base ? base + at : nullptr);
+        at += (count * sizeof(**out) + 255) / 256 * 256;
+    };
+    take(&w->a, N * H);
+    take(&w->g, N * H);
+    take(&w->carry, N * H);
+    take(&w->write, N * H);
+    take(&w->m, N * H);
+    take(&w->keep, chunks * H);
+    take(&w->S, chunks * s.state_floats());
+    take(&w->o, N * H * s.vdim);
+    return at;
+}
+size_t memory_work_bytes(const MemoryShape& s, bool, int n) {
+    MemoryWork w;
+    return carve(s, n, nullptr, &w);
+}
+MemoryWork memory_work(const MemoryShape& s, bool, int n, void* base, uint32_t* err) {
+    MemoryWork w;
+    carve(s, n, (uint8_t*)base, &w);
+    w.err = err;
+    return w;
+}
 
 cudaError_t launch_memory_prompt(cudaStream_t st, bool bf16, const MemoryArgs& a, const MemoryShape& s, const RowState& rs, const MemoryWork& w,
                                  void* out, int ldo) {

@@ -1,5 +1,4 @@
 // Launch wrappers of the matrix memory with exponential gates.
-//
 #pragma once
 #include "hybrid_kernels.cuh"
 
@@ -19,14 +18,17 @@ struct MemoryShape {
 };
 constexpr int MEMORY_CHUNK = 64;
 constexpr int MEMORY_MAX_DIM = 4096;  // of keys and of values
-// Work memory for n tokens of one sequence.
+// Work memory for n tokens of one sequence, carved out of one allocation of memory_work_bytes().
 struct MemoryWork {
     double *a = nullptr, *g = nullptr;                   // [H][n]: log weight of token j in token t's sum = a[t] + g[j] (same chunk)
     float *carry = nullptr, *write = nullptr, *m = nullptr;  // [H][n]: weight of the chunk's first state; of token j in the next; m
     float* keep = nullptr;                               // [H][chunks]: weight of the chunk's first state in the next
     float* S = nullptr;                                  // [chunks][H][vdim + 1][dimp] states at the chunks' starts
     float* o = nullptr;                                  // [n][H * vdim] read-outs
+    uint32_t* err = nullptr;                             // device word for expired waits
 };
+size_t memory_work_bytes(const MemoryShape& s, bool bf16, int n);
+MemoryWork memory_work(const MemoryShape& s, bool bf16, int n, void* base, uint32_t* err);
 // Projections: q | k | v | g act columns of a row of p (ldp) in this order, gates f32 [n][ldi]: H input, then H forget logits.
 struct MemoryArgs {
     const void* p = nullptr;

@@ -231,6 +231,64 @@ def channel_delta(proj: torch.Tensor, off_beta: int, decay: torch.Tensor, gate: 
     return out
 
 
+def residual_norm(x: torch.Tensor, eps: float, gain=None, x0=None, y=None, post=None, shift=None, y_rows=None, y_parts: int = 1, y_scale: float = 1.0,
+                  h_rows=None, h_parts: int = 1, dtype=torch.float32) -> torch.Tensor:
+    """Residual update (in place on x [n, width] f32) and the next sublayer's input: [n, width], or [n, 2 width] with x0."""
+    n, w = x.shape
+    wide = w if gain is not None else 2 * w
+    h = torch.zeros((n * h_parts if h_rows is not None else n, wide + -wide % 8), dtype=dtype, device=x.device)
+    check(_lib.load().wick_cuda_residual_norm(_compute(h), _ptr(x), n, w, _opt(y), y_parts, _opt(y_rows), y_scale, _opt(post), _opt(shift), _opt(gain), _opt(x0),
+                                              eps, _ptr(h), h.shape[1], h_parts, _opt(h_rows), _stream()))
+    return h[:, :wide]
+
+
+def _up8(n: int) -> int:
+    return n + -n % 8
+
+
+def latent_weights(uq: torch.Tensor, uk: torch.Tensor, uv: torch.Tensor, heads: int, dim: int, rot_dim: int, vdim: int):
+    """The layouts that latent_attention takes, from uq [heads * (dim + rot_dim), q_rank], uk [heads * dim, kv_rank] and
+    uv [heads * vdim, kv_rank] (bfloat16)."""
+    d8, r8, v8, c = _up8(dim), _up8(rot_dim), _up8(vdim), uk.shape[1]
+    q = uq.new_zeros((heads, d8 + r8, _up8(uq.shape[1])))
+    u = uq.view(heads, dim + rot_dim, -1)
+    q[:, :dim, :uq.shape[1]] = u[:, :dim]
+    q[:, d8:d8 + rot_dim, :uq.shape[1]] = u[:, dim:]
+    k_t = pad8(uk.view(heads, dim, c).transpose(1, 2))
+    kv = uk.new_zeros((heads * (d8 + v8), _up8(c)))
+    kv[:heads * d8].view(heads, d8, -1)[:, :dim, :c] = uk.view(heads, dim, c)
+    kv[heads * d8:].view(heads, v8, -1)[:, :vdim, :c] = uv.view(heads, vdim, c)
+    return q, k_t, pad8(uv), kv
+
+
+_LATENT_FORMS = {"auto": 0, "absorbed": 1, "prompt": 2}
+
+
+def latent_attention(p: torch.Tensor, cache: torch.Tensor, start_pos: int, weights, sink, q_norm, kv_norm, rope, heads: int, dim: int, rot_dim: int,
+                     rot_dims: int, vdim: int, q_rank: int, kv_rank: int, size: int, scale: float, eps: float, form: str = "auto") -> torch.Tensor:
+    """Latent attention with a sink; p [n, q_rank up to 8 | kv_rank | rot_dim] (its query latent is normalised in place in a copy),
+    weights from latent_weights(); appends to cache [max_seq, kv_rank up to 8 | rot_dim up to 8]."""
+    p8, n = pad8(p), p.shape[0]
+    if p8.data_ptr() == p.data_ptr():
+        p8 = p8.clone()
+    uq, uk_t, uv, ukv = weights
+    out = torch.zeros((n, _up8(heads * vdim)), dtype=p.dtype, device=p.device)
+    check(_lib.load().wick_cuda_latent_attention(_compute(p), _ptr(p8), p8.shape[1], n, start_pos, _ptr(cache), cache.shape[0], _ptr(uq), _ptr(uk_t), _ptr(uv),
+                                                 _ptr(ukv) if p.dtype == torch.bfloat16 else None, _ptr(sink), _ptr(q_norm), _ptr(kv_norm), _ptr(rope), heads, dim,
+                                                 rot_dim, rot_dims, vdim, q_rank, kv_rank, size, scale, eps, _LATENT_FORMS[form], _ptr(out), out.shape[1], _stream()))
+    return out[:, :heads * vdim]
+
+
+def matrix_memory(p: torch.Tensor, gates: torch.Tensor, i_bias, f_bias, norm, heads: int, dim: int, vdim: int, cap: float, eps: float,
+                  state: torch.Tensor, m: torch.Tensor, step: bool = False) -> torch.Tensor:
+    """Matrix memory with exponential gates, gated output norm; state [heads, vdim + 1, dim up to 32] and m [heads] are updated."""
+    n, p8 = p.shape[0], pad8(p)
+    out = torch.zeros((n, _up8(heads * vdim)), dtype=p.dtype, device=p.device)
+    check(_lib.load().wick_cuda_matrix_memory(_compute(p), _ptr(p8), p8.shape[1], _ptr(gates), gates.shape[1], n, heads, dim, vdim, cap, eps, _ptr(i_bias),
+                                              _ptr(f_bias), _ptr(norm), _ptr(state), _ptr(m), int(step), _ptr(out), out.shape[1], _stream()))
+    return out[:, :heads * vdim]
+
+
 def argmax(logits: torch.Tensor) -> torch.Tensor:
     out = torch.empty(1, dtype=torch.int32, device=logits.device)
     check(_lib.load().wick_cuda_argmax(_ptr(logits), logits.numel(), _ptr(out), _stream()))
