@@ -18,7 +18,7 @@ _HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(_HERE, "csrc")
 LIB_PATH = os.path.join(_HERE, "libwick_cuda.so")
 SOURCES = ["kernels_basic.cu", "kernels_gemv.cu", "kernels_attn.cu", "kernels_q6k.cu", "kernels_batch.cu", "kernels_sample.cu", "tp_comm.cu", "decode_mega.cu", "gemm_tc.cu", "argmax_noalloc.cu",
-           "kernels_hyper.cu", "kernels_residual.cu", "kernels_dense.cu", "kernels_route.cu", "gemm_bf16.cu", "kernels_mixattn.cu", "attn_mix_tc.cu", "kernels_delta.cu", "delta_chunk.cu", "kernels_latent.cu", "attn_latent_step.cu", "attn_latent_tc.cu", "kernels_memory.cu", "hybrid_ops.cu", "hybrid_load.cu", "hybrid.cu", "wick_cuda.cu"]
+           "kernels_hyper.cu", "kernels_residual.cu", "kernels_dense.cu", "kernels_route.cu", "gemm_bf16.cu", "kernels_mixattn.cu", "attn_mix_tc.cu", "kernels_delta.cu", "delta_chunk.cu", "kernels_latent.cu", "attn_latent_step.cu", "attn_latent_tc.cu", "kernels_memory.cu", "memory_tc.cu", "hybrid_ops.cu", "hybrid_load.cu", "hybrid.cu", "wick_cuda.cu"]
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",

@@ -12,6 +12,7 @@
 //   k_memory_states  per (chunk, head, tile of value channels): sum_j w_j k_j v_j^T
 //   k_memory_scan    per state element: states at the chunks' starts, and the final one
 //   k_memory_out     per (chunk, head, tile of value channels): q S_0 and the chunk's own (q k^T) v, divided
+// (bfloat16 models: memory_tc.cu does the last three on the tensor cores.)
 // The row of z rides along as one more value channel that is 1 for every token.
 // k_memory_step is the decode form: everything for one token of a (row, head), with the gated norm.
 #include <cooperative_groups.h>
@@ -39,54 +40,57 @@ __device__ __forceinline__ Gates memory_gates(const MemoryShape& s, const float*
     return g;
 }
 
-// A CTA per head; a warp per chunk, two tokens per lane.
+// A CTA per head; a warp per chunk of 32 TPL tokens.
 constexpr int GT_THREADS = 512, GT_MAX_CHUNKS = 512;
 
 __device__ __forceinline__ double shfl_up(double v, int o) { return __shfl_up_sync(0xffffffffu, v, o); }
 
+template <int TPL>
 __global__ void __launch_bounds__(GT_THREADS) k_memory_gates(const float* __restrict__ gates, int ldi, int n, const __grid_constant__ MemoryShape s,
                                                              float* __restrict__ m_state, const __grid_constant__ MemoryWork w) {
-    static_assert(MC == 64, "two tokens per lane");
+    constexpr int L = 32 * TPL;
     __shared__ double last_b[GT_MAX_CHUNKS], last_g[GT_MAX_CHUNKS];  // b and max(i - b) of whole chunks
     __shared__ float m0[GT_MAX_CHUNKS + 1];
-    const int h = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, chunks = (n + MC - 1) / MC;
+    const int h = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, chunks = (n + L - 1) / L;
     double* ga = w.a + (size_t)h * n;
     double* gg = w.g + (size_t)h * n;
     for (int c = warp; c < chunks; c += GT_THREADS / 32) {
-        double f[2], g[2];
-        float in[2];
+        double b[TPL], g[TPL], sum = 0.0;
 #pragma unroll
-        for (int x = 0; x < 2; x++) {
-            const int t = c * MC + 2 * lane + x;
+        for (int x = 0; x < TPL; x++) {
+            const int t = c * L + TPL * lane + x;
             Gates v = {-INFINITY, 0.0f};
             if (t < n) v = memory_gates(s, gates + (size_t)t * ldi, h);
-            f[x] = v.f;
-            in[x] = v.i;
+            b[x] = sum += (double)v.f;
+            g[x] = v.i;
         }
-        double b = f[0] + f[1];
+        double all = sum;
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
-            const double u = shfl_up(b, o);
-            if (lane >= o) b += u;
+            const double u = shfl_up(all, o);
+            if (lane >= o) all += u;
         }
-        const double b1 = b, b0 = b - f[1];
-        g[0] = (double)in[0] - b0;
-        g[1] = (double)in[1] - b1;
-        double mx = fmax(g[0], g[1]);
+        double mx = -INFINITY;
+#pragma unroll
+        for (int x = 0; x < TPL; x++) {
+            b[x] += all - sum;
+            g[x] -= b[x];
+            mx = fmax(mx, g[x]);
+        }
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
             const double u = shfl_up(mx, o);
             if (lane >= o) mx = fmax(mx, u);
         }
         if (lane == 31) {
-            last_b[c] = b1;
+            last_b[c] = b[TPL - 1];
             last_g[c] = mx;
         }
 #pragma unroll
-        for (int x = 0; x < 2; x++) {  // a: b for now
-            const int t = c * MC + 2 * lane + x;
+        for (int x = 0; x < TPL; x++) {  // a: b for now
+            const int t = c * L + TPL * lane + x;
             if (t < n) {
-                ga[t] = x ? b1 : b0;
+                ga[t] = b[x];
                 gg[t] = g[x];
             }
         }
@@ -103,14 +107,14 @@ __global__ void __launch_bounds__(GT_THREADS) k_memory_gates(const float* __rest
     }
     __syncthreads();
     for (int c = warp; c < chunks; c += GT_THREADS / 32) {
-        double b[2], g[2];
+        double b[TPL], g[TPL], mx = -INFINITY;
 #pragma unroll
-        for (int x = 0; x < 2; x++) {
-            const int t = c * MC + 2 * lane + x;
+        for (int x = 0; x < TPL; x++) {
+            const int t = c * L + TPL * lane + x;
             b[x] = t < n ? ga[t] : 0.0;
             g[x] = t < n ? gg[t] : -INFINITY;
+            mx = fmax(mx, g[x]);
         }
-        double mx = fmax(g[0], g[1]);
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
             const double u = shfl_up(mx, o);
@@ -120,8 +124,8 @@ __global__ void __launch_bounds__(GT_THREADS) k_memory_gates(const float* __rest
         if (lane == 0) before = -INFINITY;
         const double first = m0[c];
 #pragma unroll
-        for (int x = 0; x < 2; x++) {
-            const int t = c * MC + 2 * lane + x;
+        for (int x = 0; x < TPL; x++) {
+            const int t = c * L + TPL * lane + x;
             before = fmax(before, g[x]);
             if (t < n) {
                 const float m = (float)(b[x] + fmax(first, before));
@@ -182,14 +186,24 @@ __global__ void __launch_bounds__(256) k_memory_scan(int chunks, const __grid_co
     float4* st = reinterpret_cast<float4*>(state) + (size_t)h * per4 + i;
     float4* S = reinterpret_cast<float4*>(w.S) + (size_t)h * per4 + i;
     const size_t step = (size_t)s.heads * per4;
-    const float* keep = w.keep + (size_t)h * chunks;
+    const float* __restrict__ keep = w.keep + (size_t)h * chunks;
     float4 cur = *st;
-#pragma unroll 4
-    for (int c = 0; c < chunks; c++) {
-        const float4 d = S[c * step];
-        const float k = keep[c];
-        S[c * step] = cur;
-        cur = make_float4(fmaf(cur.x, k, d.x), fmaf(cur.y, k, d.y), fmaf(cur.z, k, d.z), fmaf(cur.w, k, d.w));
+    constexpr int SB = 4;  // chunks in flight
+    for (int c0 = 0; c0 < chunks; c0 += SB) {
+        float4 d[SB];
+        float k[SB];
+#pragma unroll
+        for (int c = 0; c < SB; c++)
+            if (c0 + c < chunks) {
+                d[c] = S[(c0 + c) * step];
+                k[c] = keep[c0 + c];
+            }
+#pragma unroll
+        for (int c = 0; c < SB; c++)
+            if (c0 + c < chunks) {
+                S[(c0 + c) * step] = cur;
+                cur = make_float4(fmaf(cur.x, k[c], d[c].x), fmaf(cur.y, k[c], d[c].y), fmaf(cur.z, k[c], d[c].z), fmaf(cur.w, k[c], d[c].w));
+            }
     }
     *st = cur;
 }
@@ -384,7 +398,7 @@ cudaError_t memory_prompt_go(cudaStream_t st, const MemoryArgs& a, const MemoryS
     const int chunks = (a.n + MC - 1) / MC;
     if (chunks > GT_MAX_CHUNKS) return cudaErrorInvalidValue;
     g_kernel_launches += 4;
-    k_memory_gates<<<s.heads, GT_THREADS, 0, st>>>(a.gates, a.ldi, a.n, s, (float*)rs.s1, w);
+    k_memory_gates<MC / 32><<<s.heads, GT_THREADS, 0, st>>>(a.gates, a.ldi, a.n, s, (float*)rs.s1, w);
     const int vt = (s.rows() + TV - 1) / TV, dt = (s.dimp() + TV - 1) / TV;
     k_memory_states<T><<<dim3(vt * dt, s.heads, chunks), 256, 0, st>>>((const T*)a.p, a.ldp, a.n, s, w);
     k_memory_scan<<<dim3((s.rows() * s.dimp() / 4 + 255) / 256, s.heads), 256, 0, st>>>(chunks, s, (float*)rs.s0, w);
@@ -394,9 +408,12 @@ cudaError_t memory_prompt_go(cudaStream_t st, const MemoryArgs& a, const MemoryS
 
 }  // namespace
 
+static bool use_tc(const MemoryShape& s, bool bf16, int n) { return bf16 && n >= MEMORY_TC_MIN_ROWS && memory_tc_supported(s); }
+
 // One walk over the parts of the work memory: sizes, or (base given) pointers.
-static size_t carve(const MemoryShape& s, int n, uint8_t* base, MemoryWork* w) {
-    const size_t N = (size_t)n, H = s.heads, chunks = (N + MC - 1) / MC;
+static size_t carve(const MemoryShape& s, bool bf16, int n, uint8_t* base, MemoryWork* w) {
+    const bool tc = use_tc(s, bf16, n);
+    const size_t N = (size_t)n, H = s.heads, L = tc ? MEMORY_TC_CHUNK : MC, chunks = (N + L - 1) / L;
     size_t at = 0;
     auto take = [&](auto** out, size_t count) {
         *out = (std::remove_reference_t<decltype(*out)>)(base ? base + at : nullptr);
@@ -409,16 +426,22 @@ static size_t carve(const MemoryShape& s, int n, uint8_t* base, MemoryWork* w) {
     take(&w->m, N * H);
     take(&w->keep, chunks * H);
     take(&w->S, chunks * s.state_floats());
+    if (tc) {
+        take((__nv_bfloat16**)&w->S_hi, chunks * s.state_floats());
+        take((__nv_bfloat16**)&w->S_lo, chunks * s.state_floats());
+    }
     take(&w->o, N * H * s.vdim);
     return at;
 }
-size_t memory_work_bytes(const MemoryShape& s, bool, int n) {
+size_t memory_work_bytes(const MemoryShape& s, bool bf16, int n) {
     MemoryWork w;
-    return carve(s, n, nullptr, &w);
+    size_t bytes = carve(s, bf16, n, nullptr, &w);
+    if (use_tc(s, bf16, n)) bytes = std::max(bytes, carve(s, bf16, MEMORY_TC_MIN_ROWS - 1, nullptr, &w));  // shorter portions take the other form
+    return bytes;
 }
-MemoryWork memory_work(const MemoryShape& s, bool, int n, void* base, uint32_t* err) {
+MemoryWork memory_work(const MemoryShape& s, bool bf16, int n, void* base, uint32_t* err) {
     MemoryWork w;
-    carve(s, n, (uint8_t*)base, &w);
+    carve(s, bf16, n, (uint8_t*)base, &w);
     w.err = err;
     return w;
 }
@@ -426,7 +449,15 @@ MemoryWork memory_work(const MemoryShape& s, bool, int n, void* base, uint32_t* 
 cudaError_t launch_memory_prompt(cudaStream_t st, bool bf16, const MemoryArgs& a, const MemoryShape& s, const RowState& rs, const MemoryWork& w,
                                  void* out, int ldo) {
     if (a.n <= 0) return cudaSuccess;
-    const cudaError_t e = bf16 ? memory_prompt_go<__nv_bfloat16>(st, a, s, rs, w) : memory_prompt_go<float>(st, a, s, rs, w);
+    cudaError_t e;
+    if (use_tc(s, bf16, a.n)) {
+        if ((a.n + MEMORY_TC_CHUNK - 1) / MEMORY_TC_CHUNK > GT_MAX_CHUNKS) return cudaErrorInvalidValue;
+        g_kernel_launches++;
+        k_memory_gates<MEMORY_TC_CHUNK / 32><<<s.heads, GT_THREADS, 0, st>>>(a.gates, a.ldi, a.n, s, (float*)rs.s1, w);
+        e = launch_memory_tc(st, a, s, rs, w);
+    } else {
+        e = bf16 ? memory_prompt_go<__nv_bfloat16>(st, a, s, rs, w) : memory_prompt_go<float>(st, a, s, rs, w);
+    }
     if (e != cudaSuccess) return e;
     const int off = 2 * s.heads * s.dim + s.heads * s.vdim;
     const void* gate = bf16 ? (const void*)((const __nv_bfloat16*)a.p + off) : (const void*)((const float*)a.p + off);

@@ -23,7 +23,8 @@ struct MemoryWork {
     double *a = nullptr, *g = nullptr;                   // [H][n]: log weight of token j in token t's sum = a[t] + g[j] (same chunk)
     float *carry = nullptr, *write = nullptr, *m = nullptr;  // [H][n]: weight of the chunk's first state; of token j in the next; m
     float* keep = nullptr;                               // [H][chunks]: weight of the chunk's first state in the next
-    float* S = nullptr;                                  // [chunks][H][vdim + 1][dimp] states at the chunks' starts
+    float* S = nullptr;                                  // [chunks][H][vdim + 1][dimp] chunk sums, then states at the chunks' starts
+    void *S_hi = nullptr, *S_lo = nullptr;               // bf16 [chunks][H][vdim + 1][dimp]: the latter of the tensor-core form
     float* o = nullptr;                                  // [n][H * vdim] read-outs
     uint32_t* err = nullptr;                             // device word for expired waits
 };
@@ -39,6 +40,11 @@ struct MemoryArgs {
 // Consecutive tokens of one sequence: read-outs, normalised and gated, to out act [n][ldo].
 cudaError_t launch_memory_prompt(cudaStream_t st, bool bf16, const MemoryArgs& a, const MemoryShape& s, const RowState& rs, const MemoryWork& w,
                                  void* out, int ldo);
+// Its tensor-core form (memory_tc.cu): everything between the gates and the output norm, bf16, portions of at least
+// MEMORY_TC_MIN_ROWS tokens.
+constexpr int MEMORY_TC_CHUNK = 128, MEMORY_TC_MIN_ROWS = 65;
+bool memory_tc_supported(const MemoryShape& s);
+cudaError_t launch_memory_tc(cudaStream_t st, const MemoryArgs& a, const MemoryShape& s, const RowState& rs, const MemoryWork& w);
 // One decode token per row.
 void launch_memory_step(cudaStream_t st, bool bf16, const MemoryArgs& a, const MemoryShape& s, const RowState& rs, void* out, int ldo);
 
