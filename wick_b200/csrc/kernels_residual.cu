@@ -8,15 +8,16 @@ namespace wick {
 
 namespace {
 
-constexpr int RN_THREADS = 256;
+constexpr int RN_THREADS = 256;  // of the form for any width
 
+template <int TH>
 __device__ __forceinline__ float block_sum(float v, float* red, int tid) {
     v = warp_sum(v);
     if ((tid & 31) == 0) red[tid >> 5] = v;
     __syncthreads();
     float t = 0.0f;
 #pragma unroll
-    for (int i = 0; i < RN_THREADS / 32; i++) t += red[i];
+    for (int i = 0; i < TH / 32; i++) t += red[i];
     return t;
 }
 
@@ -33,30 +34,28 @@ __device__ __forceinline__ void put4(T* p, const float4& q) {
     }
 }
 
-// NV > 0: NV groups of four coordinates per thread in registers (W a multiple of 4, at most 4 * NV * RN_THREADS);
+// TH threads.  NV > 0: NV groups of four coordinates per thread in registers (W a multiple of 4, at most 4 * NV * TH);
 // NV == 0: any W, one coordinate at a time through shared memory.
-template <class T, int NV>
-__global__ void __launch_bounds__(RN_THREADS) k_residual_norm(const __grid_constant__ ResidualArgs a) {
+template <class T, int NV, int TH>
+__global__ void __launch_bounds__(TH) k_residual_norm(const __grid_constant__ ResidualArgs a) {
     extern __shared__ float row_sh[];  // NV == 0: [W]
-    __shared__ float red[2][RN_THREADS / 32];
+    __shared__ float red[2][TH / 32];
     const int tid = threadIdx.x, W = a.W, row = blockIdx.x;
     constexpr int N4 = NV > 0 ? NV : 1;
-    float4 gain[N4], post[N4];
-    if constexpr (NV > 0) {  // weights: readable before the kernel in front has finished
-#pragma unroll
-        for (int i = 0; i < N4; i++) {
-            const int c = (i * RN_THREADS + tid) * 4;
-            if (c < W) {
-                if (a.gain) gain[i] = *reinterpret_cast<const float4*>(a.gain + c);
-                if (a.post || a.shift) post[i] = *reinterpret_cast<const float4*>((a.post ? a.post : a.shift) + c);
-            }
-        }
+    constexpr bool EARLY = NV == 1;  // weights are readable before the kernel in front has finished; otherwise registers count more
+    const float* post_row = a.post ? a.post : a.shift;
+    float4 early_gain = {}, early_post = {};
+    if (EARLY && tid * 4 < W) {
+        if (a.gain) early_gain = *reinterpret_cast<const float4*>(a.gain + tid * 4);
+        if (post_row) early_post = *reinterpret_cast<const float4*>(post_row + tid * 4);
     }
+    auto gain_at = [&](int c) { return EARLY ? early_gain : __ldg(reinterpret_cast<const float4*>(a.gain + c)); };
+    auto post_at = [&](int c) { return EARLY ? early_post : __ldg(reinterpret_cast<const float4*>(post_row + c)); };
     pdl_launch_next();
     pdl_wait();
     const int src = a.rows ? a.rows[row] : row;
     float* x = a.x + (size_t)src * W;
-    const __nv_bfloat16* e = a.embed ? a.embed + (size_t)(a.tokens ? a.tokens[src] : a.ctl->token) * a.ld_embed : nullptr;
+    const __nv_bfloat16* e = a.embed && (a.init || !a.gain) ? a.embed + (size_t)(a.tokens ? a.tokens[src] : a.ctl->token) * a.ld_embed : nullptr;
     const float* fr = a.frames ? a.frames + (size_t)src * W : nullptr;
     auto start = [&](int c) { return e ? __bfloat162float(e[c]) : fr[c]; };
     auto y_row = [&](int p) { return a.y + (size_t)(a.y_rows ? a.y_rows[src * a.y_parts + p] : src * a.y_parts + p) * a.ldy; };
@@ -67,7 +66,7 @@ __global__ void __launch_bounds__(RN_THREADS) k_residual_norm(const __grid_const
         float ss = 0.0f;
 #pragma unroll
         for (int i = 0; i < N4; i++) {
-            const int c = (i * RN_THREADS + tid) * 4;
+            const int c = (i * TH + tid) * 4;
             if (c < W) {
                 if (a.init) v[i] = make_float4(start(c), start(c + 1), start(c + 2), start(c + 3));
                 else if (a.y && !a.post) v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -76,29 +75,42 @@ __global__ void __launch_bounds__(RN_THREADS) k_residual_norm(const __grid_const
         }
         if (a.y) {
             float4 u[N4];
+            const float* y = y_row(0);
 #pragma unroll
             for (int i = 0; i < N4; i++) {
-                const int c = (i * RN_THREADS + tid) * 4;
-                if (c < W) {
-                    u[i] = *reinterpret_cast<const float4*>(y_row(0) + c);
-                    for (int p = 1; p < a.y_parts; p++) {
-                        const float4 t = *reinterpret_cast<const float4*>(y_row(p) + c);
+                const int c = (i * TH + tid) * 4;
+                if (c < W) u[i] = *reinterpret_cast<const float4*>(y + c);
+            }
+            for (int p = 1; p < a.y_parts; p++) {
+                y = y_row(p);
+#pragma unroll
+                for (int i = 0; i < N4; i++) {
+                    const int c = (i * TH + tid) * 4;
+                    if (c < W) {
+                        const float4 t = *reinterpret_cast<const float4*>(y + c);
                         u[i].x += t.x; u[i].y += t.y; u[i].z += t.z; u[i].w += t.w;
                     }
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < N4; i++) {
+                const int c = (i * TH + tid) * 4;
+                if (c < W) {
                     u[i].x *= a.y_scale; u[i].y *= a.y_scale; u[i].z *= a.y_scale; u[i].w *= a.y_scale;
                     ss = fmaf(u[i].x, u[i].x, fmaf(u[i].y, u[i].y, fmaf(u[i].z, u[i].z, fmaf(u[i].w, u[i].w, ss))));
                 }
             }
-            const float r = a.post ? 1.0f / sqrtf(block_sum(ss, red[0], tid) / (float)W + a.eps) : 1.0f;
+            const float r = a.post ? 1.0f / sqrtf(block_sum<TH>(ss, red[0], tid) / (float)W + a.eps) : 1.0f;
 #pragma unroll
             for (int i = 0; i < N4; i++) {
-                const int c = (i * RN_THREADS + tid) * 4;
+                const int c = (i * TH + tid) * 4;
                 if (c < W) {
+                    const float4 g = post_at(c);
                     if (a.post) {
-                        v[i].x = fmaf(u[i].x * r, post[i].x, v[i].x); v[i].y = fmaf(u[i].y * r, post[i].y, v[i].y);
-                        v[i].z = fmaf(u[i].z * r, post[i].z, v[i].z); v[i].w = fmaf(u[i].w * r, post[i].w, v[i].w);
+                        v[i].x = fmaf(u[i].x * r, g.x, v[i].x); v[i].y = fmaf(u[i].y * r, g.y, v[i].y);
+                        v[i].z = fmaf(u[i].z * r, g.z, v[i].z); v[i].w = fmaf(u[i].w * r, g.w, v[i].w);
                     } else {
-                        v[i].x = u[i].x + post[i].x; v[i].y = u[i].y + post[i].y; v[i].z = u[i].z + post[i].z; v[i].w = u[i].w + post[i].w;
+                        v[i].x = u[i].x + g.x; v[i].y = u[i].y + g.y; v[i].z = u[i].z + g.z; v[i].w = u[i].w + g.w;
                     }
                 }
             }
@@ -106,25 +118,28 @@ __global__ void __launch_bounds__(RN_THREADS) k_residual_norm(const __grid_const
         ss = 0.0f;
 #pragma unroll
         for (int i = 0; i < N4; i++) {
-            const int c = (i * RN_THREADS + tid) * 4;
+            const int c = (i * TH + tid) * 4;
             if (c < W) {
                 if (a.store_x && (a.y || a.init)) *reinterpret_cast<float4*>(x + c) = v[i];
                 ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, ss))));
             }
         }
         if (a.gain) {
-            const float r = 1.0f / sqrtf(block_sum(ss, red[1], tid) / (float)W + a.eps);
+            const float r = 1.0f / sqrtf(block_sum<TH>(ss, red[1], tid) / (float)W + a.eps);
 #pragma unroll
             for (int i = 0; i < N4; i++) {
-                v[i].x = v[i].x * r * gain[i].x; v[i].y = v[i].y * r * gain[i].y;
-                v[i].z = v[i].z * r * gain[i].z; v[i].w = v[i].w * r * gain[i].w;
+                const int c = (i * TH + tid) * 4;
+                if (c < W) {
+                    const float4 g = gain_at(c);
+                    v[i].x = v[i].x * r * g.x; v[i].y = v[i].y * r * g.y; v[i].z = v[i].z * r * g.z; v[i].w = v[i].w * r * g.w;
+                }
             }
         }
         for (int p = 0; p < outs; p++) {
             T* h = h_row(p);
 #pragma unroll
             for (int i = 0; i < N4; i++) {
-                const int c = (i * RN_THREADS + tid) * 4;
+                const int c = (i * TH + tid) * 4;
                 if (c < W) {
                     put4(h + c, v[i]);
                     if (!a.gain) put4(h + W + c, make_float4(start(c), start(c + 1), start(c + 2), start(c + 3)));
@@ -135,17 +150,17 @@ __global__ void __launch_bounds__(RN_THREADS) k_residual_norm(const __grid_const
     } else {
         float ss = 0.0f, r = 1.0f;
         if (a.y) {
-            for (int c = tid; c < W; c += RN_THREADS) {
+            for (int c = tid; c < W; c += TH) {
                 float u = 0.0f;
                 for (int p = 0; p < a.y_parts; p++) u += y_row(p)[c];
                 u *= a.y_scale;
                 row_sh[c] = u;
                 ss = fmaf(u, u, ss);
             }
-            if (a.post) r = 1.0f / sqrtf(block_sum(ss, red[0], tid) / (float)W + a.eps);
+            if (a.post) r = 1.0f / sqrtf(block_sum<TH>(ss, red[0], tid) / (float)W + a.eps);
         }
         ss = 0.0f;
-        for (int c = tid; c < W; c += RN_THREADS) {  // the coordinates this thread wrote
+        for (int c = tid; c < W; c += TH) {  // the coordinates this thread wrote
             float v;
             if (a.y && !a.post) v = row_sh[c] + a.shift[c];
             else {
@@ -156,8 +171,8 @@ __global__ void __launch_bounds__(RN_THREADS) k_residual_norm(const __grid_const
             row_sh[c] = v;
             ss = fmaf(v, v, ss);
         }
-        r = a.gain ? 1.0f / sqrtf(block_sum(ss, red[1], tid) / (float)W + a.eps) : 1.0f;
-        for (int c = tid; c < W; c += RN_THREADS) {
+        r = a.gain ? 1.0f / sqrtf(block_sum<TH>(ss, red[1], tid) / (float)W + a.eps) : 1.0f;
+        for (int c = tid; c < W; c += TH) {
             const float v = a.gain ? row_sh[c] * r * a.gain[c] : row_sh[c];
             for (int p = 0; p < outs; p++) {
                 T* h = h_row(p);
@@ -169,20 +184,28 @@ __global__ void __launch_bounds__(RN_THREADS) k_residual_norm(const __grid_const
     }
 }
 
+template <class T, int NV, int TH>
+void residual_launch(cudaStream_t st, const ResidualArgs& a, size_t smem = 0) {
+    if (smem > 40 * 1024) cudaFuncSetAttribute(k_residual_norm<T, NV, TH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    launch_pdl(k_residual_norm<T, NV, TH>, dim3(a.n), dim3(TH), smem, st, a);
+}
+
 template <class T>
 void residual_go(cudaStream_t st, const ResidualArgs& a) {
-    const dim3 grid(a.n), block(RN_THREADS);
-    const int groups = (a.W + 4 * RN_THREADS - 1) / (4 * RN_THREADS);
-    if (a.W % 4 == 0 && (!a.y || a.ldy % 4 == 0) && groups <= 8) {
-        if (groups <= 1) launch_pdl(k_residual_norm<T, 1>, grid, block, 0, st, a);
-        else if (groups <= 2) launch_pdl(k_residual_norm<T, 2>, grid, block, 0, st, a);
-        else if (groups <= 4) launch_pdl(k_residual_norm<T, 4>, grid, block, 0, st, a);
-        else launch_pdl(k_residual_norm<T, 8>, grid, block, 0, st, a);
-        return;
+    const int fours = a.W % 4 == 0 && (!a.y || a.ldy % 4 == 0) ? a.W / 4 : 0;
+    if (!fours || fours > 4096) return residual_launch<T, 0, RN_THREADS>(st, a, (size_t)a.W * 4);
+    if (a.n >= 256) {  // throughput: small CTAs, four loads of x and of y in flight per thread
+        if (fours <= 4 * 64) return residual_launch<T, 4, 64>(st, a);
+        if (fours <= 4 * 128) return residual_launch<T, 4, 128>(st, a);
+        if (fours <= 4 * 256) return residual_launch<T, 4, 256>(st, a);
+    } else {           // latency: many threads
+        if (fours <= 128) return residual_launch<T, 1, 128>(st, a);
+        if (fours <= 256) return residual_launch<T, 1, 256>(st, a);
+        if (fours <= 512) return residual_launch<T, 1, 512>(st, a);
     }
-    const size_t smem = (size_t)a.W * 4;
-    if (smem > 40 * 1024) cudaFuncSetAttribute(k_residual_norm<T, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    launch_pdl(k_residual_norm<T, 0>, grid, block, smem, st, a);
+    if (fours <= 1024) return residual_launch<T, 2, 512>(st, a);
+    if (fours <= 2048) return residual_launch<T, 4, 512>(st, a);
+    return residual_launch<T, 8, 512>(st, a);
 }
 
 }  // namespace
