@@ -31,6 +31,7 @@ struct GbParams {
     int n;
     int act;
     float scale, softcap;
+    int block_rows, x_step, y_step;  // > 0: block-diagonal (DenseBlocks)
     int experts;               // > 0: one matrix of m rows per expert, rows of X sorted by expert
     const int* expert_start;   // [experts + 1]
     uint32_t* err;
@@ -47,7 +48,8 @@ struct GbShape {
 };
 
 struct GbTile {
-    int job, m0, n0, n_end, w_row;  // w_row: where rows m0.. are in the weight map
+    int job, m0, m_end, n0, n_end;
+    int w_row, x_col, y_col;  // where the tile's rows are in the weight map, its first column of X, and rows' places in Y
 };
 // Experts: expert_tiles[e] = tiles before those of expert e.
 template <bool EXPERTS>
@@ -67,12 +69,27 @@ __device__ __forceinline__ GbTile gb_tile(const GbParams& p, int t, int tiles_n,
         r.m0 = local / tiles_n * GB_M;
         r.n0 = s0 + local % tiles_n * bn;
         r.w_row = lo * p.m[0] + r.m0;
+        r.m_end = p.m[0];
+        r.x_col = 0;
+        r.y_col = r.m0;
     } else {
         r.job = t >= p.tile_start[1] ? 1 : 0;
         const int local = t - p.tile_start[r.job];
-        r.m0 = r.w_row = local / tiles_n * GB_M;
         r.n0 = local % tiles_n * bn;
         r.n_end = p.n;
+        const int mt = local / tiles_n;
+        if (p.block_rows > 0) {
+            const int per = (p.block_rows + GB_M - 1) / GB_M, b = mt / per;
+            r.m0 = mt % per * GB_M;
+            r.m_end = p.block_rows;
+            r.w_row = b * p.block_rows + r.m0;
+            r.x_col = b * p.x_step;
+            r.y_col = b * p.y_step + r.m0;
+        } else {
+            r.m0 = r.w_row = r.y_col = mt * GB_M;
+            r.m_end = p.m[r.job];
+            r.x_col = 0;
+        }
     }
     return r;
 }
@@ -153,7 +170,7 @@ __global__ void __launch_bounds__(GB_THREADS, 1) k_gemm_bf16(const __grid_consta
                     mbar_arrive_expect_tx(bar, Sh::STAGE);
                     tma_load_2d(dst, &p.map_w[tl.job], bar, i * GB_K, tl.w_row);
                     if (DUAL) tma_load_2d(dst + GB_M * GB_K * 2, &p.map_w[1], bar, i * GB_K, tl.w_row);
-                    tma_load_2d(dst + Sh::A_BYTES, &p.map_x[tl.job], bar, i * GB_K, tl.n0);
+                    tma_load_2d(dst + Sh::A_BYTES, &p.map_x[tl.job], bar, tl.x_col + i * GB_K, tl.n0);
                 }
             }
         }
@@ -196,8 +213,8 @@ __global__ void __launch_bounds__(GB_THREADS, 1) k_gemm_bf16(const __grid_consta
             const uint32_t buf = it & 1;
             if (!mbar_wait_bounded(smem_u32(&acc_full[buf]), (it >> 1) & 1, abort, p.err, 14)) break;
             tc_fence_after();
-            const int row = tl.m0 + quarter * 32 + lane;
-            const bool row_ok = row < p.m[tl.job];
+            const int row = tl.y_col + quarter * 32 + lane;
+            const bool row_ok = tl.m0 + quarter * 32 + lane < tl.m_end;
             const uint32_t base = tmem + buf * 256 + ((uint32_t)(quarter * 32) << 16) + half * HALF;
             const bool f32 = p.f32[tl.job];
             const int ldy = p.ldy[tl.job];
@@ -247,6 +264,11 @@ __global__ void __launch_bounds__(GB_THREADS, 1) k_gemm_bf16(const __grid_consta
     }
 }
 
+int gb_tiles_m(const DenseCall& c, int job) {
+    if (c.blocks) return c.job[job].w.m / c.blocks.rows * ((c.blocks.rows + GB_M - 1) / GB_M);
+    return (c.job[job].w.m + GB_M - 1) / GB_M;
+}
+
 template <int BN, bool DUAL, bool EXPERTS>
 cudaError_t gb_launch(cudaStream_t st, GbParams& p, int jobs, const DenseCall& c, int sms) {
     using Sh = GbShape<BN, DUAL>;
@@ -254,13 +276,15 @@ cudaError_t gb_launch(cudaStream_t st, GbParams& p, int jobs, const DenseCall& c
     int t = 0;
     for (int i = 0; i < 2; i++) {
         p.tile_start[i] = t;
-        if (i < jobs) t += (c.job[i].w.m + GB_M - 1) / GB_M * tiles_n;
+        if (i < jobs) t += gb_tiles_m(c, i) * tiles_n;
     }
     p.tile_start[2] = t;
     if (EXPERTS) t = (c.job[0].w.m + GB_M - 1) / GB_M * (c.n / BN + std::min(c.n, copies));  // no more than this many
     for (int i = 0; i < c.count; i++) {
         cudaError_t e = encode_bf16_map(c.job[i].w.w, c.job[i].w.m * copies, c.job[i].w.k, c.job[i].w.ld, GB_M, &p.map_w[i]);
-        if (e == cudaSuccess && i < jobs) e = encode_bf16_map(c.job[i].x, c.n, c.job[i].w.k, c.job[i].ldx, BN, &p.map_x[i]);
+        // (blocks: columns of X beyond a block's k belong to others and meet zeros of W)
+        const int x_cols = c.blocks ? (c.job[i].w.m / c.blocks.rows - 1) * c.blocks.x_step + c.job[i].w.k : c.job[i].w.k;
+        if (e == cudaSuccess && i < jobs) e = encode_bf16_map(c.job[i].x, c.n, x_cols, c.job[i].ldx, BN, &p.map_x[i]);
         if (e != cudaSuccess) return e;
     }
     static cudaError_t configured = cudaFuncSetAttribute(k_gemm_bf16<BN, DUAL, EXPERTS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Sh::SMEM);
@@ -283,7 +307,7 @@ cudaError_t gb_bn(cudaStream_t st, GbParams& p, int jobs, const DenseCall& c, in
             const int used = std::min(c.n, c.experts.count);
             tiles = (long)((c.job[0].w.m + GB_M - 1) / GB_M) * std::max<long>(used, (long)(c.n / (double)bn + 0.5 * used));
         } else {
-            for (int i = 0; i < jobs; i++) tiles += (long)((c.job[i].w.m + GB_M - 1) / GB_M) * ((c.n + bn - 1) / bn);
+            for (int i = 0; i < jobs; i++) tiles += (long)gb_tiles_m(c, i) * ((c.n + bn - 1) / bn);
         }
         const double step = std::max(bn / 2.0, 32 + bn / 4.0) + 4.0;
         const double cost = (double)((tiles + sms - 1) / sms) * step;
@@ -304,7 +328,7 @@ cudaError_t gb_bn(cudaStream_t st, GbParams& p, int jobs, const DenseCall& c, in
 
 cudaError_t launch_dense_tc(cudaStream_t st, const DenseCall& c) {
     if (c.n <= 0) return cudaSuccess;
-    if (!c.err || c.blocks || (c.experts && (!c.experts.start || c.experts.count > MAX_EXPERTS || (c.count == 2 && !c.gated)))) return cudaErrorInvalidValue;
+    if (!c.err || (c.blocks && (c.count != 1 || c.blocks.x_step % 8 || c.experts)) || (c.experts && (!c.experts.start || c.experts.count > MAX_EXPERTS || (c.count == 2 && !c.gated)))) return cudaErrorInvalidValue;
     static int sms = 0;
     if (!sms) {
         int dev = 0, v = 0;
@@ -319,6 +343,9 @@ cudaError_t launch_dense_tc(cudaStream_t st, const DenseCall& c) {
     p.scale = c.scale;
     p.softcap = c.softcap;
     p.err = c.err;
+    p.block_rows = c.blocks.rows;
+    p.x_step = c.blocks.x_step;
+    p.y_step = c.blocks.y_step;
     p.experts = c.experts.count;
     p.expert_start = c.experts.start;
     const int jobs = c.gated ? 1 : c.count;

@@ -263,7 +263,8 @@ void launch_dense_simt(cudaStream_t st, bool bf16, const DenseCall& c) {
 }
 
 cudaError_t launch_dense(cudaStream_t st, bool bf16, const DenseCall& c) {
-    if (c.blocks || (c.experts ? !c.experts.start : c.n <= DENSE_ROWS_MAX)) launch_dense_rows(st, bf16, c);
+    const bool few = c.experts ? !c.experts.start : c.n <= DENSE_ROWS_MAX;
+    if (few || (c.blocks && (!bf16 || c.blocks.x_step % 8))) launch_dense_rows(st, bf16, c);  // (blocks of f32 models: a few rows at a time)
     else if (bf16) return launch_dense_tc(st, c);
     else launch_dense_simt(st, bf16, c);
     return cudaGetLastError();
