@@ -1,7 +1,7 @@
 // CPU oracle: a C++ restatement of the arithmetic of wick's own CPU path
 // (aarch64 / NEON integer flavour) for the LFM2 decode + prefill hot path.
 //
-// THIS FILE IS TEST INFRASTRUCTURE.  It is the checker the CUDA kernels are
+// THIS FILE IS TEST INFRASTRUCTURE.  It is what the CUDA kernels are
 // compared against and the timed CPU baseline of the benchmark.  Nothing in
 // the product library links, imports or calls it.
 //
